@@ -1,9 +1,11 @@
 // A feed-forward of routed experts: every token goes through `top` of E small feed-forwards W_down act(W_up h),
 // chosen by a router, and the results are added with the router's weights.
 //
-//   moe_route      logits z = W_r h in float32, scores s = sigmoid(z); the `top` experts with the largest s + bias[e]
-//                  are chosen (ties: the lower index), their weights are s * scale (the bias takes no part in the
-//                  weights, nothing is renormalised).  One block per token.
+//   moe_route      logits z = W_r h in float32, scores s = sigmoid(z), or softmax(z) over all experts; the `top` experts
+//                  with the largest s + bias[e] are chosen (ties: the lower index).  With `groups` > 1 the experts form
+//                  equal groups of neighbours and only experts of the `keep` groups with the largest best member can be
+//                  chosen.  Their weights are s * scale (the bias takes no part in the weights), divided by the sum
+//                  of the chosen s (+ 1e-20) with `renorm`.  One block per token.
 //   moe_pair_up    for every (token, chosen expert) pair: act(W_up[e] h), a warp per output value; the pair's expert
 //                  weight is streamed once per pair.  For a few tokens (decoding) and the float32 run.
 //   moe_pair_down  out[t] = base[t] + sum_k weight[t, k] W_down[e_k] a[t, k]: a warp per output value, the chosen
@@ -33,10 +35,34 @@ __device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&x)[4]) {
   x[0] = a.x, x[1] = a.y, x[2] = b.x, x[3] = b.y;
 }
 
+// Order-preserving key of a float: larger floats have larger keys (minus infinity 0x7fffff), NaN the smallest one, 1;
+// 0 is kept free for entries that cannot be chosen (any more).
+__device__ __forceinline__ unsigned choice_key(float v) {
+  if (v != v) return 1u;
+  const unsigned u = __float_as_uint(v);
+  return u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+
+// The entry with the largest key of keys[0 .. n), the lowest index among equals; the whole warp calls it.
+__device__ __forceinline__ int warp_best(const unsigned* keys, int n, int lane) {
+  unsigned best = 0;
+  int at = 0x7fffffff;
+  for (int e = lane; e < n; e += 32)
+    if (keys[e] > best) {
+      best = keys[e];
+      at = e;
+    }
+  const unsigned top = __reduce_max_sync(0xffffffffu, best);
+  return (int)__reduce_min_sync(0xffffffffu, (unsigned)(best == top ? at : 0x7fffffff));
+}
+
 template <typename T>
 __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ bias,
-                                 int* __restrict__ ids, float* __restrict__ wts, int W, int E, int top, float scale) {
-  extern __shared__ float score[];  // [E] scores, then [E] choice scores
+                                 int* __restrict__ ids, float* __restrict__ wts, int W, int E, int top, float scale,
+                                 int softmax, int groups, int keep, int renorm) {
+  extern __shared__ float score[];  // [E] scores (softmax: logits first), [E] choice keys, [groups] the groups' keys
+  unsigned* key = reinterpret_cast<unsigned*>(score + E);
+  unsigned* group_key = key + E;
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
@@ -63,27 +89,61 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
     }
     dot = warp_sum(dot);
     if (lane == 0) {
-      const float s = 1.0f / (1.0f + expf(-dot));
-      score[e] = s;
-      score[E + e] = s + (bias ? bias[e] : 0.f);
+      if (softmax) {
+        score[e] = dot;
+      } else {
+        const float s = 1.0f / (1.0f + expf(-dot));
+        score[e] = s;
+        key[e] = choice_key(s + (bias ? bias[e] : 0.f));
+      }
     }
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
-    for (int k = 0; k < top; ++k) {
-      int best = -1;
-      float bv = -INFINITY;
-      for (int e = 0; e < E; ++e) {
-        const float v = score[E + e];
-        if (v > bv || (best < 0 && !(v < bv))) {  // the second clause takes a NaN rather than nothing
-          bv = v;
-          best = e;
-        }
-      }
-      ids[(size_t)t * top + k] = best;
-      wts[(size_t)t * top + k] = score[best] * scale;
-      score[E + best] = -INFINITY;
+  if (warp > 0) return;
+  if (softmax) {  // the sum's order is the lanes' and then the warp's: a token's scores do not depend on the batch
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, score[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) sum += expf(score[e] - mx);
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      const float z = score[e], s = expf(z - mx) / sum;
+      key[e] = choice_key(bias ? s + bias[e] : z);  // without a bias the logits themselves: the same order, no underflow
+      score[e] = s;
     }
+    __syncwarp();
+  }
+  if (groups > 1) {
+    const int per = E / groups;
+    for (int n = lane; n < groups; n += 32) {
+      unsigned best = 0;
+      for (int e = n * per; e < (n + 1) * per; ++e) best = max(best, key[e]);
+      group_key[n] = best;
+    }
+    __syncwarp();
+    for (int k = 0; k < keep; ++k) {
+      const int n = warp_best(group_key, groups, lane);
+      if (lane == 0) group_key[n] = 0;  // kept
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (group_key[e / per] != 0) key[e] = 0;  // a group that is not kept
+    __syncwarp();
+  }
+  float total = 0.f;
+  int mine = -1;  // lane k keeps the k-th choice (top <= MOE_MAX_TOP = 32)
+  for (int k = 0; k < top; ++k) {
+    const int e = warp_best(key, E, lane);
+    if (lane == k) mine = e;
+    total += score[e];
+    __syncwarp();
+    if (lane == 0) key[e] = 0;
+    __syncwarp();
+  }
+  if (lane < top) {
+    ids[(size_t)t * top + lane] = mine;
+    wts[(size_t)t * top + lane] = renorm ? score[mine] / (total + 1e-20f) * scale : score[mine] * scale;
   }
 }
 
@@ -159,13 +219,16 @@ __global__ void moe_pair_down_kernel(const T* __restrict__ a, const T* __restric
   else return Q3_ERR_DTYPE;
 
 // h: [T, W] in `dtype`; wr: float32 [E, W]; bias: float32 [E] or null; ids: int32 [T, top]; wts: float32 [T, top].
+// softmax: scores by softmax instead of a sigmoid; groups, keep: see the head of the file (1, 1: no groups); renorm: the
+// weights divided by the chosen scores' sum.
 extern "C" int q3_moe_route(const void* h, const float* wr, const float* bias, int* ids, float* wts, int dtype, int T, int W,
-                            int E, int top, float scale, cudaStream_t stream) {
+                            int E, int top, float scale, int softmax, int groups, int keep, int renorm, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (W <= 0 || E <= 0 || top <= 0 || top > E || top > q3::MOE_MAX_TOP || E > 4096) return Q3_ERR_SIZE;
-  Q3_BY_DTYPE(dtype, q3::launch(q3::moe_route_kernel<E_>, dim3(T), dim3(E >= 16 ? 512 : (E >= 8 ? 256 : 128)), (size_t)2 * E * sizeof(float),
+  if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups)) return Q3_ERR_SIZE;
+  Q3_BY_DTYPE(dtype, q3::launch(q3::moe_route_kernel<E_>, dim3(T), dim3(E >= 16 ? 512 : (E >= 8 ? 256 : 128)), (size_t)(2 * E + groups) * sizeof(float),
                                 stream,
-                                (const E_*)h, wr, bias, ids, wts, W, E, top, scale))
+                                (const E_*)h, wr, bias, ids, wts, W, E, top, scale, softmax, groups, keep, renorm))
   return q3::launch_status();
 }
 

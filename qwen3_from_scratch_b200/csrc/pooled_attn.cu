@@ -2,7 +2,8 @@
 // per block of P tokens.  A query at position i reads the tokens j with 0 <= i - j < window, and block b (the
 // positions b P .. b P + P - 1) once the whole block lies before the window: b P + P - 1 <= i - window.  A pooled key
 // is the mean of the block's keys as the pages hold them (after norm and rotation), a pooled value the mean of its
-// values; tokens and blocks share one softmax.  Scores may be capped: s <- cap * tanh(s / cap).
+// values; tokens and blocks share one softmax.  Scores may be capped: s <- cap * tanh(s / cap); a token's score may take
+// a bias per head and distance, and the softmax a sink per head (a learned logit without a key).
 //
 // Two caches per layer run: pages with one entry per token (planes k [G, D] and v [G, Dv]), of which the manager
 // keeps the last max(window, P) tokens' pages, and pages with one entry per block (planes pk and pv), kept for good.
@@ -161,7 +162,8 @@ pw_attn_ref_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const
                    const int* __restrict__ tok_seq, const int* __restrict__ table, int stride, int num_pages,
                    const int* __restrict__ ptable, int pstride, int num_ppages, int page_size, T* __restrict__ out, int ldo,
                    int Ttot, int H, int G, int D, int Dv, int window, int P, float scale, float cap, float out_scale,
-                   int block_limit, int* status) {
+                   int block_limit, const float* __restrict__ dist_bias, int dist_n, const float* __restrict__ sink,
+                   int* status) {
   pdl_wait();
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31;
@@ -209,6 +211,7 @@ pw_attn_ref_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const
     }
     float s = warp_sum(dot) * scale;
     if (cap > 0.f) s = cap * tanhf(s / cap);
+    if (dist_bias && !pooled) s += dist_bias[(size_t)h * dist_n + min(pos - idx, dist_n - 1)];
     const float m_new = fmaxf(m, s);
     const float corr = expf(m - m_new), p = expf(s - m_new);  // m = -inf at the first key: corr = 0
     l = fmaf(l, corr, p);
@@ -219,7 +222,11 @@ pw_attn_ref_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const
     }
     m = m_new;
   }
-  const float inv = l > 0.f ? out_scale / l : 0.f;
+  float inv = l > 0.f ? out_scale / l : 0.f;
+  if (sink) {  // one more exponential in the denominator, without a key or a value
+    const float top = fmaxf(m, sink[h]), corr = expf(m - top);
+    inv = out_scale * corr / fmaf(l, corr, expf(sink[h] - top));
+  }
 #pragma unroll
   for (int k = 0; k < PW_PER; ++k) {
     const int d = lane + 32 * k;
@@ -265,15 +272,19 @@ extern "C" int q3_pool_blocks(const void* k_pages, const void* v_pages, void* pk
 
 // q: [T, H, D]; out: rows of `ldo` values, head h at column h * Dv, multiplied by out_scale.  cap <= 0: no cap.
 // block_limit: only the first so many blocks are ever read (negative: all).  With P = 1 and the token pages given as
-// the block pages too, that is a window that also keeps a request's first `block_limit` tokens.
+// the block pages too, that is a window that also keeps a request's first `block_limit` tokens; with a window that
+// nothing reaches and block_limit 0, attention to every earlier token.
+// dist_bias: float32 [H, dist_n] or null: added to the (scaled, capped) score of a token n positions back, the last entry
+// from n = dist_n - 1 on.  sink: float32 [H] or null: exp(sink_h) joins the softmax's denominator.
 extern "C" int q3_pw_attn_ref(const void* q, const void* k_pages, const void* v_pages, const void* pk_pages,
                               const void* pv_pages, const int* positions, const int* tok_seq, const int* table, int stride,
                               int num_pages, const int* ptable, int pstride, int num_ppages, int page_size, void* out,
                               int ldo, int dtype, int T, int H, int G, int D, int Dv, int window, int P, float scale,
-                              float cap, float out_scale, int block_limit, int* status, cudaStream_t stream) {
+                              float cap, float out_scale, int block_limit, const float* dist_bias, int dist_n,
+                              const float* sink, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || D <= 0 || D > 32 * q3::PW_PER || Dv <= 0 || Dv > 32 * q3::PW_PER || window <= 0 ||
-      P <= 0 || page_size <= 0 || stride <= 0 || pstride <= 0)
+      P <= 0 || page_size <= 0 || stride <= 0 || pstride <= 0 || (dist_bias && dist_n <= 0))
     return Q3_ERR_SIZE;
   const long long blocks = ((long long)T * H + 3) / 4;
   if (blocks > 0x7fffffffll) return Q3_ERR_SIZE;
@@ -281,6 +292,6 @@ extern "C" int q3_pw_attn_ref(const void* q, const void* k_pages, const void* v_
                                 (const E*)k_pages, (const E*)v_pages, (const E*)pk_pages, (const E*)pv_pages, positions,
                                 tok_seq, table, stride, num_pages, ptable, pstride, num_ppages, page_size, (E*)out, ldo, T,
                                 H, G, D, Dv, window, P, scale, cap, out_scale, block_limit < 0 ? 0x7fffffff : block_limit,
-                                status))
+                                dist_bias, dist_n, sink, status))
   return q3::launch_status();
 }

@@ -36,7 +36,16 @@ struct PwShape {
 // tanh through one exponential: 1 - 2 / (e^(2x) + 1); absolute error of a few 1e-7, both tails exact
 __device__ __forceinline__ float pw_tanh(float x) { return 1.0f - __fdividef(2.0f, __expf(2.0f * x) + 1.0f); }
 
-template <int KT, int VT, bool DEC>
+// The sink joins a finished row: exp(sink) in the denominator, nothing in the numerator.  mx: the row's maximum in base-2
+// units; den and num are rescaled to the larger of it and the sink.
+__device__ __forceinline__ void pw_sink(float sink, float mx, float& den, float& num) {
+  const float s2 = sink * 1.4426950408889634f, top = fmaxf(mx, s2), corr = exp2f(mx - top);
+  den = fmaf(den, corr, exp2f(s2 - top));
+  num *= corr;
+}
+
+// BIAS: the form with a bias per head and distance and a sink per head.
+template <int KT, int VT, bool DEC, bool BIAS>
 __global__ void __launch_bounds__(PwShape<KT, VT, DEC>::WARPS * 32, PwShape<KT, VT, DEC>::MIN_BLOCKS)
 pw_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
                    const __nv_bfloat16* __restrict__ v_pages, const __nv_bfloat16* __restrict__ pk_pages,
@@ -44,7 +53,8 @@ pw_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
                    const int* __restrict__ q_start, const int* __restrict__ kv_len, const int* __restrict__ block_table,
                    int table_stride, int num_pages, const int* __restrict__ pooled_table, int ptable_stride,
                    int num_ppages, int page_size, int Hq, int Hkv, float scale, float cap, float out_scale, int window,
-                   int P, int block_limit, int splits, int T_total, float* __restrict__ part_o,
+                   int P, int block_limit, const float* __restrict__ dist_bias, int dist_n,
+                   const float* __restrict__ sink, int splits, int T_total, float* __restrict__ part_o,
                    float* __restrict__ part_ml, int* status) {
   pdl_wait();
   pdl_launch_dependents();
@@ -126,9 +136,16 @@ pw_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
   const __nv_bfloat16* q_warp = q_s + (wrow + (lane & 7) + ((lane >> 3) & 1) * 8) * KPITCH + (lane >> 4) * 8;
 
   int row_pos[2], row_lo[2], row_blocks[2];
+  [[maybe_unused]] const float* row_bias[2];  // BIAS: the row's head of the distance bias, and its last entry
+  [[maybe_unused]] float far_bias[2];
+  [[maybe_unused]] const int warp_pos = past + min(row0 + wrow, total_rows - 1) / g;  // position of the warp's first row
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int R = row0 + wrow + gid + 8 * r;
+    if constexpr (BIAS) {
+      row_bias[r] = dist_bias + (size_t)(hk * g + min(R, total_rows - 1) % g) * dist_n;
+      far_bias[r] = row_bias[r][dist_n - 1];
+    }
     row_pos[r] = R < total_rows ? past + R / g : pos_last;  // rows past the end compute something finite, unused
     row_lo[r] = max(0, row_pos[r] - window + 1);
     row_blocks[r] = min(row_lo[r] / P, block_limit);
@@ -168,16 +185,22 @@ pw_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
     }
     const bool pooled = vt < ptiles;
     const int base_n = (pooled ? vt : tile_lo + vt - ptiles) * PWM_BN;
+    // a tile whose every key is far from every row of the warp takes the last entry of the bias without a lookup
+    [[maybe_unused]] const bool near = BIAS && !pooled && warp_pos - (base_n + PWM_BN - 1) < dist_n - 1;
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         if (DEC && (nt >> 1) != warp) continue;
         const int n = base_n + nt * 8 + 2 * tid4 + (j & 1);
+        const int r = j >> 1;
         float v = s[nt][j] * scale;
         if (cap > 0.f) v = cap * pw_tanh(v * inv_cap);
+        if constexpr (BIAS) {
+          if (near) v += row_bias[r][min(max(row_pos[r] - n, 0), dist_n - 1)];
+          else if (!pooled) v += far_bias[r];
+        }
         v *= LOG2E;
-        const int r = j >> 1;
         const bool hidden = pooled ? n >= row_blocks[r] : (n > row_pos[r] || n < row_lo[r]);
         s[nt][j] = hidden ? -INFINITY : v;
       }
@@ -264,6 +287,7 @@ pw_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         den = fmaf(wgt, src[DV + 1], den);
         acc = fmaf(wgt, src[d], acc);
       }
+      if (BIAS && splits == 1 && sink) pw_sink(sink[hk * g + R % g], mx, den, acc);
       if (splits > 1) {
         const size_t row = ((size_t)sp * T_total + qs + R / g) * Hq + hk * g + R % g;
         part_o[row * DV + d] = acc;
@@ -294,7 +318,12 @@ pw_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
       for (int nt = 0; nt < 2 * VT; ++nt) *reinterpret_cast<float2*>(dst + nt * 8) = make_float2(o[nt][2 * r], o[nt][2 * r + 1]);
       continue;
     }
-    const float inv = l[r] > 0.f ? out_scale / l[r] : 0.f;
+    float inv = l[r] > 0.f ? out_scale / l[r] : 0.f;
+    if (BIAS && sink) {
+      float den = l[r], num = 1.f;
+      pw_sink(sink[hk * g + R % g], m[r], den, num);
+      inv = out_scale * num / den;
+    }
     __nv_bfloat16* dst = out + (size_t)(qs + R / g) * ldo + (size_t)(hk * g + R % g) * DV + 2 * tid4;
 #pragma unroll
     for (int nt = 0; nt < 2 * VT; ++nt)
@@ -306,7 +335,7 @@ pw_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
 // grid (tokens, heads), a thread per output value: the ranges' shares in ascending order.
 __global__ void pw_attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                      __nv_bfloat16* __restrict__ out, int ldo, int T_total, int Hq, int DV, int splits,
-                                     float out_scale) {
+                                     float out_scale, const float* __restrict__ sink) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x, h = blockIdx.y;
@@ -322,21 +351,23 @@ __global__ void pw_attn_merge_kernel(const float* __restrict__ part_o, const flo
       den = fmaf(w, part_ml[2 * row + 1], den);
       acc = fmaf(w, part_o[row * DV + d], acc);
     }
+    if (sink) pw_sink(sink[h], mx, den, acc);
     out[(size_t)t * ldo + (size_t)h * DV + d] = __float2bfloat16_rn(den > 0.f ? acc * (out_scale / den) : 0.f);
   }
 }
 
-template <int KT, int VT, bool DEC>
+template <int KT, int VT, bool DEC, bool BIAS>
 static int pw_attn_mma_launch(const void* q, const void* k_pages, const void* v_pages, const void* pk_pages,
                               const void* pv_pages, void* out, int ldo, const int* q_start, const int* kv_len,
                               const int* table, int stride, int num_pages, const int* ptable, int pstride, int num_ppages,
                               int page_size, int B, int max_q_len, int Hq, int Hkv, float scale, float cap, float out_scale,
-                              int window, int P, int block_limit, int T_total, float* part_o, float* part_ml,
-                              long long part_rows, int* status, cudaStream_t stream) {
+                              int window, int P, int block_limit, const float* dist_bias, int dist_n, const float* sink,
+                              int T_total, float* part_o, float* part_ml, long long part_rows, int* status,
+                              cudaStream_t stream) {
   using S = PwShape<KT, VT, DEC>;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(pw_attn_mma_kernel<KT, VT, DEC>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(pw_attn_mma_kernel<KT, VT, DEC, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          (int)S::SMEM_BYTES);
     if (e != cudaSuccess) return (int)e;
     configured = true;
@@ -354,14 +385,14 @@ static int pw_attn_mma_launch(const void* q, const void* k_pages, const void* v_
     splits = (int)(want < 1 ? 1 : (want > 32 ? 32 : want));
     if ((long long)B * splits > 65535) splits = 1;
   }
-  q3::launch(pw_attn_mma_kernel<KT, VT, DEC>, dim3((unsigned)tiles, Hkv, B * splits), dim3(S::WARPS * 32), S::SMEM_BYTES, stream,
+  q3::launch(pw_attn_mma_kernel<KT, VT, DEC, BIAS>, dim3((unsigned)tiles, Hkv, B * splits), dim3(S::WARPS * 32), S::SMEM_BYTES, stream,
              (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages,
              (const __nv_bfloat16*)pk_pages, (const __nv_bfloat16*)pv_pages, (__nv_bfloat16*)out, ldo, q_start, kv_len, table,
              stride, num_pages, ptable, pstride, num_ppages, page_size, Hq, Hkv, scale, cap, out_scale, window, P, block_limit,
-             splits, T_total, part_o, part_ml, status);
+             dist_bias, dist_n, sink, splits, T_total, part_o, part_ml, status);
   if (splits > 1)
     q3::launch(pw_attn_merge_kernel, dim3(T_total, Hq), dim3(S::DV < 128 ? S::DV : 128), 0, stream, (const float*)part_o,
-               (const float*)part_ml, (__nv_bfloat16*)out, ldo, T_total, Hq, S::DV, splits, out_scale);
+               (const float*)part_ml, (__nv_bfloat16*)out, ldo, T_total, Hq, S::DV, splits, out_scale, sink);
   return launch_status();
 }
 
@@ -376,35 +407,39 @@ extern "C" int q3_pw_attn_mma_takes(int D, int Dv) {
 // q: bf16 [T, Hq, D]; token pages k [pages, Hkv, page, D], v [.., Dv]; block pages pk, pv alike; out: rows of `ldo`
 // values, head h at column h * Dv, times out_scale.  cap <= 0: no cap.  part_o (float32, part_rows * Dv values) and part_ml
 // (float32, part_rows * 2 values), or null: scratch for a step of T tokens whose keys are cut into ranges (part_rows /
-// (T * Hq) of them at most).  block_limit: only the first so many blocks are ever read (negative: all).
+// (T * Hq) of them at most).  block_limit: only the first so many blocks are ever read (negative: all).  dist_bias,
+// dist_n, sink: as in q3_pw_attn_ref; a sink only with a bias.
 extern "C" int q3_pw_attn_mma(const void* q, const void* k_pages, const void* v_pages, const void* pk_pages,
                               const void* pv_pages, void* out, int ldo, const int* q_start, const int* kv_len,
                               const int* table, int stride, int num_pages, const int* ptable, int pstride, int num_ppages,
                               int page_size, int B, int max_q_len, int Hq, int Hkv, int D, int Dv, float scale, float cap,
-                              float out_scale, int window, int P, int block_limit, int T, float* part_o, float* part_ml,
-                              long long part_rows, int* status, cudaStream_t stream) {
+                              float out_scale, int window, int P, int block_limit, const float* dist_bias, int dist_n,
+                              const float* sink, int T, float* part_o, float* part_ml, long long part_rows, int* status,
+                              cudaStream_t stream) {
   if (block_limit < 0) block_limit = 0x7fffffff;  // all blocks
   if (B <= 0 || max_q_len <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || !q3_pw_attn_mma_takes(D, Dv) || page_size <= 0 || stride <= 0 || pstride <= 0 || B > 65535 ||
-      Hkv > 65535 || window <= 0 || P <= 0 || ldo % 2)
+      Hkv > 65535 || window <= 0 || P <= 0 || ldo % 2 || (dist_bias && dist_n <= 0) || (sink && !dist_bias))
     return Q3_ERR_SIZE;
   if ((uintptr_t)q % 16 || (uintptr_t)k_pages % 16 || (uintptr_t)v_pages % 16 || (uintptr_t)pk_pages % 16 ||
       (uintptr_t)pv_pages % 16 || (uintptr_t)out % 4)
     return Q3_ERR_ALIGN;
-#define Q3_PW_CASE(KT, VT)                                                                                              \
-  if (D == 16 * KT && Dv == 16 * VT) {                                                                                  \
-    if ((long long)max_q_len * (Hq / Hkv) <= 16)                                                                        \
-      return q3::pw_attn_mma_launch<KT, VT, true>(q, k_pages, v_pages, pk_pages, pv_pages, out, ldo, q_start, kv_len,   \
-                                                  table, stride, num_pages, ptable, pstride, num_ppages, page_size, B,  \
-                                                  max_q_len, Hq, Hkv, scale, cap, out_scale, window, P, block_limit, T, part_o, \
-                                                  part_ml, part_rows, status, stream);                                  \
-    return q3::pw_attn_mma_launch<KT, VT, false>(q, k_pages, v_pages, pk_pages, pv_pages, out, ldo, q_start, kv_len,    \
-                                                 table, stride, num_pages, ptable, pstride, num_ppages, page_size, B,   \
-                                                 max_q_len, Hq, Hkv, scale, cap, out_scale, window, P, block_limit, T, part_o, \
-                                                 part_ml, part_rows, status, stream);                                   \
+#define Q3_PW_CALL(KT, VT, DEC, BIAS)                                                                                    \
+  return q3::pw_attn_mma_launch<KT, VT, DEC, BIAS>(q, k_pages, v_pages, pk_pages, pv_pages, out, ldo, q_start, kv_len,   \
+                                                   table, stride, num_pages, ptable, pstride, num_ppages, page_size, B,  \
+                                                   max_q_len, Hq, Hkv, scale, cap, out_scale, window, P, block_limit,    \
+                                                   dist_bias, dist_n, sink, T, part_o, part_ml, part_rows, status, stream)
+#define Q3_PW_CASE(KT, VT)                                                                                               \
+  if (D == 16 * KT && Dv == 16 * VT) {                                                                                   \
+    const bool few = (long long)max_q_len * (Hq / Hkv) <= 16;                                                            \
+    if (few && dist_bias) Q3_PW_CALL(KT, VT, true, true);                                                                \
+    if (few) Q3_PW_CALL(KT, VT, true, false);                                                                            \
+    if (dist_bias) Q3_PW_CALL(KT, VT, false, true);                                                                      \
+    Q3_PW_CALL(KT, VT, false, false);                                                                                    \
   }
   Q3_PW_CASE(2, 2) Q3_PW_CASE(2, 4) Q3_PW_CASE(2, 8) Q3_PW_CASE(4, 2) Q3_PW_CASE(4, 4) Q3_PW_CASE(4, 8) Q3_PW_CASE(8, 2)
   Q3_PW_CASE(8, 4) Q3_PW_CASE(8, 8)
 #undef Q3_PW_CASE
+#undef Q3_PW_CALL
   return Q3_ERR_SIZE;
 }

@@ -157,11 +157,12 @@ _SIGNATURES = {
                        _c_void_p, _c_void_p],
     "q3_pw_attn_ref": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
                        _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-                       _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_int, _c_void_p, _c_void_p],
+                       _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_int, _c_void_p, _c_int, _c_void_p,
+                       _c_void_p, _c_void_p],
     "q3_pw_attn_mma": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
                        _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                       _c_int, _c_int, _c_float, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p,
-                       _c_ll, _c_void_p, _c_void_p],
+                       _c_int, _c_int, _c_float, _c_float, _c_float, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p,
+                       _c_int, _c_void_p, _c_void_p, _c_ll, _c_void_p, _c_void_p],
     "q3_mingru_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                        _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p],
     "q3_moe_grouped": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
@@ -171,7 +172,7 @@ _SIGNATURES = {
                                _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                _c_float, _c_void_p, _c_void_p],
     "q3_moe_route": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-                     _c_float, _c_void_p],
+                     _c_float, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "q3_moe_pairs": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
                      _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "q3_add_dyt": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
@@ -182,6 +183,16 @@ _SIGNATURES = {
     "q3_mlstm_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p,
                       _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                       _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
+    "q3_sum_norm": [_c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_float,
+                    _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
+                    _c_float, _c_void_p],
+    "q3_memory_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p,
+                       _c_void_p, _c_void_p, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int,
+                       _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+    "q3_memory_out": [_c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_void_p, _c_int, _c_int,
+                      _c_int, _c_int, _c_int, _c_void_p],
+    "q3_rotate_columns": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_void_p, _c_int, _c_int,
+                          _c_void_p],
     "q3_mlstm_out": [_c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_float, _c_float, _c_void_p, _c_int, _c_int, _c_int,
                      _c_int, _c_int, _c_void_p],
 }
@@ -231,6 +242,8 @@ def library() -> ctypes.CDLL:
                 lib.q3_mingru_chunk.restype = _c_int
                 lib.q3_mlstm_max_dim.argtypes = []
                 lib.q3_mlstm_max_dim.restype = _c_int
+                lib.q3_memory_max_dim.argtypes = []
+                lib.q3_memory_max_dim.restype = _c_int
                 lib.q3_moe_tile_rows.argtypes = []
                 lib.q3_moe_tile_rows.restype = _c_int
                 lib.q3_sample_scratch_bytes.argtypes = [_c_int]
@@ -1880,21 +1893,34 @@ def pool_blocks(k_pages: torch.Tensor, v_pages: torch.Tensor, pk_pages: torch.Te
     _done("pool_blocks", code, f"pool {pool}")
 
 
+def _dist_args(name: str, dist_bias: Optional[torch.Tensor], sink: Optional[torch.Tensor], heads: int) -> None:
+    for n, t in (("dist_bias", dist_bias), ("sink", sink)):
+        if t is not None:
+            _check(f"{name}.{n}", t, torch.float32)
+    if ((dist_bias is not None and (dist_bias.dim() != 2 or dist_bias.shape[0] != heads or dist_bias.shape[1] < 1))
+            or (sink is not None and sink.numel() != heads)):
+        raise KernelError(f"{name}: a distance bias is [heads, distances], a sink [heads], for {heads} heads")
+
+
 def pw_attn_ref(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, pk_pages: torch.Tensor,
                 pv_pages: torch.Tensor, positions: torch.Tensor, tok_seq: torch.Tensor, table: torch.Tensor,
                 ptable: torch.Tensor, out: torch.Tensor, window: int, pool: int, scale: float, softcap: Optional[float],
-                out_scale: float, status: torch.Tensor, block_limit: int = -1) -> None:
+                out_scale: float, status: torch.Tensor, block_limit: int = -1, dist_bias: Optional[torch.Tensor] = None,
+                sink: Optional[torch.Tensor] = None) -> None:
     """Softmax attention of q [T, H, D] over the last ``window`` tokens and the pooled blocks before them (with
     ``block_limit`` >= 0 only the first so many blocks are ever read: with blocks of one token whose pages are the
     token pages themselves, that is a window that also keeps a request's first tokens); head h's
     result times ``out_scale`` goes to columns h * vdim .. of ``out`` (rows of any pitch: a column view of a wider
-    buffer is taken).  A warp per (token, head), float32 arithmetic, keys one by one."""
+    buffer is taken).  ``dist_bias`` float32 [H, n]: added to the score of a token d positions back, entry min(d, n - 1);
+    ``sink`` float32 [H]: exp(sink_h) joins the softmax's denominator.  A warp per (token, head), float32 arithmetic,
+    keys one by one."""
     _check("pw_attn_ref.q", q)
     _pw_pages("pw_attn_ref", k_pages, v_pages, pk_pages, pv_pages, q.dtype)
     for name, t in (("positions", positions), ("tok_seq", tok_seq), ("table", table), ("ptable", ptable)):
         _check(f"pw_attn_ref.{name}", t, torch.int32)
     T, H, D = q.shape
     G, Dv = k_pages.shape[1], v_pages.shape[3]
+    _dist_args("pw_attn_ref", dist_bias, sink, H)
     if (out.dtype != q.dtype or out.dim() != 2 or out.shape[0] != T or out.shape[1] != H * Dv or out.stride(1) != 1
             or k_pages.shape[3] != D or not out.is_cuda):
         raise KernelError(f"pw_attn_ref: q {tuple(q.shape)}, k pages {tuple(k_pages.shape)}, out {tuple(out.shape)} "
@@ -1904,7 +1930,8 @@ def pw_attn_ref(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, p
                                     table.shape[1], k_pages.shape[0], ptable.data_ptr(), ptable.shape[1], pk_pages.shape[0],
                                     k_pages.shape[2], out.data_ptr(), out.stride(0), dtype_tag(q.dtype), T, H, G, D, Dv,
                                     int(window), int(pool), float(scale), float(softcap or 0.0), float(out_scale),
-                                    int(block_limit), status.data_ptr(), _stream())
+                                    int(block_limit), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[1],
+                                    _ptr(sink), status.data_ptr(), _stream())
     _done("pw_attn_ref", code, f"heads {H}/{G}, dim {D}, vdim {Dv}")
 
 
@@ -1916,12 +1943,16 @@ def pw_attention_fast(dtype: torch.dtype, dim: int, vdim: int) -> bool:
 def pw_attn_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, pk_pages: torch.Tensor,
                 pv_pages: torch.Tensor, ctx, table: torch.Tensor, ptable: torch.Tensor, out: torch.Tensor, window: int,
                 pool: int, scale: float, softcap: Optional[float], out_scale: float, status: torch.Tensor,
-                partial: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, block_limit: int = -1) -> None:
+                partial: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, block_limit: int = -1,
+                dist_bias: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> None:
     """The same attention as ``pw_attn_ref`` on the tensor cores (bfloat16): tiles of 64 entries of the block pages
     and of the token pages in one online softmax, 128 (token, head) rows of one kv head to a block.  ``partial``
     (``pw_attn_partial``): scratch with which a step of single tokens cuts every request's keys into ranges that run
-    side by side and are merged in ascending order."""
+    side by side and are merged in ascending order.  A ``sink`` only beside a ``dist_bias``."""
     _check("pw_attn_mma.q", q, torch.bfloat16)
+    _dist_args("pw_attn_mma", dist_bias, sink, q.shape[1])
+    if sink is not None and dist_bias is None:
+        raise KernelError("pw_attn_mma: a sink needs a distance bias (zeros, where there is none)")
     _pw_pages("pw_attn_mma", k_pages, v_pages, pk_pages, pv_pages, q.dtype)
     for name, t in (("q_start", ctx.q_start), ("kv_len", ctx.kv_len), ("table", table), ("ptable", ptable)):
         _check(f"pw_attn_mma.{name}", t, torch.int32)
@@ -1943,7 +1974,8 @@ def pw_attn_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, p
                                     ctx.kv_len.data_ptr(), table.data_ptr(), table.shape[1], k_pages.shape[0],
                                     ptable.data_ptr(), ptable.shape[1], pk_pages.shape[0], k_pages.shape[2], ctx.num_seqs,
                                     ctx.max_q_len, H, G, D, Dv, float(scale), float(softcap or 0.0), float(out_scale),
-                                    int(window), int(pool), int(block_limit), T, _ptr(part_o), _ptr(part_ml), part_rows,
+                                    int(window), int(pool), int(block_limit), _ptr(dist_bias),
+                                    0 if dist_bias is None else dist_bias.shape[1], _ptr(sink), T, _ptr(part_o), _ptr(part_ml), part_rows,
                                     status.data_ptr(), _stream())
     _done("pw_attn_mma", code, f"heads {H}/{G}, dim {D}, vdim {Dv}")
 
@@ -1963,16 +1995,20 @@ def pooled_window_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: tor
                             pv_pages: torch.Tensor, ctx, table: torch.Tensor, ptable: torch.Tensor, out: torch.Tensor,
                             window: int, pool: int, scale: float, softcap: Optional[float], out_scale: float,
                             status: torch.Tensor, partial: Optional[Tuple[torch.Tensor, torch.Tensor]] = None,
-                            block_limit: int = -1) -> None:
+                            block_limit: int = -1, dist_bias: Optional[torch.Tensor] = None,
+                            sink: Optional[torch.Tensor] = None) -> None:
     """The attention of a step's batch over windows and pooled blocks, by the kernel that suits dtype and shape: the
     tensor-core kernel for bfloat16 heads it takes (an output whose rows and start allow paired stores), the plain
     one for everything else."""
     if (pw_attention_fast(q.dtype, q.shape[2], v_pages.shape[3]) and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0):
         pw_attn_mma(q, k_pages, v_pages, pk_pages, pv_pages, ctx, table, ptable, out, window, pool, scale, softcap,
-                    out_scale, status, partial, block_limit)
+                    out_scale, status, partial, block_limit, dist_bias, sink)
     else:
         pw_attn_ref(q, k_pages, v_pages, pk_pages, pv_pages, ctx.positions, ctx.tok_seq, table, ptable, out, window, pool,
-                    scale, softcap, out_scale, status, block_limit)
+                    scale, softcap, out_scale, status, block_limit, dist_bias, sink)
+
+
+NO_WINDOW = 0x7fffffff  # a window that nothing reaches: every earlier token is read
 
 
 # ------------------------------------------------------------------ a recurrence gated by the current token alone
@@ -2036,10 +2072,15 @@ def mingru_scan(proj: torch.Tensor, z_col: int, u_col: int, g_col: int, z_bias: 
 MOE_MAX_TOP = 32  # experts per token that the routing kernel lists
 
 
+MOE_SCORES = {"sigmoid": 0, "softmax": 1}  # what makes scores of the router's logits
+
+
 def moe_route(h: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.Tensor, weights: torch.Tensor,
-              scale: float) -> None:
-    """Scores s = sigmoid(h router^T) in float32; ``ids`` [T, top] the experts with the largest s + bias, ``weights``
-    [T, top] their s * scale."""
+              scale: float, score: str = "sigmoid", groups: int = 1, keep: int = 1, renormalise: bool = False) -> None:
+    """Scores s = sigmoid(h router^T) (``score="softmax"``: softmax over the experts) in float32; ``ids`` [T, top] the
+    experts with the largest s + bias, ``weights`` [T, top] their s * scale (``renormalise``: divided by the sum of the
+    chosen s + 1e-20).  ``groups`` > 1: only experts of the ``keep`` groups of neighbours with the largest best member can
+    be chosen."""
     _check("moe_route.h", h)
     _check("moe_route.router", router, torch.float32)
     _check("moe_route.ids", ids, torch.int32)
@@ -2053,7 +2094,8 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor
             or (bias is not None and bias.numel() != E)):
         raise KernelError(f"moe_route: h {tuple(h.shape)}, router {tuple(router.shape)}, ids {tuple(ids.shape)}")
     code = library().q3_moe_route(h.data_ptr(), router.data_ptr(), _ptr(bias), ids.data_ptr(), weights.data_ptr(),
-                                  dtype_tag(h.dtype), T, W, E, top, float(scale), _stream())
+                                  dtype_tag(h.dtype), T, W, E, top, float(scale), MOE_SCORES[score], int(groups), int(keep),
+                                  1 if renormalise else 0, _stream())
     _done("moe_route", code, f"experts {E}, top {top}")
 
 
@@ -2366,3 +2408,153 @@ def mlstm_out(o: torch.Tensor, proj: torch.Tensor, g_col: int, weight: torch.Ten
                                   float(out_scale), out.data_ptr(), out.stride(0), dtype_tag(proj.dtype), T, int(heads),
                                   n // heads, _stream())
     _done("mlstm_out", code)
+
+
+# ------------------------------------------------------------------ sums into the stream and the norm for both sub-layers
+SUM_NORM_TERMS = 3  # open terms that one pass over the stream takes
+
+
+def sum_norm(stream: torch.Tensor, terms, term_eps: float, weight: torch.Tensor, out: torch.Tensor, eps: float,
+             second=None, rows: Optional[torch.Tensor] = None) -> None:
+    """stream += sum of ``terms``, then out = stream / rms(stream) * weight.  A term is (delta [T, W], weight or None,
+    scale): with a weight delta / sqrt(mean(delta^2) + term_eps) * weight * scale, without one delta as it is.
+    ``second``: (weight, out) of another norm of the same rows.  ``rows`` (int32): only these rows are worked out, into
+    ``out`` [len(rows), W], and the stream stays as it is."""
+    _check("sum_norm.stream", stream, torch.float32)
+    _check("sum_norm.out", out)
+    _check("sum_norm.weight", weight, torch.float32)
+    T, W = stream.shape
+    n = T
+    if rows is not None:
+        _check("sum_norm.rows", rows, torch.int32)
+        n = rows.numel()
+    if len(terms) > SUM_NORM_TERMS:
+        raise KernelError(f"sum_norm: {len(terms)} terms, the kernel takes {SUM_NORM_TERMS}")
+    if tuple(out.shape) != (n, W) or weight.numel() != W:
+        raise KernelError(f"sum_norm: stream {tuple(stream.shape)}, out {tuple(out.shape)}, weight {tuple(weight.shape)}")
+    args = []
+    for delta, w, scale in list(terms) + [(None, None, 1.0)] * (SUM_NORM_TERMS - len(terms)):
+        if delta is not None:
+            _check("sum_norm.delta", delta, out.dtype)
+            if tuple(delta.shape) != (T, W):
+                raise KernelError(f"sum_norm: stream {tuple(stream.shape)}, term {tuple(delta.shape)}")
+        if w is not None:
+            _check("sum_norm.term_weight", w, torch.float32)
+            if w.numel() != W:
+                raise KernelError(f"sum_norm: term weight {tuple(w.shape)} for width {W}")
+        args += [_ptr(delta), _ptr(w), float(scale)]
+    w2 = out2 = None
+    if second is not None:
+        w2, out2 = second
+        _check("sum_norm.second", w2, torch.float32)
+        _check("sum_norm.second", out2, out.dtype)
+        if tuple(out2.shape) != (n, W) or w2.numel() != W:
+            raise KernelError(f"sum_norm: second norm: out {tuple(out2.shape)}, weight {tuple(w2.shape)}")
+    code = library().q3_sum_norm(stream.data_ptr(), *args, len(terms), float(term_eps), weight.data_ptr(), out.data_ptr(),
+                                 _ptr(w2), _ptr(out2), _ptr(rows), n, dtype_tag(out.dtype), T, W, float(eps), _stream())
+    _done("sum_norm", code, f"rows {n}, width {W}")
+
+
+# ------------------------------------------------------------------ matrix memories: fixed decays, the gated delta rule
+def memory_max_dim() -> int:
+    """The largest key size per head that ``memory_scan`` takes."""
+    if "memory max dim" not in _DEVICE_FACTS:
+        _DEVICE_FACTS["memory max dim"] = int(library()._lib.q3_memory_max_dim())
+    return _DEVICE_FACTS["memory max dim"]
+
+
+class MemoryDecay:
+    """Fixed decays per head as the kernels want them, from float64 numbers: the decay, the decay minus one and the
+    decay's logarithm (minus infinity for a decay of zero), each rounded once to float32."""
+
+    def __init__(self, decay, device):
+        d = torch.tensor(list(decay), dtype=torch.float64)
+        self.decay = d.to(torch.float32).to(device)
+        self.minus_one = (d - 1.0).to(torch.float32).to(device)
+        self.log = torch.log(d).to(torch.float32).to(device)
+
+
+class DeltaGates:
+    """The delta rule's per-token scalars of a step: the pre-activations at columns ``b_col`` and ``a_col`` of ``proj`` [T, any]
+    (one per head each), ``a_log`` and ``dt_bias`` (float32 [heads])."""
+
+    def __init__(self, proj: torch.Tensor, b_col: int, a_col: int, a_log: torch.Tensor, dt_bias: torch.Tensor):
+        self.proj, self.b_col, self.a_col, self.a_log, self.dt_bias = proj, int(b_col), int(a_col), a_log, dt_bias
+
+
+def memory_scan(x: torch.Tensor, q_col: int, k_col: int, v_col: int, rule, q_scale: float, activation: str,
+                state: torch.Tensor, kv_heads: int, q_start: torch.Tensor, slot_ids: torch.Tensor, num_seqs: int,
+                out: torch.Tensor, status: torch.Tensor) -> None:
+    """A matrix memory per head over every request's tokens in order.  ``x`` [T, any]: q and k (kv_heads * dim each) and v
+    (heads * vdim) from the given columns, each through ``activation`` ("silu" or "none"); head h reads q and k of head
+    h / (heads / kv_heads).  ``rule``: a ``MemoryDecay`` (S <- decay S + k v^T, o = S^T q q_scale) or ``DeltaGates`` (the
+    gated delta rule, q and k brought to length one first).  ``state`` float32 [slots, heads, vdim, dim] (column by
+    column) is read and renewed; ``out`` float32 [T, heads * vdim]."""
+    _check("memory_scan.x", x)
+    _check("memory_scan.state", state, torch.float32)
+    _check("memory_scan.out", out, torch.float32)
+    for name, t in (("q_start", q_start), ("slot_ids", slot_ids)):
+        _check(f"memory_scan.{name}", t, torch.int32)
+    T, ld = x.shape
+    slots, H, Dv, D = state.shape
+    G = int(kv_heads)
+    if (tuple(out.shape) != (T, H * Dv) or G <= 0 or H % G or min(q_col, k_col, v_col) < 0
+            or max(q_col + G * D, k_col + G * D, v_col + H * Dv) > ld):
+        raise KernelError(f"memory_scan: x {tuple(x.shape)}, state {tuple(state.shape)}, out {tuple(out.shape)}")
+    if isinstance(rule, MemoryDecay):
+        gates = [None, 0, 0, 0, None, None, rule.decay.data_ptr(), rule.minus_one.data_ptr()]
+        if rule.decay.numel() != H or rule.minus_one.numel() != H:
+            raise KernelError(f"memory_scan: {rule.decay.numel()} decays for {H} heads")
+    else:
+        _check("memory_scan.gates", rule.proj, x.dtype)
+        for t in (rule.a_log, rule.dt_bias):
+            _check("memory_scan.gates", t, torch.float32)
+        if (rule.proj.shape[0] != T or min(rule.b_col, rule.a_col) < 0 or max(rule.b_col, rule.a_col) + H > rule.proj.shape[1]
+                or rule.a_log.numel() != H or rule.dt_bias.numel() != H):
+            raise KernelError(f"memory_scan: gates {tuple(rule.proj.shape)} for {H} heads")
+        gates = [rule.proj.data_ptr(), rule.proj.shape[1], rule.b_col, rule.a_col, rule.a_log.data_ptr(),
+                 rule.dt_bias.data_ptr(), None, None]
+    code = library().q3_memory_scan(x.data_ptr(), ld, int(q_col), int(k_col), int(v_col), *gates, float(q_scale),
+                                    activation_code(activation), state.data_ptr(), q_start.data_ptr(), slot_ids.data_ptr(),
+                                    slots, out.data_ptr(), dtype_tag(x.dtype), int(num_seqs), H, G, D, Dv,
+                                    status.data_ptr(), _stream())
+    _done("memory_scan", code, f"heads {H}/{G}, dim {D}, vdim {Dv}")
+
+
+MEMORY_GATES = {"silu": 0, "sigmoid": 3}
+
+
+def memory_out(o: torch.Tensor, proj: torch.Tensor, g_col: int, weight: Optional[torch.Tensor], eps: float, gate: str,
+               out: torch.Tensor, parts: int) -> None:
+    """out = o / rms(o) * weight * gate(proj[:, g_col:]), the root mean square over each of ``parts`` equal parts of a row;
+    ``weight``: one value per column, one per column of a part (shared by the parts), or None; ``gate``: "silu" or
+    "sigmoid"; o float32 [T, n]; ``out`` in the compute dtype, possibly a column view of a wider buffer."""
+    _check("memory_out.o", o, torch.float32)
+    _check("memory_out.proj", proj)
+    T, n = o.shape
+    if weight is not None:
+        _check("memory_out.weight", weight, torch.float32)
+    if (n % parts or out.dtype != proj.dtype or out.dim() != 2 or tuple(out.shape) != (T, n) or out.stride(1) != 1
+            or not out.is_cuda or (weight is not None and weight.numel() not in (n, n // parts)) or g_col < 0
+            or g_col + n > proj.shape[1] or proj.shape[0] != T):
+        raise KernelError(f"memory_out: o {tuple(o.shape)}, proj {tuple(proj.shape)}, out {tuple(out.shape)}")
+    shared = weight is not None and weight.numel() != n
+    code = library().q3_memory_out(o.data_ptr(), proj.data_ptr(), proj.shape[1], int(g_col), _ptr(weight), 1 if shared else 0,
+                                   float(eps), MEMORY_GATES[gate], out.data_ptr(), out.stride(0), dtype_tag(proj.dtype), T, n,
+                                   int(parts), _stream())
+    _done("memory_out", code)
+
+
+def rotate_columns(x: torch.Tensor, column: int, heads: int, dim: int, dims: int, freq: torch.Tensor, magnitude: float,
+                   positions: torch.Tensor) -> None:
+    """Rotates the first ``dims`` values of ``heads`` vectors of ``dim`` values from column ``column`` of ``x`` in place, value i
+    with value i + dims / 2, by position * freq (sines and cosines times ``magnitude``)."""
+    _check("rotate_columns.x", x)
+    _check("rotate_columns.positions", positions, torch.int32)
+    _check("rotate_columns.freq", freq, torch.float32)
+    T, ld = x.shape
+    if column < 0 or column + heads * dim > ld or freq.numel() < dims // 2 or positions.numel() != T:
+        raise KernelError(f"rotate_columns: x {tuple(x.shape)}, {heads} heads of {dim} from column {column}")
+    code = library().q3_rotate_columns(x.data_ptr(), ld, int(column), int(heads), int(dim), int(dims), freq.data_ptr(),
+                                       float(magnitude), positions.data_ptr(), dtype_tag(x.dtype), T, _stream())
+    _done("rotate_columns", code, f"rotated {dims} of {dim}")

@@ -2,7 +2,8 @@
 k, an optional position encoding and an optional sliding window), sigmoid attention whose values are its keys,
 softmax attention through a latent (one latent vector and one rotated key part per token, shared by the heads; with
 optional output gates and an optional sink in the softmax), softmax attention over a window and pooled blocks, and
-softmax attention over a window that also keeps a request's first tokens.
+softmax attention over a window that also keeps a request's first tokens, or over all tokens with a bias by distance and
+a sink.
 
 Reference: models/self_attn.py:300-386 (packed [T, hidden] input, merged QKV, head norm then
 rotation, keys/values written to pages, causal attention over the cache, output projection),
@@ -15,6 +16,7 @@ rotation and the page write itself, from the raw QKV projection.
 
 from __future__ import annotations
 
+import math
 from typing import Dict, List, Optional
 
 import torch
@@ -463,39 +465,67 @@ class PooledWindowAttention(Mixer):
         return self.out_proj(o)
 
 
+def distance_buckets(rows: int, most: float) -> List[int]:
+    """The row of a distance bias's table for every distance 0, 1, ... up to the first one from which all further ones
+    read the last row (see ``KeptWindowAttention``)."""
+    half = rows // 2
+    out = []
+    while not out or out[-1] < rows - 1:
+        n = len(out)
+        if n < half:
+            out.append(n)
+        elif half == 0 or most <= half:
+            out.append(rows - 1)
+        else:
+            out.append(min(rows - 1, half + math.floor(math.log(n / half) / math.log(most / half) * (rows - half))))
+    return out
+
+
 @register_part("mixer", "kept_window_attention")
 class KeptWindowAttention(Mixer):
-    """Grouped-query softmax attention over a sliding window that also keeps a request's first tokens.  With h the
-    input, H heads on G key/value heads (head n reads key/value head n // (H / G)), keys of ``dim`` and values of
-    ``vdim`` values:
+    """Grouped-query softmax attention over a sliding window that also keeps a request's first tokens, or (``window`` None)
+    over every earlier token.  With h the input, H heads on G key/value heads (head n reads key/value head n // (H / G)),
+    keys of ``dim`` and values of ``vdim`` values:
 
         q = W_q h;  k = W_k h;  v = W_v h;  q, k rotated by ``position`` (a part with ``frequencies()``: the first ``dims``
-        values of every head, value i with value i + dims / 2), the values not
-        score = q . k * scale;  position i reads j <= i with i - j < window or j < keep_first, the kept tokens at their
-        true positions;  ordinary softmax over what is read
+        values of every head, value i with value i + dims / 2; None: no rotation), the values not
+        score = q . k * scale + rel[bucket(i - j), head];  position i reads j <= i with i - j < window or j < keep_first, the
+        kept tokens at their true positions
+        softmax over what is read, the denominator with one more term exp(sink_head)
         out = W_o (concat_heads(softmax(scores) values) * sigmoid(W_g h))          (``gate``; without it no W_g)
 
+    ``bias`` = {"most": D, "rows": B}: the learned distance bias of T5 (Raffel et al., "Exploring the Limits of Transfer
+    Learning with a Unified Text-to-Text Transformer"), a table ``<name>.rel`` [B, H] whose rows stand for distances:
+    bucket(n) = n below B / 2, then min(B - 1, B / 2 + floor(ln(n / (B / 2)) / ln(D / (B / 2)) (B - B / 2))).  The table's
+    stored size says what B is ("rows" only sizes random weights); at load it becomes one value per head and distance up
+    to the distance from which the last row is read.  None: no bias.  It does not go with kept first tokens.
+    ``sink``: the learned logits ``<name>.sink`` [H]; nothing is scored or weighted by them and ``scale`` is not applied.
+
     One paged cache (planes ``k`` and ``v``), of which the manager keeps the pages of the last ``window`` tokens and those
-    of the first ``keep_first``.  The attention kernels are those of the window with pooled blocks, run with blocks of
+    of the first ``keep_first`` (all pages without a window).  The attention kernels are those of the window with pooled blocks, run with blocks of
     one token whose pages are the token pages themselves and with no more than ``keep_first`` of them.  ``scale`` is used
     as given.  Angles, scores, weights and the gate are float32 in every run.  ``names``: the tensors' names after the
     part's own."""
 
     graph_capturable = True
     splittable = True
-    NAMES = {"q": "q", "k": "k", "v": "v", "gate": "g", "out": "o"}
+    NAMES = {"q": "q", "k": "k", "v": "v", "gate": "g", "out": "o", "bias": "rel", "sink": "sink"}
 
     def __init__(self, name: str, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float,
-                 window: int, keep_first: int, position: PartSpec, gate: bool = True, names: Optional[Dict[str, str]] = None):
+                 window: Optional[int] = None, keep_first: int = 0, position: Optional[PartSpec] = None, gate: bool = True,
+                 names: Optional[Dict[str, str]] = None, bias: Optional[dict] = None, sink: bool = False):
         super().__init__(name)
         self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
         if self.num_heads % self.num_kv_heads:
             raise ValueError(f"{self.num_heads} query heads are not a multiple of {self.num_kv_heads} kv heads")
         self.dim, self.vdim, self.scale = int(dim), int(vdim), float(scale)
-        self.window, self.keep_first, self.has_gate = int(window), int(keep_first), bool(gate)
-        if self.window < 1 or self.keep_first < 0:
+        self.window, self.keep_first, self.has_gate = None if window is None else int(window), int(keep_first), bool(gate)
+        if (self.window is not None and self.window < 1) or self.keep_first < 0:
             raise ValueError(f"attention {name}: window {self.window} must be positive, keep_first {self.keep_first} not negative")
-        self.position = create_part("position", position, name=f"{name}.position")
+        self.bias, self.has_sink = dict(bias) if bias else None, bool(sink)
+        if self.bias and self.keep_first and self.window is not None:
+            raise ValueError(f"attention {name}: a distance bias and kept first tokens together are not built")
+        self.position = None if position is None else create_part("position", position, name=f"{name}.position")
         n = dict(self.NAMES)
         n.update(names or {})
         self.tensors = {k: f"{name}.{v}" for k, v in n.items()}
@@ -503,13 +533,15 @@ class KeptWindowAttention(Mixer):
     def weight_specs(self) -> List[WeightSpec]:
         t, w, H, G, D, Dv = self.tensors, self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim
         return [WeightSpec(t["q"], (H * D, w)), WeightSpec(t["k"], (G * D, w)), WeightSpec(t["v"], (G * Dv, w))] + (
-            [WeightSpec(t["gate"], (H * Dv, w))] if self.has_gate else []) + [
-            WeightSpec(t["out"], (w, H * Dv))] + self.position.weight_specs()
+            [WeightSpec(t["gate"], (H * Dv, w))] if self.has_gate else []) + (
+            [WeightSpec(t["bias"], (int(self.bias["rows"]), H), kind="vector", init="normal", free_dims=(0,))] if self.bias else []) + (
+            [WeightSpec(t["sink"], (H,), kind="vector", init="normal")] if self.has_sink else []) + [
+            WeightSpec(t["out"], (w, H * Dv))] + (self.position.weight_specs() if self.position is not None else [])
 
     def cache_spec(self):
         G = self.num_kv_heads
         return PagedCacheSpec((CachePlane("k", G, self.dim), CachePlane("v", G, self.vdim)), window=self.window,
-                              keep_first=self.keep_first)
+                              keep_first=self.keep_first if self.window is not None else 0)
 
     # ------------------------------------------------------------------ the two products and what lies between
     def input_weight(self, weights: Dict[str, torch.Tensor]) -> torch.Tensor:
@@ -527,7 +559,17 @@ class KeptWindowAttention(Mixer):
 
     def setup_core(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
         self.rt = rt
-        self.position.setup(rt, weights)
+        self.freq, self.magnitude, self.dims = torch.empty(0, dtype=torch.float32, device=rt.device), 1.0, 0
+        if self.position is not None:
+            self.position.setup(rt, weights)
+            self.freq, self.magnitude, self.dims = self.position.frequencies()
+        self.dist_bias, self.sink = None, weights[self.tensors["sink"]] if self.has_sink else None
+        if self.bias:
+            table = weights[self.tensors["bias"]]  # [rows, heads]
+            index = torch.tensor(distance_buckets(table.shape[0], float(self.bias["most"])), device=rt.device)
+            self.dist_bias = table[index].t().contiguous()
+        elif self.has_sink:  # the kernels take a sink beside a bias: one of zeros
+            self.dist_bias = torch.zeros(self.num_heads, 1, dtype=torch.float32, device=rt.device)
         self._q = rt.shared("kwattn.q", rt.max_tokens, self.num_heads, self.dim)
         self._partial = None
         if ops.pw_attention_fast(rt.dtype, self.dim, self.vdim):
@@ -545,15 +587,16 @@ class KeptWindowAttention(Mixer):
         T, H, G, D, Dv = proj.shape[0], self.num_heads, self.num_kv_heads, self.dim, self.vdim
         planes, table = ctx.pages(cache_id)
         k_pages, v_pages = planes["k"], planes["v"]
-        freq, mag, dims = self.position.frequencies()
         status = self.rt.status
         q = self._q[:T]
         k_col, v_col = column + H * D, column + (H + G) * D
-        ops.pw_qkv_post(proj, column, k_col, v_col, H, G, D, Dv, None, None, 0.0, dims, freq, mag, ctx.positions,
-                        ctx.tok_seq, table, q, k_pages, v_pages, write_cache, status)
+        ops.pw_qkv_post(proj, column, k_col, v_col, H, G, D, Dv, None, None, 0.0, self.dims, self.freq, self.magnitude,
+                        ctx.positions, ctx.tok_seq, table, q, k_pages, v_pages, write_cache, status)
+        window, first = (ops.NO_WINDOW, 0) if self.window is None else (self.window, self.keep_first)
         # the kept first tokens are "blocks" of one token read from the token pages, at most keep_first of them
-        ops.pooled_window_attention(q, k_pages, v_pages, k_pages, v_pages, ctx, table, table, out, self.window, 1,
-                                    self.scale, None, out_scale, status, self._partial, block_limit=self.keep_first)
+        ops.pooled_window_attention(q, k_pages, v_pages, k_pages, v_pages, ctx, table, table, out, window, 1,
+                                    self.scale, None, out_scale, status, self._partial, block_limit=first,
+                                    dist_bias=self.dist_bias, sink=self.sink)
         if self.has_gate:
             ops.sigmoid_gate(out, proj, v_col + G * Dv)
 

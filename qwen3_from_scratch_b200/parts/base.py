@@ -52,6 +52,8 @@ class WeightSpec:
       ``vector``  small parameter read by float32 arithmetic (norm weights):
                   held in float32 on the device whatever it was stored as.
       ``index``   integer table: held as int32.
+    free_dims: the dimensions whose size the folder decides (a table with as many rows as it was stored
+    with); ``shape`` then says what the random-weights writer makes.
     init: how the random-weights writer fills it (``normal``: N(0, 0.02);
       ``one_plus_normal``: 1 + N(0, 0.1); ``zeros``; ``identity_plus_normal``: a matrix, I + N(0, 0.1)).
     """
@@ -60,6 +62,12 @@ class WeightSpec:
     shape: Tuple[int, ...]
     kind: str = "matrix"
     init: str = "normal"
+    free_dims: Tuple[int, ...] = ()
+
+    def takes(self, shape) -> bool:
+        """Whether a stored tensor of this shape is what the part asks for."""
+        return len(shape) == len(self.shape) and all(
+            got == want or (i in self.free_dims and got > 0) for i, (got, want) in enumerate(zip(shape, self.shape)))
 
 
 # ---------------------------------------------------------------------- cache needs
@@ -255,6 +263,40 @@ class PendingNormed:
 
     delta: torch.Tensor  # [T, W] in the compute dtype
     norm: "Norm"
+
+
+@dataclass
+class PendingTerm:
+    """Something that still has to be added to the residual stream: ``delta`` as it is, or (with a ``weight``) brought to
+    unit root mean square over its row, times the weight, times ``scale``."""
+
+    delta: torch.Tensor  # [T, W] in the compute dtype
+    weight: Optional[torch.Tensor] = None  # float32 [W]
+    scale: float = 1.0
+
+
+@dataclass
+class PendingSum:
+    """Several terms that still have to be added to the residual stream (sub-layers side by side, mixers side by side whose
+    outputs are normed one by one).  ``eps``: inside the root of the terms' root mean squares."""
+
+    terms: Tuple[PendingTerm, ...]
+    eps: float = 0.0
+
+    @staticmethod
+    def of(*parts) -> "PendingSum":
+        """The sum of sub-layer outputs, each a tensor or a ``PendingSum``."""
+        terms, eps = [], None
+        for p in parts:
+            if not isinstance(p, PendingSum):
+                terms.append(PendingTerm(p))
+                continue
+            if any(t.weight is not None for t in p.terms):
+                if eps is not None and eps != p.eps:
+                    raise ValueError(f"terms with different epsilons ({eps}, {p.eps}) in one sum")
+                eps = p.eps
+            terms += p.terms
+        return PendingSum(tuple(terms), 0.0 if eps is None else eps)
 
 
 @dataclass

@@ -1,7 +1,8 @@
 """The arrangements of norms, mixer and feed-forward around the residual stream: the norm before each
 sub-layer (``pre_norm``), the norm after each sub-layer's sum (``post_norm``), the norm before each sub-layer
-of a model that keeps several residual streams per token (``hyper_pre_norm``), and a norm on both sides of each
-sub-layer (``sandwich_norm``, at the end of the file).
+of a model that keeps several residual streams per token (``hyper_pre_norm``), a norm on both sides of each
+sub-layer (``sandwich_norm``), and both sub-layers side by side on the same stream (``parallel_pre_norm``, at the end of
+the file).
 
 Pre-norm residual block: h = x + mixer(norm1(x)); y = h + feed_forward(norm2(h)).
 
@@ -21,7 +22,7 @@ import torch
 from ..registry import create_part, register_part
 from ..kernels import ops
 from .base import (EMBEDDING_OUTPUT, EMBEDDING_SIDE, LAYER_REPEAT, NEXT_NORM_WEIGHT, STREAM_SUMSQ, Block, PartSpec, PendingNormed,
-                   PendingStreamWrite, Runtime, StateSpec, StepContext, WeightSpec)
+                   PendingStreamWrite, PendingSum, Runtime, StateSpec, StepContext, WeightSpec)
 from .linear import Linear
 
 
@@ -437,3 +438,52 @@ class SandwichNormBlock(Block):
         ops.side_gate(self.side_gate(x), shared[EMBEDDING_SIDE], int(self.side["column"]), g)
         ops.add_unit_rms(stream, self.side_proj(g), self.side_norm, float(self.side["eps"]))
         return None
+
+
+@register_part("block", "parallel_pre_norm")
+class ParallelPreNormBlock(Block):
+    """Both sub-layers read the same stream, each behind a norm of its own:
+
+        x <- x + (mixer(norm1(x)) + feed_forward(norm2(x)))
+
+    The norms (``add_norm_pair``: RMS norms with one epsilon) share their statistics, and one kernel closes what the block
+    before left open and writes both norms' outputs.  Everything this block adds is left open in its turn, as a
+    ``PendingSum``.  ``feed_forward`` (and ``norm2``) may be None: the block is then the mixer alone."""
+
+    def __init__(self, name: str, norm1: PartSpec, mixer: PartSpec, norm2: Optional[PartSpec] = None,
+                 feed_forward: Optional[PartSpec] = None, names: Optional[Dict[str, str]] = None):
+        super().__init__(name)
+        n = {"norm1": "norm1", "mixer": "mixer", "norm2": "norm2", "feed_forward": "feed_forward"}
+        n.update(names or {})
+        self.norm1 = create_part("norm", norm1, name=f"{name}.{n['norm1']}")
+        self.mixer = create_part("mixer", mixer, name=f"{name}.{n['mixer']}")
+        self.norm2 = self.feed_forward = None
+        if feed_forward is not None:
+            if norm2 is None:
+                raise ValueError(f"block {name}: a feed-forward needs the norm before it")
+            self.norm2 = create_part("norm", norm2, name=f"{name}.{n['norm2']}")
+            self.feed_forward = create_part("feed_forward", feed_forward, name=f"{name}.{n['feed_forward']}")
+            if not hasattr(self.norm1, "add_norm_pair"):
+                raise ValueError(f"block {name}: {type(self.norm1).__name__} cannot norm for two sub-layers at once")
+
+    def _parts(self):
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.feed_forward) if p is not None]
+
+    @property
+    def graph_capturable(self) -> bool:
+        return all(p.graph_capturable for p in self._parts())
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [s for p in self._parts() for s in p.weight_specs()]
+
+    def setup(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
+        super().setup(rt, weights)
+        for part in self._parts():
+            part.setup(rt, weights)
+
+    def forward(self, stream: torch.Tensor, pending, ctx: StepContext, cache_id: Optional[int],
+                write_cache: bool) -> PendingSum:
+        if self.feed_forward is None:
+            return PendingSum.of(self.mixer.forward(self.norm1.add_norm(stream, pending), ctx, cache_id, write_cache))
+        x, y = self.norm1.add_norm_pair(stream, pending, self.norm2)
+        return PendingSum.of(self.mixer.forward(x, ctx, cache_id, write_cache), self.feed_forward.forward(y))

@@ -8,7 +8,7 @@ one product feeds the gate kernel.
 
 from __future__ import annotations
 
-from typing import Dict, List, Optional
+from typing import Dict, List, Optional, Tuple
 
 import torch
 
@@ -148,7 +148,11 @@ class RoutedExperts(FeedForward):
     ``<name>.<expert><e>.<gate>`` [ff, width].  ``weigh="input"``: the router's weight multiplies what the expert reads
     instead of what it returns, y = sum_chosen expert_e(s_e * router_scale * h).
 
-    The correction takes part in the choice only; the weights are not renormalised.  ``shared``: a feed-forward
+    ``score="softmax"``: s = softmax(W_router h) over all experts.  ``groups`` = (count, keep): the experts form ``count`` equal
+    groups of neighbours, a group's score is the largest in it, and only experts of the ``keep`` best groups can be chosen.
+    ``renormalise``: the chosen experts' s are divided by their sum (+ 1e-20).
+
+    The correction takes part in the choice only.  ``shared``: a feed-forward
     (any registered one) that every token goes through, added to the sum, or None.  Tensors: ``<name>.<router>``
     [E, width], ``<name>.<correction>`` [E] (absent with ``correction=False``), ``<name>.<expert><e>.<up>`` [ff, width]
     and ``.<down>`` [width, ff], and the shared part's under ``<name>.<shared>``."""
@@ -159,8 +163,15 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, name: str, hidden_size: int, experts: int, top: int, expert_ff: int, router_scale: float = 1.0,
                  activation: str = "relu_sq", correction: bool = True, shared: Optional[PartSpec] = None,
-                 names: Optional[Dict[str, str]] = None, gated: bool = False, weigh: str = "output"):
+                 names: Optional[Dict[str, str]] = None, gated: bool = False, weigh: str = "output",
+                 score: str = "sigmoid", groups: Optional[Tuple[int, int]] = None, renormalise: bool = False):
         super().__init__(name)
+        if score not in ops.MOE_SCORES:
+            raise ValueError(f"feed-forward {name}: scores are made by {' or '.join(ops.MOE_SCORES)}, got {score!r}")
+        self.score, self.renormalise = score, bool(renormalise)
+        self.groups, self.keep = (1, 1) if groups is None else (int(groups[0]), int(groups[1]))
+        if not 1 <= self.keep <= self.groups or experts % self.groups or top > self.keep * (experts // self.groups):
+            raise ValueError(f"feed-forward {name}: top {top} of {experts} experts in {self.groups} groups, {self.keep} kept")
         if weigh not in ("output", "input"):
             raise ValueError(f"feed-forward {name}: the router's weight goes to an expert's 'input' or 'output', got {weigh!r}")
         self.gated, self.weigh_input = bool(gated), weigh == "input"
@@ -223,7 +234,8 @@ class RoutedExperts(FeedForward):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         T = x.shape[0]
         ids, wts = self._ids[:T], self._weights[:T]
-        ops.moe_route(x, self.router, self.correction, ids, wts, self.router_scale)
+        ops.moe_route(x, self.router, self.correction, ids, wts, self.router_scale, self.score, self.groups, self.keep,
+                      self.renormalise)
         base = self.shared.forward(x) if self.shared is not None else None
         out = self._out[:T]
         ops.routed_experts(x, self.up, self.down, ids, self._ones[:T] if self.weigh_input else wts, base,

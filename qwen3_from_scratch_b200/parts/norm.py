@@ -1,4 +1,4 @@
-"""RMSNorm: y = x / sqrt(mean(x^2) + eps) * w, and layer norm with weight and bias; statistics in float32.  And Dynamic
+"""RMSNorm: y = x / sqrt(mean(x^2) + eps) * w (or * (1 + w)), and layer norm with weight and bias; statistics in float32.  And Dynamic
 Tanh, which stands where a norm stands but computes no statistics: y = tanh(alpha x) w + b.
 
 Reference: models/norm.py:11-22 (weight multiplies directly, eps from the configuration),
@@ -13,26 +13,28 @@ import torch
 
 from ..kernels import ops
 from ..registry import register_part
-from .base import Norm, PendingNormed, Runtime, StreamNorm, StreamStats, WeightSpec
+from .base import Norm, PendingNormed, PendingSum, Runtime, StreamNorm, StreamStats, WeightSpec
 
 
 @register_part("norm", "rms_norm")
 class RMSNorm(Norm):
     graph_capturable = True
 
-    def __init__(self, name: str, dim: int, eps: float, suffix: str = ".weight"):
+    def __init__(self, name: str, dim: int, eps: float, suffix: str = ".weight", one_plus: bool = False):
         """``suffix``: what follows the part's name in its tensor's name ("" where the tensor bears the
-        part's name itself)."""
+        part's name itself).  ``one_plus``: the weight is stored around zero, y = x / rms(x) * (1 + w)."""
         super().__init__(name)
-        self.dim, self.eps = int(dim), float(eps)
+        self.dim, self.eps, self.one_plus = int(dim), float(eps), bool(one_plus)
         self.tensor = f"{name}{suffix}"
 
     def weight_specs(self) -> List[WeightSpec]:
-        return [WeightSpec(self.tensor, (self.dim,), kind="vector", init="one_plus_normal")]
+        return [WeightSpec(self.tensor, (self.dim,), kind="vector", init="normal" if self.one_plus else "one_plus_normal")]
 
     def setup(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
         super().setup(rt, weights)
         self.weight = weights[self.tensor]
+        if self.one_plus:
+            self.weight = 1.0 + self.weight
         self._out = rt.shared("normed", rt.max_tokens, self.dim)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
@@ -40,10 +42,30 @@ class RMSNorm(Norm):
         ops.rmsnorm(x, self.weight, out, self.eps)
         return out
 
-    def add_norm(self, stream: torch.Tensor, delta: Optional[torch.Tensor]) -> torch.Tensor:
+    def add_norm(self, stream: torch.Tensor, delta) -> torch.Tensor:
+        """``delta``: a tensor, None, or a ``PendingSum``."""
         out = self._out[: stream.shape[0]]
-        ops.add_rmsnorm(stream, delta, self.weight, out, self.eps)
+        if isinstance(delta, PendingSum):
+            ops.sum_norm(stream, self._terms(delta), delta.eps, self.weight, out, self.eps)
+        else:
+            ops.add_rmsnorm(stream, delta, self.weight, out, self.eps)
         return out
+
+    @staticmethod
+    def _terms(pending: Optional[PendingSum]):
+        return [] if pending is None else [(t.delta, t.weight, t.scale) for t in pending.terms]
+
+    def add_norm_pair(self, stream: torch.Tensor, pending, other: "RMSNorm"):
+        """This norm and ``other`` (with the same epsilon) of the same rows, in one pass: (this one's output, the other's)."""
+        if other.eps != self.eps or other.dim != self.dim:
+            raise ValueError(f"norms {self.name} and {other.name} do not share their statistics")
+        if pending is not None and not isinstance(pending, PendingSum):
+            pending = PendingSum.of(pending)
+        out = self._out[: stream.shape[0]]
+        second = self.rt.shared("normed.second", self.rt.max_tokens, self.dim)[: stream.shape[0]]
+        ops.sum_norm(stream, self._terms(pending), 0.0 if pending is None else pending.eps, self.weight, out, self.eps,
+                     second=(other.weight, second))
+        return out, second
 
     def scale_add_norm(self, stream: torch.Tensor, delta: Optional[torch.Tensor], alpha: float,
                        want_copy: bool = True) -> Optional[torch.Tensor]:
@@ -65,7 +87,10 @@ class RMSNorm(Norm):
 
     def norm_rows(self, stream: torch.Tensor, delta: Optional[torch.Tensor], rows: torch.Tensor) -> torch.Tensor:
         out = torch.empty(rows.numel(), self.dim, dtype=self.rt.dtype, device=stream.device)
-        ops.add_rmsnorm_rows(stream, delta, self.weight, rows, out, self.eps)
+        if isinstance(delta, PendingSum):
+            ops.sum_norm(stream, self._terms(delta), delta.eps, self.weight, out, self.eps, rows=rows)
+        else:
+            ops.add_rmsnorm_rows(stream, delta, self.weight, rows, out, self.eps)
         return out
 
 

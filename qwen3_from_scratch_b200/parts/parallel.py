@@ -1,9 +1,11 @@
-"""Several mixers side by side on the same input: y = sum_i scale_i mixer_i(h).
+"""Several mixers side by side on the same input: y = sum_i scale_i mixer_i(h), or, with a norm of its own behind each
+branch, y = sum_i scale_i unit_rms(mixer_i(h)) * w_i.
 
 Every branch is a mixer of the kind that is one product of its input, a core and one product to its output
 (``Mixer.splittable``).  The branches' input matrices are stacked into one, so that h is read by one product, and
 their output matrices are laid side by side, so that one product over the cores' results (each times its scale)
-gives the sum.  What a branch keeps per request is filed under the branch's label: a branch asks the context as if it
+gives the sum.  Branches that are normed one by one have an output product each; their norms and their sum are left
+open (``PendingSum``) for the next norm over the stream, which closes them on its way.  What a branch keeps per request is filed under the branch's label: a branch asks the context as if it
 were alone, and the context it is handed puts the label in front.
 """
 
@@ -14,7 +16,7 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..registry import create_part, register_part
-from .base import Mixer, PartSpec, Runtime, StepContext, WeightSpec
+from .base import Mixer, PendingSum, PendingTerm, Runtime, StepContext, WeightSpec
 from .linear import Linear
 
 
@@ -44,11 +46,13 @@ class ScopedContext:
 @register_part("mixer", "parallel")
 class ParallelMixer(Mixer):
     """``branches``: a list of ``{"label": str, "mixer": PartSpec, "scale": float}``; a branch's tensors are named
-    ``<name>.<label>.*``."""
+    ``<name>.<label>.*``.  ``out_norm``: ``{"suffix": str, "eps": float}``; each branch's output is then brought to unit root
+    mean square over the width and multiplied by the tensor ``<name>.<label>.<suffix>`` before its scale."""
 
-    def __init__(self, name: str, hidden_size: int, branches: Sequence[dict]):
+    def __init__(self, name: str, hidden_size: int, branches: Sequence[dict], out_norm: Optional[dict] = None):
         super().__init__(name)
         self.hidden_size = int(hidden_size)
+        self.out_norm = dict(out_norm) if out_norm else None
         if not branches:
             raise ValueError(f"mixer {name}: needs at least one branch")
         self.labels = [str(b["label"]) for b in branches]
@@ -64,8 +68,15 @@ class ParallelMixer(Mixer):
     def graph_capturable(self) -> bool:
         return all(b.graph_capturable for b in self.branches)
 
+    def _norm_tensor(self, label: str) -> str:
+        return f"{self.name}.{label}.{self.out_norm['suffix']}"
+
     def weight_specs(self) -> List[WeightSpec]:
-        return [s for b in self.branches for s in b.weight_specs()]
+        specs = [s for b in self.branches for s in b.weight_specs()]
+        if self.out_norm:
+            specs += [WeightSpec(self._norm_tensor(label), (self.hidden_size,), kind="vector", init="one_plus_normal")
+                      for label in self.labels]
+        return specs
 
     def cache_spec(self):
         needs = {}
@@ -89,14 +100,29 @@ class ParallelMixer(Mixer):
         for m in outs:
             self.out_columns.append(self.out_columns[-1] + m.shape[1])
         self.in_proj = Linear(torch.cat([m.to(dtype) for m in ins], dim=0), rt, tag="parallel.in")
-        self.out_proj = Linear(torch.cat([m.to(dtype) for m in outs], dim=1), rt, tag="parallel.out")
+        if self.out_norm:
+            self.out_projs = [Linear(m.to(dtype), rt, tag=f"parallel.out.{label}") for label, m in zip(self.labels, outs)]
+            self.norm_weights = [weights[self._norm_tensor(label)] for label in self.labels]
+        else:
+            self.out_proj = Linear(torch.cat([m.to(dtype) for m in outs], dim=1), rt, tag="parallel.out")
         del ins, outs
         for b in self.branches:
             b.setup_core(rt, weights)
-        self._mid = rt.shared("parallel.mid", rt.max_tokens, self.out_columns[-1])
+        if self.out_norm:
+            self._mids = [rt.shared(f"parallel.mid.{label}", rt.max_tokens, b - a)
+                          for label, a, b in zip(self.labels, self.out_columns, self.out_columns[1:])]
+        else:
+            self._mid = rt.shared("parallel.mid", rt.max_tokens, self.out_columns[-1])
 
-    def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool):
         proj = self.in_proj(x)
+        if self.out_norm:
+            terms = []
+            for i, (label, branch) in enumerate(zip(self.labels, self.branches)):
+                mid = self._mids[i][: x.shape[0]]
+                branch.core(proj, self.in_columns[i], ScopedContext(ctx, label), cache_id, write_cache, mid, 1.0)
+                terms.append(PendingTerm(self.out_projs[i](mid), self.norm_weights[i], self.scales[i]))
+            return PendingSum(tuple(terms), float(self.out_norm["eps"]))
         mid = self._mid[: x.shape[0]]
         for i, (label, branch) in enumerate(zip(self.labels, self.branches)):
             branch.core(proj, self.in_columns[i], ScopedContext(ctx, label), cache_id, write_cache,

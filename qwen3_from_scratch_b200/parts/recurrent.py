@@ -13,6 +13,8 @@
 ``mlstm``           the matrix memory of the xLSTM (Beck et al., "xLSTM: Extended Long Short-Term Memory"): per head a
                     memory S [dim, vdim] with exponential input and forget gates kept stable by a running maximum
                     (see the class).
+``decayed_memory``  a matrix memory with a fixed decay per head and no softmax (retention, lightning attention).
+``gated_delta``     a matrix memory with the gated delta rule.
 
 The first two keep two things per request, named in ``cache_spec()``: ``state`` (float32) and ``conv`` (the last
 taps - 1 inputs of the short convolution, float32).  A new request's slot is zero.  The projections are
@@ -23,13 +25,13 @@ The names of the tensors are parameters (``names``), with the defaults below.
 
 from __future__ import annotations
 
-from typing import Dict, List, Optional
+from typing import Dict, List, Optional, Sequence
 
 import torch
 
 from ..kernels import ops
-from ..registry import register_part
-from .base import Mixer, Runtime, StateSpec, StepContext, WeightSpec
+from ..registry import create_part, register_part
+from .base import Mixer, PartSpec, Runtime, StateSpec, StepContext, WeightSpec
 from .linear import Linear
 
 
@@ -424,4 +426,188 @@ class MLSTM(Mixer, _NamedTensors):
     def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
         gated = self._gated[: x.shape[0]]
         self.core(self.in_proj(x), 0, ctx, cache_id, write_cache, gated, 1.0)
+        return self.out_proj(gated)
+
+
+def _stack_rows(parts: Sequence[torch.Tensor], pad_to: int = 8) -> torch.Tensor:
+    """Matrices that read the same input as one, padded with zero rows to whole groups of ``pad_to``."""
+    dtype = torch.float32 if any(p.dtype == torch.float32 for p in parts) else parts[0].dtype
+    rows = sum(p.shape[0] for p in parts)
+    pad = torch.zeros((-rows) % pad_to, parts[0].shape[1], dtype=dtype, device=parts[0].device)
+    return torch.cat([p.to(dtype) for p in parts] + [pad], dim=0)
+
+
+@register_part("mixer", "decayed_memory")
+class DecayedMemory(Mixer, _NamedTensors):
+    """Linear attention with a fixed decay per head: no softmax, no denominator.  With h the input, H heads, keys of ``dim`` and
+    values of ``vdim`` values:
+
+        q = act(W_q h);  k = act(W_k h);  v = act(W_v h)                     (``activation``: "silu" or "none")
+        q, k rotated by ``position`` (a part with ``frequencies()``; None: no rotation)
+        S <- decay_h S + k v^T;   o = S^T q * q_scale
+        out = W_o (unit_rms(o) * norm * gate(W_g h))                         (``gate``: "silu" or "sigmoid")
+
+    ``norm``: "row" (one mean over all heads' values) or "heads" (one per head); ``norm_weight``: whether there is a weight
+    ``<name>.norm`` [H * vdim].  Retention (Sun et al., "Retentive Network: A Successor to Transformer for Large Language
+    Models") and lightning attention (Qin et al., "Lightning Attention-2: A Free Lunch for Handling Unlimited Sequence
+    Lengths in Large Language Models") are such memories.  S starts at zero for a new request and is float32, kept column by
+    column (as S^T); decays, angles, the norm and the gate are float32 in every run.  ``names``: the tensors' names after
+    the part's own."""
+
+    graph_capturable = True
+    splittable = True
+    NAMES = {"q": "q", "k": "k", "v": "v", "gate": "g", "norm": "norm", "out": "o"}
+
+    def __init__(self, name: str, hidden_size: int, num_heads: int, dim: int, vdim: int, decay: Sequence[float], norm_eps: float,
+                 activation: str = "none", position: Optional[PartSpec] = None, q_scale: float = 1.0, norm: str = "heads",
+                 norm_weight: bool = False, gate: str = "silu", names: Optional[Dict[str, str]] = None):
+        super().__init__(name)
+        self.hidden_size, self.num_heads, self.dim, self.vdim = int(hidden_size), int(num_heads), int(dim), int(vdim)
+        self.decay, self.norm_eps, self.q_scale = [float(d) for d in decay], float(norm_eps), float(q_scale)
+        if len(self.decay) != self.num_heads or any(not 0.0 <= d <= 1.0 for d in self.decay):
+            raise ValueError(f"mixer {name}: needs a decay between 0 and 1 for each of its {self.num_heads} heads, got {self.decay}")
+        if activation not in ("silu", "none") or norm not in ("row", "heads") or gate not in ops.MEMORY_GATES:
+            raise ValueError(f"mixer {name}: activation {activation!r}, norm {norm!r} or gate {gate!r} is not built")
+        self.activation, self.norm_parts, self.gate = activation, 1 if norm == "row" else self.num_heads, gate
+        self.has_norm_weight = bool(norm_weight)
+        self.position = None if position is None else create_part("position", position, name=f"{name}.position")
+        if self.position is not None and activation != "none":
+            raise ValueError(f"mixer {name}: a rotation of activated queries and keys is not built")
+        self._name_tensors(name, self.NAMES, names)
+
+    def weight_specs(self) -> List[WeightSpec]:
+        t, w, H, D, Dv = self.tensors, self.hidden_size, self.num_heads, self.dim, self.vdim
+        return [WeightSpec(t["q"], (H * D, w)), WeightSpec(t["k"], (H * D, w)), WeightSpec(t["v"], (H * Dv, w)),
+                WeightSpec(t["gate"], (H * Dv, w)), WeightSpec(t["out"], (w, H * Dv))] + (
+                    [WeightSpec(t["norm"], (H * Dv,), kind="vector", init="one_plus_normal")] if self.has_norm_weight else [])
+
+    def cache_spec(self):
+        return StateSpec((self.num_heads, self.vdim, self.dim), "float32")
+
+    def input_weight(self, weights: Dict[str, torch.Tensor]) -> torch.Tensor:
+        return _stack_rows([weights.pop(self.tensors[k]) for k in ("q", "k", "v", "gate")])  # columns: q, k, v, gates
+
+    def output_weight(self, weights: Dict[str, torch.Tensor]) -> torch.Tensor:
+        return weights.pop(self.tensors["out"])
+
+    @property
+    def output_columns(self) -> int:
+        return self.num_heads * self.vdim
+
+    def setup_core(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
+        self.rt = rt
+        if self.dim > ops.memory_max_dim():
+            raise ValueError(f"mixer {self.name}: keys of {self.dim} values exceed the {ops.memory_max_dim()} the scan takes")
+        self.rule = ops.MemoryDecay(self.decay, rt.device)
+        self.norm_weight = weights[self.tensors["norm"]] if self.has_norm_weight else None
+        if self.position is not None:
+            self.position.setup(rt, weights)
+        self._o = rt.shared("memory.o", rt.max_tokens, self.output_columns, dtype=torch.float32)
+
+    def setup(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
+        super().setup(rt, weights)
+        self.in_proj = Linear(self.input_weight(weights), rt, tag="memory.in")
+        self.out_proj = Linear(self.output_weight(weights), rt, tag="memory.out")
+        self.setup_core(rt, weights)
+        self._gated = rt.shared("memory.gated", rt.max_tokens, self.output_columns)
+
+    def core(self, proj: torch.Tensor, column: int, ctx: StepContext, cache_id: Optional[int], write_cache: bool,
+             out: torch.Tensor, out_scale: float) -> None:
+        if out_scale != 1.0:
+            raise ValueError(f"mixer {self.name}: its output cannot be scaled on the way")
+        H, D, Dv = self.num_heads, self.dim, self.vdim
+        k_col, v_col = column + H * D, column + 2 * H * D
+        if self.position is not None:
+            freq, magnitude, dims = self.position.frequencies()
+            ops.rotate_columns(proj, column, 2 * H, D, dims, freq, magnitude, ctx.positions)  # q and k lie side by side
+        o = self._o[: proj.shape[0]]
+        ops.memory_scan(proj, column, k_col, v_col, self.rule, self.q_scale, self.activation, ctx.state(cache_id), H,
+                        ctx.q_start, ctx.slot_ids, ctx.num_seqs, o, self.rt.status)
+        ops.memory_out(o, proj, v_col + H * Dv, self.norm_weight, self.norm_eps, self.gate, out, self.norm_parts)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
+        gated = self._gated[: x.shape[0]]
+        self.core(self.in_proj(x), 0, ctx, cache_id, write_cache, gated, 1.0)
+        return self.out_proj(gated)
+
+
+@register_part("mixer", "gated_delta")
+class GatedDelta(Mixer, _NamedTensors):
+    """The gated delta rule (Yang et al., "Gated Delta Networks: Improving Mamba2 with Delta Rule").  With h the input, H heads
+    of values on G heads of queries and keys (head n reads query/key head n // (H / G)), keys of ``dim``, values of ``vdim``:
+
+        q, k, v = silu(conv(W_q h)), silu(conv(W_k h)), silu(conv(W_v h))    (a short causal convolution per channel)
+        q <- q / sqrt(|q|^2 + 1e-6) * dim^-1/2;   k <- k / sqrt(|k|^2 + 1e-6)                     (per head)
+        beta = sigmoid(W_b h);   g = exp(-exp(A_log) softplus(W_a h + dt_bias))                   (per head)
+        S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+        out = W_o (unit_rms_per_head(o) * norm * silu(W_g h))                (norm: [vdim], shared by the heads)
+
+    Per request it keeps ``state`` (S column by column, float32) and, with more than one tap, ``conv`` (the last taps - 1 inputs
+    of the convolutions, float32); a new request's slots are zero.  Lengths, decays, beta, the state and the norm are
+    float32 in every run.  ``names``: the tensors' names after the part's own."""
+
+    graph_capturable = True
+    NAMES = {"q": "q", "k": "k", "v": "v", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "b": "b", "a": "a",
+             "a_log": "A_log", "dt_bias": "dt_bias", "gate": "g", "norm": "norm", "out": "o"}
+
+    def __init__(self, name: str, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, conv: int,
+                 norm_eps: float, names: Optional[Dict[str, str]] = None):
+        super().__init__(name)
+        self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
+        self.dim, self.vdim, self.taps, self.norm_eps = int(dim), int(vdim), int(conv), float(norm_eps)
+        if self.num_heads % self.num_kv_heads:
+            raise ValueError(f"mixer {name}: {self.num_heads} heads are not a multiple of {self.num_kv_heads} query/key heads")
+        if self.taps < 1:
+            raise ValueError(f"mixer {name}: the convolutions need at least one tap, got {self.taps}")
+        self.qk = self.num_kv_heads * self.dim
+        self.channels = 2 * self.qk + self.num_heads * self.vdim  # what the convolutions run over: q, k, v
+        self._name_tensors(name, self.NAMES, names)
+
+    def weight_specs(self) -> List[WeightSpec]:
+        t, w, H, Dv, qk, K = self.tensors, self.hidden_size, self.num_heads, self.vdim, self.qk, self.taps
+        specs = []
+        for x, rows in (("q", qk), ("k", qk), ("v", H * Dv)):
+            specs += [WeightSpec(t[x], (rows, w)), WeightSpec(t[f"{x}_conv"], (rows, K), kind="vector", init="normal")]
+        return specs + [WeightSpec(t["b"], (H, w)), WeightSpec(t["a"], (H, w)),
+                        WeightSpec(t["a_log"], (H,), kind="vector", init="normal"),
+                        WeightSpec(t["dt_bias"], (H,), kind="vector", init="normal"),
+                        WeightSpec(t["gate"], (H * Dv, w)),
+                        WeightSpec(t["norm"], (Dv,), kind="vector", init="one_plus_normal"),
+                        WeightSpec(t["out"], (w, H * Dv))]
+
+    def cache_spec(self):
+        needs = {"state": StateSpec((self.num_heads, self.vdim, self.dim), "float32")}
+        if self.taps > 1:
+            needs["conv"] = StateSpec((self.taps - 1, self.channels), "float32")
+        return needs
+
+    def setup(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
+        super().setup(rt, weights)
+        if self.dim > ops.memory_max_dim():
+            raise ValueError(f"mixer {self.name}: keys of {self.dim} values exceed the {ops.memory_max_dim()} the scan takes")
+        t = self.tensors
+        # columns of the product: q, k, v, gates, b, a
+        self.in_proj = Linear(_stack_rows([weights.pop(t[k]) for k in ("q", "k", "v", "gate", "b", "a")]), rt, tag="delta.in")
+        self.conv_weight = torch.cat([weights[t[f"{k}_conv"]] for k in ("q", "k", "v")], dim=0).contiguous()
+        self.a_log, self.dt_bias, self.norm_weight = weights[t["a_log"]], weights[t["dt_bias"]], weights[t["norm"]]
+        self.out_proj = Linear(weights.pop(t["out"]), rt, tag="delta.out")
+        self._no_tail = torch.empty(rt.max_seqs, 0, self.channels, dtype=torch.float32, device=rt.device)
+        self._x = rt.shared("delta.x", rt.max_tokens, self.channels)
+        self._o = rt.shared("memory.o", rt.max_tokens, self.num_heads * self.vdim, dtype=torch.float32)
+        self._gated = rt.shared("delta.gated", rt.max_tokens, self.num_heads * self.vdim)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
+        T, H, Dv = x.shape[0], self.num_heads, self.vdim
+        proj = self.in_proj(x)
+        mixed = self._x[:T]
+        tail = ctx.state(cache_id, "conv") if self.taps > 1 else self._no_tail
+        ops.causal_conv(proj, 0, None, self.conv_weight, None, tail, ctx.q_start, ctx.tok_seq, ctx.slot_ids, ctx.num_seqs,
+                        mixed, "silu", self.rt.status)
+        g_col = self.channels
+        b_col = g_col + H * Dv
+        rule = ops.DeltaGates(proj, b_col, b_col + H, self.a_log, self.dt_bias)
+        o, gated = self._o[:T], self._gated[:T]
+        ops.memory_scan(mixed, 0, self.qk, 2 * self.qk, rule, self.dim ** -0.5, "none", ctx.state(cache_id, "state"),
+                        self.num_kv_heads, ctx.q_start, ctx.slot_ids, ctx.num_seqs, o, self.rt.status)
+        ops.memory_out(o, proj, g_col, self.norm_weight, self.norm_eps, "silu", gated, H)
         return self.out_proj(gated)

@@ -88,7 +88,7 @@ def load_weights(folder: str, specs: Sequence[WeightSpec], *, device, compute_dt
             if name not in where:
                 continue
             e = where[name].entries[name]
-            if tuple(e.shape) != tuple(spec.shape):
+            if not spec.takes(tuple(e.shape)):
                 wrong_shape.append((name, tuple(e.shape), tuple(spec.shape)))
             allowed = _INT if spec.kind == "index" else _FLOAT
             if e.dtype not in allowed:
