@@ -1,5 +1,5 @@
-"""``bench.py --arch binupel|bikadra|dogidra|zasalix``: another design beside Qwen3 (Zasalix: beside Dogidra, the closest
-of the other designs) at equal layer sizes (random weights drawn on
+"""``bench.py --arch binupel|bikadra|dogidra|zasalix|domelix``: another design beside Qwen3 (Zasalix: beside Dogidra,
+Domelix: beside Zasalix, the closest of the other designs) at equal layer sizes (random weights drawn on
 the device): a prompt step of 2,048 tokens and decode steps at two batch sizes, each replayed on the device
 between CUDA events, and every kernel of one eagerly launched step timed by events of its own, with the bytes
 or flops it must move and the fraction of the measured copy bandwidth or bf16 throughput that this makes.
@@ -9,7 +9,9 @@ alternates the state-space mixer and attention through a latent, over four resid
 windowed attention over pooled blocks beside a minGRU in every layer, routed experts with a shared one behind them,
 and a span of two layers twice; a Zasalix model repeats the pattern latent attention with a dense feed-forward, windowed
 attention that keeps the first tokens beside a matrix memory with routed gated experts, a matrix memory alone with
-routed gated experts, the last two as a span that runs twice; the Qwen3 model has as many layer runs of the same width, heads, head size and
+routed gated experts, the last two as a span that runs twice; a Domelix model repeats the pattern full attention with a
+distance bias beside lightning attention, the gated delta rule, retention, each with routed gated experts chosen within
+groups; the Qwen3 model has as many layer runs of the same width, heads, head size and
 (active) feed-forward width.
 """
 
@@ -102,6 +104,25 @@ def zasalix_config(s):
     return {"architecture": "Zasalix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
             "token_side": {"dim": 64}, "loop": {"start": 1, "stop": 3, "times": 2},
             "layers": [pattern[i % 3] for i in range(s["layers"] - 2)]}
+
+
+def domelix_config(s):
+    """Full attention (heads as the other models') beside lightning attention with half as many heads of 128; the gated delta
+    rule with two value heads to a query/key head of 128; retention with as many heads of 128; behind every mixer 16 gated
+    experts of a quarter of the dense width in four groups of which two are kept, four per token."""
+    moe = {"kind": "moe", "expert": {"ff": s["ff"] // 4},
+           "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    decay = lambda heads: [1.0 - 2.0 ** (-5.0 - 4.0 * h / heads) for h in range(heads)]  # noqa: E731
+    H, D = s["heads"], s["dim"]
+    par = {"type": "parallel", "mlp": moe,
+           "mixer": {"left": {"heads": H, "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5, "bias_max": 128},
+                     "right": {"heads": H // 2, "dim": 128, "vdim": 128, "decay": decay(H // 2)}}}
+    delta = {"type": "delta", "mlp": moe, "mixer": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}}
+    ret = {"type": "retention", "mlp": moe, "mixer": {"heads": H, "dim": 128, "vdim": 128, "decay": decay(H),
+                                                      "rot": {"base": 10000.0, "dims": 128}}}
+    pattern = [par, delta, ret]
+    return {"architecture": "Domelix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "layers": [pattern[i % 3] for i in range(s["layers"])]}
 
 
 def qwen3_config(s):
@@ -234,6 +255,22 @@ class KernelClock:
             H, D, Dv = memory.shape[1], memory.shape[2], memory.shape[3]
             seqs = 1 if sc["kind"] == "prefill" else sc["batch"]
             return "bytes", out.shape[0] * H * (2 * D + Dv) * a[0].element_size() + size(out) + 2 * seqs * H * D * Dv * 4
+        if name == "memory_scan":
+            # as mlstm_scan: q, k, v and the result once, and the state in and out
+            x, state, out = a[0], a[7], a[12]
+            H, Dv, D = state.shape[1], state.shape[2], state.shape[3]
+            seqs = 1 if sc["kind"] == "prefill" else sc["batch"]
+            return "bytes", x.shape[0] * (2 * a[8] * D + H * Dv) * x.element_size() + size(out) + 2 * seqs * H * D * Dv * 4
+        if name == "memory_out":
+            o, out = a[0], a[6]
+            return "bytes", size(o) + 2 * out.numel() * out.element_size()
+        if name == "rotate_columns":
+            x, heads, dims = a[0], a[2], a[4]
+            return "bytes", 2 * x.shape[0] * heads * dims * x.element_size()
+        if name == "sum_norm":
+            stream, terms, out = a[0], a[1], a[4]
+            n = size(stream) * (2 if terms and k.get("rows") is None else 1) + sum(size(t[0]) for t in terms)
+            return "bytes", n + size(out) * (2 if k.get("second") is not None else 1)
         if name == "mlstm_out":
             o, out = a[0], a[5]
             return "bytes", size(o) + 2 * out.numel() * out.element_size()
@@ -324,7 +361,7 @@ class KernelClock:
                      "latent_q_post", "gate_heads", "latent_attention", "ssd_scan", "gated_group_norm", "add_layernorm",
                      "add_layernorm_conv1", "input_conv", "stream_concat", "pw_qkv_post", "pool_blocks", "pooled_window_attention",
                      "mingru_scan", "moe_route", "routed_experts", "add_dyt", "add_unit_rms", "side_gate", "sigmoid_gate",
-                     "mlstm_scan", "mlstm_out"):
+                     "mlstm_scan", "mlstm_out", "memory_scan", "memory_out", "rotate_columns", "sum_norm"):
             self.wrap(ops, name, name)
         real_mm = torch.mm
         clock = self
@@ -412,10 +449,11 @@ def compare(args, peaks, sample_clocks):
     sampler = sample_clocks()
     t0 = time.time()
     other = {"binupel": binupel_config, "bikadra": bikadra_config, "dogidra": dogidra_config,
-             "zasalix": zasalix_config}[args.arch]
-    # what the design stands beside: Qwen3, or for Zasalix the closest of the other designs (a windowed attention
-    # beside a recurrence, routed experts, a span of layers that runs twice)
-    beside, beside_config = ("dogidra", dogidra_config) if args.arch == "zasalix" else ("qwen3", qwen3_config)
+             "zasalix": zasalix_config, "domelix": domelix_config}[args.arch]
+    # what the design stands beside: Qwen3, or for Zasalix and Domelix the closest of the other designs (a windowed
+    # attention beside a recurrence, routed experts; an attention beside a matrix memory, matrix memories alone, gated experts)
+    beside, beside_config = {"zasalix": ("dogidra", dogidra_config),
+                             "domelix": ("zasalix", zasalix_config)}.get(args.arch, ("qwen3", qwen3_config))
     out = {"arch": args.arch, "beside": beside, "sizes": dict(size, name=args.arch_size), "dtype": "bf16",
            "data": "synthetic tokens, random weights drawn on the device", "steps": args.steps, "warmup": args.warmup,
            "peaks": peaks, "timing": "CUDA events around each replay of the step; 256 MB written between replays",

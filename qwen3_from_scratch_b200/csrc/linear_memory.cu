@@ -324,28 +324,50 @@ static int memory_scan_sizes(const MemoryIn<T>& in, float* state, const int* q_s
 }
 
 // ---------------------------------------------------------------- the norm and the gate behind a memory
-// grid (T, parts), a block per (token, part).  o: float32 [T, n]; gates at g_col of proj; weight [n] (w_stride = width of
-// a part), [width] shared by the parts (w_stride = 0), or null.
-template <typename T>
+// A unit (a warp, or with WHOLE the block) per (token, part), V values per access.  o: float32 [T, n]; gates at g_col of
+// proj; weight [n] (w_stride = width of a part), [width] shared by the parts (w_stride = 0), or null.
+template <typename T, int V>
+struct alignas(sizeof(T) * V) LmPack { T v[V]; };
+
+template <typename T, int V, bool WHOLE>
 __global__ void memory_out_kernel(const float* __restrict__ o, const T* __restrict__ proj, int ld, int g_col,
                                   const float* __restrict__ w, int w_stride, float eps, int gate, T* __restrict__ out,
-                                  int ldo, int n, int parts) {
+                                  int ldo, int n, int parts, int units) {
   __shared__ float red[32];
   pdl_wait();
   pdl_launch_dependents();
-  const int t = blockIdx.x, part = blockIdx.y, width = n / parts, c0 = part * width;
+  const int unit = WHOLE ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (unit >= units) return;
+  const int first = WHOLE ? threadIdx.x : threadIdx.x & 31, step = WHOLE ? blockDim.x : 32;
+  const int t = unit / parts, part = unit - t * parts, width = n / parts, c0 = part * width;
   const float* row = o + (size_t)t * n + c0;
   const T* gr = proj + (size_t)t * ld + g_col + c0;
+  const float* wr = w ? w + (size_t)part * w_stride : nullptr;
+  T* dst = out + (size_t)t * ldo + c0;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
-  ss = blockDim.x <= 32 ? warp_sum(ss) : block_sum(ss, red);
+#pragma unroll 4
+  for (int i = first * V; i < width; i += step * V) {
+    const LmPack<float, V> x = *reinterpret_cast<const LmPack<float, V>*>(row + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(x.v[e], x.v[e], ss);
+  }
+  ss = WHOLE ? block_sum(ss, red) : warp_sum(ss);
   const float inv = 1.0f / sqrtf(ss / (float)width + eps);
-  for (int i = threadIdx.x; i < width; i += blockDim.x) {
-    const float g = to_float(gr[i]);
-    const float s = gate == Q3_ACT_SILU ? silu_f(g) : sigmoid_f(g);
-    float v = row[i] * inv;
-    if (w) v *= w[(size_t)part * w_stride + i];
-    out[(size_t)t * ldo + c0 + i] = from_float<T>(v * s);
+#pragma unroll 4
+  for (int i = first * V; i < width; i += step * V) {
+    const LmPack<float, V> x = *reinterpret_cast<const LmPack<float, V>*>(row + i);
+    const LmPack<T, V> g = *reinterpret_cast<const LmPack<T, V>*>(gr + i);
+    LmPack<float, V> wv;
+    if (wr) wv = *reinterpret_cast<const LmPack<float, V>*>(wr + i);
+    LmPack<T, V> y;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float gv = to_float(g.v[e]);
+      float v = x.v[e] * inv;
+      if (wr) v *= wv.v[e];
+      y.v[e] = from_float<T>(v * (gate == Q3_ACT_SILU ? silu_f(gv) : sigmoid_f(gv)));
+    }
+    *reinterpret_cast<LmPack<T, V>*>(dst + i) = y;
   }
 }
 
@@ -377,9 +399,9 @@ __global__ void rotate_columns_kernel(T* __restrict__ x, int ld, int col, int he
 
 }  // namespace q3
 
-#define Q3_BY_DTYPE(dtype, CALL)                 \
-  if ((dtype) == Q3_F32) { using E = float; CALL; }  \
-  else if ((dtype) == Q3_BF16) { using E = __nv_bfloat16; CALL; } \
+#define Q3_BY_DTYPE(dtype, ...)                 \
+  if ((dtype) == Q3_F32) { using E = float; __VA_ARGS__; }  \
+  else if ((dtype) == Q3_BF16) { using E = __nv_bfloat16; __VA_ARGS__; } \
   else return Q3_ERR_DTYPE;
 
 // The largest key size the scan takes.
@@ -420,11 +442,27 @@ extern "C" int q3_memory_out(const float* o, const void* proj, int ld, int g_col
                              cudaStream_t stream) {
   if (T <= 0) return 0;
   if (n <= 0 || parts <= 0 || n % parts || parts > 65535 || ldo < n) return Q3_ERR_SIZE;
-  const int width = n / parts;
-  int threads = ((width + 3) / 4 + 31) / 32 * 32;
-  threads = threads < 32 ? 32 : (threads > 256 ? 256 : threads);
-  Q3_BY_DTYPE(dtype, q3::launch(q3::memory_out_kernel<E>, dim3(T, parts), dim3(threads), 0, stream, o, (const E*)proj, ld,
-                                g_col, weight, weight_shared ? 0 : width, eps, gate, (E*)out, ldo, n, parts))
+  const int width = n / parts, shared = weight_shared ? 0 : width;
+  const long long units = (long long)T * parts;
+  if (units > 0x7fffffffll) return Q3_ERR_SIZE;
+  const size_t es = dtype == Q3_F32 ? 4 : 2;
+  const bool by4 = width % 4 == 0 && n % 4 == 0 && ld % 4 == 0 && g_col % 4 == 0 && ldo % 4 == 0 && (uintptr_t)o % 16 == 0 &&
+                   (uintptr_t)proj % (4 * es) == 0 && (uintptr_t)out % (4 * es) == 0 && (uintptr_t)weight % 16 == 0;
+  // a block per row where the row is long or rows are few, else a warp per part
+  const bool whole = width >= 512;
+  const int threads = whole ? (width >= 2048 ? 512 : 256) : 128;
+  const unsigned grid = (unsigned)(whole ? units : (units + 3) / 4);
+#define Q3_MEMORY_OUT(V, WHOLE)                                                                                         \
+  Q3_BY_DTYPE(dtype, {                                                                                                   \
+    auto kernel = q3::memory_out_kernel<E, V, WHOLE>;                                                                    \
+    q3::launch(kernel, dim3(grid), dim3(threads), 0, stream, o, (const E*)proj, ld, g_col, weight, shared, eps, gate, (E*)out, \
+               ldo, n, parts, (int)units);                                                                               \
+  })
+  if (by4 && whole) { Q3_MEMORY_OUT(4, true) }
+  else if (by4) { Q3_MEMORY_OUT(4, false) }
+  else if (whole) { Q3_MEMORY_OUT(1, true) }
+  else { Q3_MEMORY_OUT(1, false) }
+#undef Q3_MEMORY_OUT
   return q3::launch_status();
 }
 

@@ -43,108 +43,179 @@ __device__ __forceinline__ unsigned choice_key(float v) {
   return u & 0x80000000u ? ~u : u | 0x80000000u;
 }
 
-// The entry with the largest key of keys[0 .. n), the lowest index among equals; the whole warp calls it.
-__device__ __forceinline__ int warp_best(const unsigned* keys, int n, int lane) {
-  unsigned best = 0;
-  int at = 0x7fffffff;
-  for (int e = lane; e < n; e += 32)
-    if (keys[e] > best) {
-      best = keys[e];
-      at = e;
+// What a router does with a token's logits, by one warp.  score [E]: the logits (softmax) or the scores (sigmoid); key [E]
+// scratch; kept [groups] scratch.  With up to 32 experts everything stays in the lanes.
+struct Choice {
+  int E, top, softmax, groups, keep, renorm;
+  float scale;
+};
+
+__device__ __forceinline__ void choose_experts(const Choice& c, float* score, unsigned* key, unsigned* kept,
+                                               const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ wts,
+                                               int lane) {
+  const int E = c.E, per = E / c.groups;
+  float mx = -INFINITY, sum = 0.f;
+  if (c.softmax) {  // the sum's order is the lanes' and then the warp's: a token's scores do not depend on the batch
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, score[e]);
+    mx = warp_max(mx);
+    for (int e = lane; e < E; e += 32) sum += expf(score[e] - mx);
+    sum = warp_sum(sum);
+  }
+  // the score of expert e and what it is chosen by: without a bias the logits themselves (the same order, no underflow)
+  auto make = [&](int e, float& s) {
+    const float z = score[e];
+    s = c.softmax ? expf(z - mx) / sum : z;
+    return choice_key(bias ? s + bias[e] : z);
+  };
+  float total = 0.f, my_score = 0.f;
+  int mine = -1;  // lane k keeps the k-th choice (top <= MOE_MAX_TOP = 32)
+  if (E <= 32) {
+    float s = 0.f;
+    unsigned k = lane < E ? make(lane, s) : 0u;
+    if (c.groups > 1) {  // the best group is the one of the best expert outside the groups kept so far
+      const int n = lane / per;
+      unsigned mask = 0;
+      for (int i = 0; i < c.keep; ++i) {
+        const unsigned v = (mask >> n) & 1u ? 0u : k;
+        const unsigned best = __reduce_max_sync(0xffffffffu, v);
+        const int at = __ffs(__ballot_sync(0xffffffffu, v == best && v)) - 1;
+        mask |= 1u << (at / per);
+      }
+      if (!((mask >> n) & 1u)) k = 0;
     }
-  const unsigned top = __reduce_max_sync(0xffffffffu, best);
-  return (int)__reduce_min_sync(0xffffffffu, (unsigned)(best == top ? at : 0x7fffffff));
+    for (int i = 0; i < c.top; ++i) {
+      const unsigned best = __reduce_max_sync(0xffffffffu, k);
+      const int at = __ffs(__ballot_sync(0xffffffffu, k == best && k)) - 1;
+      const float sc = __shfl_sync(0xffffffffu, s, at);
+      total += sc;
+      if (lane == i) {
+        mine = at;
+        my_score = sc;
+      }
+      if (lane == at) k = 0;
+    }
+  } else {
+    for (int e = lane; e < E; e += 32) {
+      float s;
+      key[e] = make(e, s);
+      score[e] = s;
+    }
+    auto best_of = [&](bool groups_left) {  // the largest key, the lowest index among equals
+      unsigned best = 0, at = 0x7fffffff;
+      for (int e = lane; e < E; e += 32)
+        if (key[e] > best && !(groups_left && kept[e / per])) {
+          best = key[e];
+          at = e;
+        }
+      const unsigned top = __reduce_max_sync(0xffffffffu, best);
+      return (int)__reduce_min_sync(0xffffffffu, best == top ? at : 0x7fffffffu);
+    };
+    if (c.groups > 1) {
+      for (int n = lane; n < c.groups; n += 32) kept[n] = 0;
+      __syncwarp();
+      for (int i = 0; i < c.keep; ++i) {
+        const int e = best_of(true);
+        __syncwarp();
+        if (lane == 0) kept[e / per] = 1;
+        __syncwarp();
+      }
+      for (int e = lane; e < E; e += 32)
+        if (!kept[e / per]) key[e] = 0;
+    }
+    __syncwarp();
+    for (int i = 0; i < c.top; ++i) {
+      const int e = best_of(false);
+      const float sc = score[e];
+      total += sc;
+      if (lane == i) {
+        mine = e;
+        my_score = sc;
+      }
+      __syncwarp();
+      if (lane == 0) key[e] = 0;
+      __syncwarp();
+    }
+  }
+  if (lane < c.top) {
+    ids[lane] = mine;
+    wts[lane] = c.renorm ? my_score / (total + 1e-20f) * c.scale : my_score * c.scale;
+  }
 }
 
-template <typename T>
+// TOK tokens to a block: a warp's share of an expert's row is loaded once for all of them, and with TOK > 1 the tokens' rows
+// wait in shared memory (the form for many tokens, W a multiple of 4).  The order of a dot product's additions is the same.
+template <typename T, int TOK>
 __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ bias,
-                                 int* __restrict__ ids, float* __restrict__ wts, int W, int E, int top, float scale,
-                                 int softmax, int groups, int keep, int renorm) {
-  extern __shared__ float score[];  // [E] scores (softmax: logits first), [E] choice keys, [groups] the groups' keys
-  unsigned* key = reinterpret_cast<unsigned*>(score + E);
-  unsigned* group_key = key + E;
+                                 int* __restrict__ ids, float* __restrict__ wts, int Ttot, int W, Choice c) {
+  extern __shared__ __align__(16) float score[];  // [TOK][E] scores, [TOK][E] keys, [TOK][groups] flags, TOK > 1: [TOK][W] rows
+  unsigned* key = reinterpret_cast<unsigned*>(score + TOK * c.E);
+  unsigned* kept = key + TOK * c.E;
+  T* rows = reinterpret_cast<T*>(score + ((TOK * (2 * c.E + c.groups) + 3) & ~3));
   pdl_wait();
   pdl_launch_dependents();
-  const int t = blockIdx.x;
+  const int t0 = blockIdx.x * TOK;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-  const T* row = h + (size_t)t * W;
-  // four values per lane and turn where the rows allow it, so that a warp has its loads in flight together
-  const bool by4 = (W & 3) == 0 && ((uintptr_t)row & (4 * sizeof(T) - 1)) == 0 && ((uintptr_t)wr & 15) == 0;
-  for (int e = warp; e < E; e += nwarps) {
-    const float* w = wr + (size_t)e * W;
-    float dot = 0.f;
-    if (by4) {
-#pragma unroll 8
+  const T* row = h + (size_t)t0 * W;
+  auto leave = [&](int k, int e, float dot) { score[k * c.E + e] = c.softmax ? dot : 1.0f / (1.0f + expf(-dot)); };
+  if constexpr (TOK > 1) {
+    constexpr int PER = 4;
+    const int live = min(TOK, Ttot - t0);
+    struct alignas(sizeof(T) * PER) Pack { T v[PER]; };
+    for (int i = threadIdx.x * PER; i < TOK * W; i += blockDim.x * PER)
+      *reinterpret_cast<Pack*>(rows + i) = *reinterpret_cast<const Pack*>(row + (i < live * W ? i : i % W));
+    __syncthreads();
+    for (int e = warp; e < c.E; e += nwarps) {
+      const float* w = wr + (size_t)e * W;
+      float dot[TOK];
+#pragma unroll
+      for (int k = 0; k < TOK; ++k) dot[k] = 0.f;
+#pragma unroll 4
       for (int i = 4 * lane; i < W; i += 128) {
         const float4 wv = *reinterpret_cast<const float4*>(w + i);
-        float x[4];
-        load4(row + i, x);
-        dot = fmaf(x[0], wv.x, dot);
-        dot = fmaf(x[1], wv.y, dot);
-        dot = fmaf(x[2], wv.z, dot);
-        dot = fmaf(x[3], wv.w, dot);
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) {
+          float x[4];
+          load4(rows + k * W + i, x);
+          dot[k] = fmaf(x[0], wv.x, dot[k]);
+          dot[k] = fmaf(x[1], wv.y, dot[k]);
+          dot[k] = fmaf(x[2], wv.z, dot[k]);
+          dot[k] = fmaf(x[3], wv.w, dot[k]);
+        }
       }
-    } else {
-      for (int i = lane; i < W; i += 32) dot = fmaf(to_float(row[i]), w[i], dot);
+#pragma unroll
+      for (int k = 0; k < TOK; ++k) {
+        dot[k] = warp_sum(dot[k]);
+        if (lane == 0) leave(k, e, dot[k]);
+      }
     }
-    dot = warp_sum(dot);
-    if (lane == 0) {
-      if (softmax) {
-        score[e] = dot;
+  } else {
+    // four values per lane and turn where the rows allow it, so that a warp has its loads in flight together
+    const bool by4 = (W & 3) == 0 && ((uintptr_t)row & (4 * sizeof(T) - 1)) == 0 && ((uintptr_t)wr & 15) == 0;
+    for (int e = warp; e < c.E; e += nwarps) {
+      const float* w = wr + (size_t)e * W;
+      float dot = 0.f;
+      if (by4) {
+#pragma unroll 8
+        for (int i = 4 * lane; i < W; i += 128) {
+          const float4 wv = *reinterpret_cast<const float4*>(w + i);
+          float x[4];
+          load4(row + i, x);
+          dot = fmaf(x[0], wv.x, dot);
+          dot = fmaf(x[1], wv.y, dot);
+          dot = fmaf(x[2], wv.z, dot);
+          dot = fmaf(x[3], wv.w, dot);
+        }
       } else {
-        const float s = 1.0f / (1.0f + expf(-dot));
-        score[e] = s;
-        key[e] = choice_key(s + (bias ? bias[e] : 0.f));
+        for (int i = lane; i < W; i += 32) dot = fmaf(to_float(row[i]), w[i], dot);
       }
+      dot = warp_sum(dot);
+      if (lane == 0) leave(0, e, dot);
     }
   }
   __syncthreads();
-  if (warp > 0) return;
-  if (softmax) {  // the sum's order is the lanes' and then the warp's: a token's scores do not depend on the batch
-    float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, score[e]);
-    mx = warp_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) sum += expf(score[e] - mx);
-    sum = warp_sum(sum);
-    for (int e = lane; e < E; e += 32) {
-      const float z = score[e], s = expf(z - mx) / sum;
-      key[e] = choice_key(bias ? s + bias[e] : z);  // without a bias the logits themselves: the same order, no underflow
-      score[e] = s;
-    }
-    __syncwarp();
-  }
-  if (groups > 1) {
-    const int per = E / groups;
-    for (int n = lane; n < groups; n += 32) {
-      unsigned best = 0;
-      for (int e = n * per; e < (n + 1) * per; ++e) best = max(best, key[e]);
-      group_key[n] = best;
-    }
-    __syncwarp();
-    for (int k = 0; k < keep; ++k) {
-      const int n = warp_best(group_key, groups, lane);
-      if (lane == 0) group_key[n] = 0;  // kept
-      __syncwarp();
-    }
-    for (int e = lane; e < E; e += 32)
-      if (group_key[e / per] != 0) key[e] = 0;  // a group that is not kept
-    __syncwarp();
-  }
-  float total = 0.f;
-  int mine = -1;  // lane k keeps the k-th choice (top <= MOE_MAX_TOP = 32)
-  for (int k = 0; k < top; ++k) {
-    const int e = warp_best(key, E, lane);
-    if (lane == k) mine = e;
-    total += score[e];
-    __syncwarp();
-    if (lane == 0) key[e] = 0;
-    __syncwarp();
-  }
-  if (lane < top) {
-    ids[(size_t)t * top + lane] = mine;
-    wts[(size_t)t * top + lane] = renorm ? score[mine] / (total + 1e-20f) * scale : score[mine] * scale;
-  }
+  for (int k = warp; k < TOK && t0 + k < Ttot; k += nwarps)
+    choose_experts(c, score + k * c.E, key + k * c.E, kept + k * c.groups, bias, ids + (size_t)(t0 + k) * c.top,
+                   wts + (size_t)(t0 + k) * c.top, lane);
 }
 
 // grid (pairs, ceil(F / warps)).  a[pair, f] = act(sum_i up[e, f, i] h[t, i]), t = pair / top.
@@ -213,9 +284,9 @@ __global__ void moe_pair_down_kernel(const T* __restrict__ a, const T* __restric
 
 }  // namespace q3
 
-#define Q3_BY_DTYPE(dtype, CALL)                 \
-  if ((dtype) == Q3_F32) { using E_ = float; CALL; }  \
-  else if ((dtype) == Q3_BF16) { using E_ = __nv_bfloat16; CALL; } \
+#define Q3_BY_DTYPE(dtype, ...)                 \
+  if ((dtype) == Q3_F32) { using E_ = float; __VA_ARGS__; }  \
+  else if ((dtype) == Q3_BF16) { using E_ = __nv_bfloat16; __VA_ARGS__; } \
   else return Q3_ERR_DTYPE;
 
 // h: [T, W] in `dtype`; wr: float32 [E, W]; bias: float32 [E] or null; ids: int32 [T, top]; wts: float32 [T, top].
@@ -226,9 +297,32 @@ extern "C" int q3_moe_route(const void* h, const float* wr, const float* bias, i
   if (T <= 0) return 0;
   if (W <= 0 || E <= 0 || top <= 0 || top > E || top > q3::MOE_MAX_TOP || E > 4096) return Q3_ERR_SIZE;
   if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups)) return Q3_ERR_SIZE;
-  Q3_BY_DTYPE(dtype, q3::launch(q3::moe_route_kernel<E_>, dim3(T), dim3(E >= 16 ? 512 : (E >= 8 ? 256 : 128)), (size_t)(2 * E + groups) * sizeof(float),
-                                stream,
-                                (const E_*)h, wr, bias, ids, wts, W, E, top, scale, softmax, groups, keep, renorm))
+  if ((size_t)(2 * E + groups + 3) * sizeof(float) > 48 * 1024) return Q3_ERR_SIZE;
+  const q3::Choice choice{E, top, softmax, groups, keep, renorm, scale};
+  // many tokens: eight to a block, so that the experts' rows are read an eighth as often
+  constexpr int MANY = 8;
+  const size_t es = dtype == Q3_F32 ? 4 : 2;
+  const size_t smem_many = (size_t)((MANY * (2 * E + groups) + 3) & ~3) * sizeof(float) + (size_t)MANY * W * es;
+  if (T >= 4 * MANY * 32 && W % 4 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)wr % 16 == 0 && smem_many <= 96 * 1024) {
+    const int threads = 32 * (E < 8 ? (E < 4 ? 2 : 4) : 8);
+    Q3_BY_DTYPE(dtype, {
+      auto kernel = q3::moe_route_kernel<E_, MANY>;
+      static bool configured = false;
+      if (!configured) {
+        const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+        if (err != cudaSuccess) return (int)err;
+        configured = true;
+      }
+      q3::launch(kernel, dim3((T + MANY - 1) / MANY), dim3(threads), smem_many, stream, (const E_*)h, wr, bias, ids, wts, T, W,
+                 choice);
+    })
+    return q3::launch_status();
+  }
+  Q3_BY_DTYPE(dtype, {
+    auto kernel = q3::moe_route_kernel<E_, 1>;
+    q3::launch(kernel, dim3(T), dim3(E >= 16 ? 512 : (E >= 8 ? 256 : 128)), (size_t)(2 * E + groups + 3) * sizeof(float), stream,
+               (const E_*)h, wr, bias, ids, wts, T, W, choice);
+  })
   return q3::launch_status();
 }
 

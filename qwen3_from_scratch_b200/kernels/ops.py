@@ -189,6 +189,10 @@ _SIGNATURES = {
     "q3_memory_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p,
                        _c_void_p, _c_void_p, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int,
                        _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+    "q3_memory_scan_mma": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p,
+                           _c_void_p, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
+                           _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                           _c_void_p, _c_void_p],
     "q3_memory_out": [_c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_void_p, _c_int, _c_int,
                       _c_int, _c_int, _c_int, _c_void_p],
     "q3_rotate_columns": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_void_p, _c_int, _c_int,
@@ -244,6 +248,10 @@ def library() -> ctypes.CDLL:
                 lib.q3_mlstm_max_dim.restype = _c_int
                 lib.q3_memory_max_dim.argtypes = []
                 lib.q3_memory_max_dim.restype = _c_int
+                lib.q3_memory_chunk.argtypes = []
+                lib.q3_memory_chunk.restype = _c_int
+                lib.q3_memory_mma_takes.argtypes = [_c_int, _c_int]
+                lib.q3_memory_mma_takes.restype = _c_int
                 lib.q3_moe_tile_rows.argtypes = []
                 lib.q3_moe_tile_rows.restype = _c_int
                 lib.q3_sample_scratch_bytes.argtypes = [_c_int]
@@ -2482,14 +2490,41 @@ class DeltaGates:
         self.proj, self.b_col, self.a_col, self.a_log, self.dt_bias = proj, int(b_col), int(a_col), a_log, dt_bias
 
 
+MEMORY_CHUNKED_FROM = 32  # the longest portion of a step from which the matrix form runs
+
+
+def memory_matrix_form(dtype: torch.dtype, dim: int, vdim: int) -> bool:
+    """Whether the matrix form (chunks of a portion as tensor-core products) takes these heads: bfloat16, keys of 64 or 128
+    values, values in multiples of 32."""
+    return dtype == torch.bfloat16 and bool(library()._lib.q3_memory_mma_takes(int(dim), int(vdim)))
+
+
+class MemoryScratch:
+    """What the matrix form of at most ``max_tokens`` tokens of ``max_seqs`` requests keeps between its kernels: a state per
+    chunk and, for the delta rule, a corrected key and value and two scalars per token and head."""
+
+    def __init__(self, alloc, max_tokens: int, max_seqs: int, heads: int, dim: int, vdim: int, delta: bool):
+        self.chunk = int(library()._lib.q3_memory_chunk())
+        self.max_tokens = int(max_tokens)
+        self.max_records = max_tokens // self.chunk + max_seqs + 1
+        self.records = alloc("memory.records", self.max_records * heads * vdim * dim, dtype=torch.float32)
+        self.keys = self.values = self.scalars = None
+        if delta:
+            self.keys = alloc("memory.keys", 2 * max_tokens * heads * dim, dtype=torch.bfloat16)
+            self.values = alloc("memory.values", max_tokens * heads * vdim, dtype=torch.float32)
+            self.scalars = alloc("memory.scalars", max_tokens * heads * 2, dtype=torch.float32)
+
+
 def memory_scan(x: torch.Tensor, q_col: int, k_col: int, v_col: int, rule, q_scale: float, activation: str,
                 state: torch.Tensor, kv_heads: int, q_start: torch.Tensor, slot_ids: torch.Tensor, num_seqs: int,
-                out: torch.Tensor, status: torch.Tensor) -> None:
+                out: torch.Tensor, status: torch.Tensor, max_q_len: int = 1, scratch: Optional[MemoryScratch] = None) -> None:
     """A matrix memory per head over every request's tokens in order.  ``x`` [T, any]: q and k (kv_heads * dim each) and v
     (heads * vdim) from the given columns, each through ``activation`` ("silu" or "none"); head h reads q and k of head
     h / (heads / kv_heads).  ``rule``: a ``MemoryDecay`` (S <- decay S + k v^T, o = S^T q q_scale) or ``DeltaGates`` (the
     gated delta rule, q and k brought to length one first).  ``state`` float32 [slots, heads, vdim, dim] (column by
-    column) is read and renewed; ``out`` float32 [T, heads * vdim]."""
+    column) is read and renewed; ``out`` float32 [T, heads * vdim].  With ``scratch`` and a portion of ``MEMORY_CHUNKED_FROM``
+    tokens or more the step runs in the matrix form (bfloat16 only: the float32 run keeps the walk, whose sums have one
+    order whatever the cut)."""
     _check("memory_scan.x", x)
     _check("memory_scan.state", state, torch.float32)
     _check("memory_scan.out", out, torch.float32)
@@ -2514,6 +2549,20 @@ def memory_scan(x: torch.Tensor, q_col: int, k_col: int, v_col: int, rule, q_sca
             raise KernelError(f"memory_scan: gates {tuple(rule.proj.shape)} for {H} heads")
         gates = [rule.proj.data_ptr(), rule.proj.shape[1], rule.b_col, rule.a_col, rule.a_log.data_ptr(),
                  rule.dt_bias.data_ptr(), None, None]
+    if scratch is not None and max_q_len >= MEMORY_CHUNKED_FROM and ld % 8 == 0 and (q_col | k_col | v_col) % 8 == 0:
+        _check("memory_scan.x", x, torch.bfloat16)
+        delta = not isinstance(rule, MemoryDecay)
+        if (T > scratch.max_tokens or num_seqs + T // scratch.chunk + 1 > scratch.max_records
+                or scratch.records.numel() < scratch.max_records * H * Dv * D or (delta and scratch.keys is None)):
+            raise KernelError(f"memory_scan: the scratch was made for {scratch.max_tokens} tokens, the step has {T}")
+        code = library().q3_memory_scan_mma(x.data_ptr(), ld, int(q_col), int(k_col), int(v_col), *gates[:6],
+                                            None if delta else rule.log.data_ptr(), float(q_scale),
+                                            activation_code(activation), state.data_ptr(), q_start.data_ptr(),
+                                            slot_ids.data_ptr(), slots, out.data_ptr(), scratch.records.data_ptr(),
+                                            _ptr(scratch.keys), _ptr(scratch.values), _ptr(scratch.scalars), T, int(num_seqs),
+                                            int(max_q_len), H, G, D, Dv, status.data_ptr(), _stream())
+        _done("memory_scan_mma", code, f"heads {H}/{G}, dim {D}, vdim {Dv}")
+        return
     code = library().q3_memory_scan(x.data_ptr(), ld, int(q_col), int(k_col), int(v_col), *gates, float(q_scale),
                                     activation_code(activation), state.data_ptr(), q_start.data_ptr(), slot_ids.data_ptr(),
                                     slots, out.data_ptr(), dtype_tag(x.dtype), int(num_seqs), H, G, D, Dv,

@@ -503,6 +503,9 @@ class DecayedMemory(Mixer, _NamedTensors):
         if self.position is not None:
             self.position.setup(rt, weights)
         self._o = rt.shared("memory.o", rt.max_tokens, self.output_columns, dtype=torch.float32)
+        self._scratch = None
+        if ops.memory_matrix_form(rt.dtype, self.dim, self.vdim) and rt.max_tokens >= ops.MEMORY_CHUNKED_FROM:
+            self._scratch = ops.MemoryScratch(rt.shared, rt.max_tokens, rt.max_seqs, self.num_heads, self.dim, self.vdim, False)
 
     def setup(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
         super().setup(rt, weights)
@@ -522,7 +525,7 @@ class DecayedMemory(Mixer, _NamedTensors):
             ops.rotate_columns(proj, column, 2 * H, D, dims, freq, magnitude, ctx.positions)  # q and k lie side by side
         o = self._o[: proj.shape[0]]
         ops.memory_scan(proj, column, k_col, v_col, self.rule, self.q_scale, self.activation, ctx.state(cache_id), H,
-                        ctx.q_start, ctx.slot_ids, ctx.num_seqs, o, self.rt.status)
+                        ctx.q_start, ctx.slot_ids, ctx.num_seqs, o, self.rt.status, ctx.max_q_len, self._scratch)
         ops.memory_out(o, proj, v_col + H * Dv, self.norm_weight, self.norm_eps, self.gate, out, self.norm_parts)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
@@ -595,6 +598,9 @@ class GatedDelta(Mixer, _NamedTensors):
         self._x = rt.shared("delta.x", rt.max_tokens, self.channels)
         self._o = rt.shared("memory.o", rt.max_tokens, self.num_heads * self.vdim, dtype=torch.float32)
         self._gated = rt.shared("delta.gated", rt.max_tokens, self.num_heads * self.vdim)
+        self._scratch = None
+        if ops.memory_matrix_form(rt.dtype, self.dim, self.vdim) and rt.max_tokens >= ops.MEMORY_CHUNKED_FROM:
+            self._scratch = ops.MemoryScratch(rt.shared, rt.max_tokens, rt.max_seqs, self.num_heads, self.dim, self.vdim, True)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
         T, H, Dv = x.shape[0], self.num_heads, self.vdim
@@ -608,6 +614,7 @@ class GatedDelta(Mixer, _NamedTensors):
         rule = ops.DeltaGates(proj, b_col, b_col + H, self.a_log, self.dt_bias)
         o, gated = self._o[:T], self._gated[:T]
         ops.memory_scan(mixed, 0, self.qk, 2 * self.qk, rule, self.dim ** -0.5, "none", ctx.state(cache_id, "state"),
-                        self.num_kv_heads, ctx.q_start, ctx.slot_ids, ctx.num_seqs, o, self.rt.status)
+                        self.num_kv_heads, ctx.q_start, ctx.slot_ids, ctx.num_seqs, o, self.rt.status, ctx.max_q_len,
+                        self._scratch)
         ops.memory_out(o, proj, g_col, self.norm_weight, self.norm_eps, "silu", gated, H)
         return self.out_proj(gated)
