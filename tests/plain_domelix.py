@@ -109,14 +109,15 @@ def attention(h: torch.Tensor, w, pre: str, m: dict, positions: Sequence[int], s
     longest = max(positions)
     rows = torch.tensor([bucket(n, rel.shape[0], float(m["bias_max"])) for n in range(longest + 1)])
     out = torch.zeros(T, H, Dv, dtype=F64)
-    for t, p in enumerate(positions):
-        far = rows[torch.arange(p, -1, -1)]  # the bias row of every key 0 .. p
-        for n in range(H):
-            g = n // (H // G)
-            s = st["k"][: p + 1, g] @ q[t, n] * float(m["scale"]) + rel[far, n]
-            top = torch.maximum(s.max(), sink[n])
-            e = torch.exp(s - top)
-            out[t, n] = e @ st["v"][: p + 1, g] / (e.sum() + torch.exp(sink[n] - top))
+    n = st["k"].shape[0]
+    back = torch.tensor(positions)[:, None] - torch.arange(n)[None, :]  # how far back a key is; negative: not yet there
+    for head in range(H):
+        g = head // (H // G)
+        s = q[:, head] @ st["k"][:, g].t() * float(m["scale"]) + rel[rows[back.clamp(min=0)], head]
+        s = torch.where(back >= 0, s, torch.tensor(-math.inf, dtype=F64))
+        top = torch.maximum(s.max(dim=1).values, sink[head])[:, None]
+        e = torch.exp(s - top)
+        out[:, head] = e @ st["v"][:, g] / (e.sum(1) + torch.exp(sink[head] - top[:, 0]))[:, None]
     gated = out.reshape(T, H * Dv) * sigmoid(linear(h, w[pre + "g"]))
     return linear(gated, w[pre + "o"])
 
@@ -220,47 +221,82 @@ def experts(h: torch.Tensor, w, pre: str, mlp: dict) -> torch.Tensor:
 
 
 # ---------------------------------------------------------------------- a request's states and the whole model
-def new_state(config: dict, w) -> List[dict]:
+def new_state(config: dict) -> List[dict]:
     states = []
     for entry in config["layers"]:
         m, z = entry["mixer"], lambda *s: torch.zeros(*s, dtype=F64)
         if entry["type"] == "parallel":
             a, b = m["left"], m["right"]
-            states.append({"left": {"k": z(0, a["kv_heads"], a["dim"]), "v": z(0, a["kv_heads"], a["vdim"])},
-                           "right": {"S": z(b["heads"], b["dim"], b["vdim"])}})
+            st = {"left": {"k": z(0, a["kv_heads"], a["dim"]), "v": z(0, a["kv_heads"], a["vdim"])},
+                  "right": {"S": z(b["heads"], b["dim"], b["vdim"])}}
         elif entry["type"] == "delta":
             qk = m["kv_heads"] * m["dim"]
-            states.append({"S": z(m["heads"], m["dim"], m["vdim"]), "q": z(m["conv"] - 1, qk), "k": z(m["conv"] - 1, qk),
-                           "v": z(m["conv"] - 1, m["heads"] * m["vdim"])})
+            st = {"S": z(m["heads"], m["dim"], m["vdim"]), "q": z(m["conv"] - 1, qk), "k": z(m["conv"] - 1, qk),
+                  "v": z(m["conv"] - 1, m["heads"] * m["vdim"])}
         else:
-            states.append({"S": z(m["heads"], m["dim"], m["vdim"])})
+            st = {"S": z(m["heads"], m["dim"], m["vdim"])}
+        st["length"] = 0
+        states.append(st)
     return states
 
 
+def branches(h: torch.Tensor, w, pre: str, m: dict, eps: float, positions: Sequence[int], st: dict) -> torch.Tensor:
+    """Two mixers side by side on the same input: half the sum of their outputs, each normed over the width."""
+    a = attention(h, w, pre + "left.", m["left"], positions, st["left"])
+    b = lightning(h, w, pre + "right.", m["right"], eps, st["right"])
+    return 0.5 * (unit_rms(a, eps) * w[pre + "left.out"] + unit_rms(b, eps) * w[pre + "right.out"])
+
+
 def mixer(h: torch.Tensor, w, pre: str, entry: dict, eps: float, positions: Sequence[int], st: dict) -> torch.Tensor:
-    m = entry["mixer"]
     if entry["type"] == "parallel":
-        a = attention(h, w, pre + "left.", m["left"], positions, st["left"])
-        b = lightning(h, w, pre + "right.", m["right"], eps, st["right"])
-        return 0.5 * (unit_rms(a, eps) * w[pre + "left.out"] + unit_rms(b, eps) * w[pre + "right.out"])
+        return branches(h, w, pre, entry["mixer"], eps, positions, st)
     if entry["type"] == "delta":
-        return delta(h, w, pre, m, eps, st)
-    return retention(h, w, pre, m, eps, positions, st)
+        return delta(h, w, pre, entry["mixer"], eps, st)
+    return retention(h, w, pre, entry["mixer"], eps, positions, st)
 
 
-def run(config: dict, w, tokens: Sequence[int], states: List[dict], start: int = 0,
-        residuals: Optional[list] = None) -> torch.Tensor:
-    """The next ``tokens`` of a request, from and into ``states``; logits [T, vocab].  ``residuals`` collects the stream
-    after every layer."""
+def forward(config: dict, w, tokens: Sequence[int], state: Optional[List[dict]] = None,
+            layers_out: Optional[list] = None) -> torch.Tensor:
+    """Logits [T, vocab] of a request's next ``tokens``; ``state`` (``new_state``) carries what earlier portions left."""
+    if state is None:
+        state = new_state(config)
     eps = float(config["norm"]["eps"])
+    start = state[0]["length"]
     positions = list(range(start, start + len(tokens)))
     x = w["embed"][torch.tensor(list(tokens))].clone()
     for i, entry in enumerate(config["layers"]):
         p = f"l{i}."
-        y = mixer(norm_one_plus(x, w[p + "norm1"], eps), w, p + "mix.", entry, eps, positions, states[i])
+        y = mixer(norm_one_plus(x, w[p + "norm1"], eps), w, p + "mix.", entry, eps, positions, state[i])
         if entry["mlp"] is not None:
             y = y + experts(norm_one_plus(x, w[p + "norm2"], eps), w, p + "mlp.", entry["mlp"])
         x = x + y
-        if residuals is not None:
-            residuals.append(x.clone())
+        state[i]["length"] = start + len(tokens)
+        if layers_out is not None:
+            layers_out.append(x.clone())
     return linear(norm_one_plus(x, w["final.norm"], eps), w["head"])
+
+
+def forward_logits(config: dict, w, ids: Sequence[int]) -> torch.Tensor:
+    return forward(config, w, ids)
+
+
+def rounding_error(config: dict, w, ids: Sequence[int]) -> float:
+    """The largest difference that rounding every projection's operand and result to bfloat16 makes to a logit of this
+    prompt, relative to the largest logit."""
+    exact = forward(config, w, ids)
+    with bfloat16_projections():
+        rounded = forward(config, w, ids)
+    return float((rounded - exact).abs().max()) / float(exact.abs().max())
+
+
+def greedy(config: dict, w, prompt: Sequence[int], new_tokens: int):
+    """(generated ids, gap between the two largest logits at every step), token by token through the states."""
+    state = new_state(config)
+    logits = forward(config, w, prompt, state)
+    out, margins = [], []
+    for _ in range(new_tokens):
+        top = torch.topk(logits[-1], 2).values
+        margins.append(float(top[0] - top[1]))
+        out.append(int(torch.argmax(logits[-1])))
+        logits = forward(config, w, [out[-1]], state)
+    return out, margins
