@@ -324,7 +324,7 @@ static int memory_scan_sizes(const MemoryIn<T>& in, float* state, const int* q_s
 }
 
 // ---------------------------------------------------------------- the norm and the gate behind a memory
-// A unit (a warp, or with WHOLE the block) per (token, part), V values per access.  o: float32 [T, n]; gates at g_col of
+// A unit (a warp, or with WHOLE a block) per (token, part), V values per access.  o: float32 [T, n]; gates at g_col of
 // proj; weight [n] (w_stride = width of a part), [width] shared by the parts (w_stride = 0), or null.
 template <typename T, int V>
 struct alignas(sizeof(T) * V) LmPack { T v[V]; };
@@ -448,7 +448,7 @@ extern "C" int q3_memory_out(const float* o, const void* proj, int ld, int g_col
   const size_t es = dtype == Q3_F32 ? 4 : 2;
   const bool by4 = width % 4 == 0 && n % 4 == 0 && ld % 4 == 0 && g_col % 4 == 0 && ldo % 4 == 0 && (uintptr_t)o % 16 == 0 &&
                    (uintptr_t)proj % (4 * es) == 0 && (uintptr_t)out % (4 * es) == 0 && (uintptr_t)weight % 16 == 0;
-  // a block per row where the row is long or rows are few, else a warp per part
+  // a block per part where parts are long, else a warp per part
   const bool whole = width >= 512;
   const int threads = whole ? (width >= 2048 ? 512 : 256) : 128;
   const unsigned grid = (unsigned)(whole ? units : (units + 3) / 4);
