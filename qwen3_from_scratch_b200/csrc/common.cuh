@@ -87,6 +87,7 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
 #define Q3_ACT_GELU_TANH 2
 #define Q3_ACT_NONE 3
 #define Q3_ACT_RELU_SQ 4  // the square of relu
+#define Q3_ACT_LIMITED 5  // of a gate and its up value together, see gated_f
 
 __device__ __forceinline__ float silu_f(float g) { return g / (1.0f + expf(-g)); }
 __device__ __forceinline__ float sigmoid_f(float g) { return 1.0f / (1.0f + expf(-g)); }
@@ -102,6 +103,18 @@ __device__ __forceinline__ float activate(float g, int act) {
     case Q3_ACT_RELU_SQ: { const float r = fmaxf(g, 0.f); return r * r; }
     default: return g;
   }
+}
+
+constexpr float LIMITED_SLOPE = 1.702f;  // the gate's sigmoid in the limited form
+// A gate and its up value: act(g) * u, or (Q3_ACT_LIMITED) both held back by a limit, the gate from above only,
+// g sigmoid(1.702 g) (u + 1).
+__device__ __forceinline__ float gated_f(float g, float u, int act, float limit) {
+  if (act == Q3_ACT_LIMITED) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-LIMITED_SLOPE * g)) * (u + 1.0f);
+  }
+  return activate(g, act) * u;
 }
 
 static inline int launch_status() { return (int)cudaGetLastError(); }

@@ -70,6 +70,10 @@ struct SkinnyFuse {
   int early;            // EPI 2: the stream may be read ahead of the wait (the launch before did not write it)
   int gate_act;         // EPI 1: the gate's activation, a Q3_ACT_* code (0: SiLU)
   int plain_act;        // EPI 0: 0, or 1 + a Q3_ACT_* code applied to every result (a feed-forward without a gate)
+  const float* bias;    // EPI 1, optional: float32 [N] in the order of W's rows, added before the gate
+  float limit;          // EPI 1: of Q3_ACT_LIMITED
+  int x_rows;           // 0, or: the features in groups of so many (a multiple of 16), group i reads the i-th of several X
+  long long x_stride;   // values from one X to the next
 };
 
 constexpr int GS_SS_ROWS = 16;  // row pitch of the partial sums
@@ -158,6 +162,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ X, const __nv_bfloat16* __r
     const int tok = i * 8 + gid;
     x_ok[i] = tok < T;
     x_row[i] = X + (size_t)(x_ok[i] ? tok : 0) * K + 8 * tid4;
+    if (fuse.x_rows && active) x_row[i] += (row0 / fuse.x_rows) * fuse.x_stride;
   }
   auto multiply = [&](int g0, const uint4 (&lo)[GS_UNROLL], const uint4 (&hi)[GS_UNROLL]) {
     constexpr int XU = GS_UNROLL;  // groups whose activations are fetched together
@@ -270,7 +275,11 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ X, const __nv_bfloat16* __r
         gate *= rs_s[tok];
         up *= rs_s[tok];
       }
-      out[(size_t)tok * ldo + (row0 >> 1) + f] = from_float<OutT>(up * activate(gate, fuse.gate_act));
+      if (fuse.bias) {
+        gate += fuse.bias[row0 + f];
+        up += fuse.bias[row0 + f + 8];
+      }
+      out[(size_t)tok * ldo + (row0 >> 1) + f] = from_float<OutT>(gated_f(gate, up, fuse.gate_act, fuse.limit));
     }
   }
 }
@@ -358,6 +367,38 @@ extern "C" int q3_gemm_skinny(const void* X, const void* W, void* out, int T, in
   }
   if (T <= 8) return q3::gemm_skinny_launch<1, 0, bf16>(X, W, out, T, N, K, ldo, stream);
   return q3::gemm_skinny_launch<2, 0, bf16>(X, W, out, T, N, K, ldo, stream);
+}
+
+// out[T, N / 2] = a gate and its up value (W's rows alternate in blocks of eight, N a multiple of 16), with a bias (float32 [N]
+// in the order of W's rows, or null) in front of it; act: a Q3_ACT_* code of gated_f, with its limit.  T <= 16, bfloat16.
+extern "C" int q3_gemm_skinny_gated(const void* X, const void* W, void* out, int T, int N, int K, int ldo, int act,
+                                    const float* bias, float limit, cudaStream_t stream) {
+  if (T <= 0 || N <= 0) return 0;
+  if (T > 16 || K <= 0 || K % 8 || N % 16 || act < Q3_ACT_SILU || act > Q3_ACT_LIMITED || act == Q3_ACT_NONE)
+    return Q3_ERR_SIZE;
+  if ((uintptr_t)X % 16 || (uintptr_t)W % 16) return Q3_ERR_ALIGN;
+  using bf16 = __nv_bfloat16;
+  q3::SkinnyFuse fuse{};
+  fuse.gate_act = act;
+  fuse.bias = bias;
+  fuse.limit = limit;
+  if (T <= 8) return q3::gemm_skinny_launch<1, 1, bf16>(X, W, out, T, N, K, ldo, stream, fuse);
+  return q3::gemm_skinny_launch<2, 1, bf16>(X, W, out, T, N, K, ldo, stream, fuse);
+}
+
+// Several products with inputs of their own as one: X is [N / group, T, K], the features come in groups of `group` (a multiple
+// of 16) and group i reads X[i].  T <= 16, bfloat16 in and out.
+extern "C" int q3_gemm_skinny_groups(const void* X, const void* W, void* out, int T, int N, int K, int group, int ldo,
+                                     cudaStream_t stream) {
+  if (T <= 0 || N <= 0) return 0;
+  if (T > 16 || K <= 0 || K % 8 || group <= 0 || group % 16 || N % group) return Q3_ERR_SIZE;
+  if ((uintptr_t)X % 16 || (uintptr_t)W % 16) return Q3_ERR_ALIGN;
+  using bf16 = __nv_bfloat16;
+  q3::SkinnyFuse fuse{};
+  fuse.x_rows = group;
+  fuse.x_stride = (long long)T * K;
+  if (T <= 8) return q3::gemm_skinny_launch<1, 0, bf16>(X, W, out, T, N, K, ldo, stream, fuse);
+  return q3::gemm_skinny_launch<2, 0, bf16>(X, W, out, T, N, K, ldo, stream, fuse);
 }
 
 // The forms that take the norm kernels out of a decode step (see the head of the file), T <= 16.

@@ -44,7 +44,7 @@ template <int EPI>
 struct TcThreads {
   // the SwiGLU epilogue too has two warps per quarter of the rows (they take every second piece of 32 columns): with
   // one warp per scheduler a tile's epilogue is a single chain of latencies, which the last tile of a block shows
-  static constexpr int EPI_WARPS = EPI == 2 ? TC_QKV_EPI_WARPS : ((EPI == 1 || EPI == 3) ? 8 : 4);
+  static constexpr int EPI_WARPS = EPI == 2 ? TC_QKV_EPI_WARPS : (EPI != 0 ? 8 : 4);
   static constexpr int THREADS = 64 + 32 * EPI_WARPS;
 };
 
@@ -75,6 +75,10 @@ struct QkvEpilogue {
   int table_stride, page_size, num_pages, Hq, Hkv;
   float eps;
   int write_kv;
+  // EPI 4
+  const float* gate_bias;  // float32 [N] in the order of W's rows, or null
+  int gate_act;            // Q3_ACT_SILU, Q3_ACT_GELU_TANH or Q3_ACT_LIMITED
+  float gate_limit;
 };
 
 // One head of the warp's 32 rows, in two passes.
@@ -301,10 +305,11 @@ __device__ __forceinline__ void qkv_tile_epilogue(uint32_t tmem_acc, unsigned ch
 }
 
 // Stores 32 consecutive columns of one row.  EPI 0: as they are.  EPI 1: SwiGLU on column blocks
-// (gate 8, up 8, ...), 16 outputs at half the column index.  EPI 3: the same with a ReLU gate.
+// (gate 8, up 8, ...), 16 outputs at half the column index.  EPI 3: the same with a ReLU gate.  EPI 4: with the gate
+// that `e` names, behind a bias.
 template <int EPI, typename OutT>
 __device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], OutT* __restrict__ C, int row, int col0, int N,
-                                               int ldc) {
+                                               int ldc, const QkvEpilogue& e) {
   if (EPI == 0) {
     OutT* dst = C + (size_t)row * ldc + col0;
     if (col0 + 32 <= N && ((uintptr_t)dst & 15) == 0) {
@@ -337,7 +342,23 @@ __device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], OutT* __
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        const float gate = __uint_as_float(v[16 * j + i]), up = __uint_as_float(v[16 * j + 8 + i]);
+        float gate = __uint_as_float(v[16 * j + i]), up = __uint_as_float(v[16 * j + 8 + i]);
+        if (EPI == 4) {
+          if (e.gate_bias && col0 + 16 * j + 8 + i < N) {  // the whole warp reads the same entries
+            gate += e.gate_bias[col0 + 16 * j + i];
+            up += e.gate_bias[col0 + 16 * j + 8 + i];
+          }
+          float slope = 1.f;  // gate * sigmoid(slope * gate)
+          if (e.gate_act == Q3_ACT_LIMITED) {
+            gate = fminf(gate, e.gate_limit);
+            up = fminf(fmaxf(up, -e.gate_limit), e.gate_limit) + 1.0f;
+            slope = LIMITED_SLOPE;
+          } else if (e.gate_act == Q3_ACT_GELU_TANH) {  // (1 + tanh(y)) / 2 = sigmoid(2 y)
+            slope = 1.5957691216057308f * fmaf(0.044715f * gate, gate, 1.0f);
+          }
+          r[8 * j + i] = up * __fdividef(gate, 1.0f + __expf(-slope * gate));
+          continue;
+        }
         // silu by the fast exponential and division: their error (about 2^-21) is far below the
         // bfloat16 rounding of the result, and the exact forms made this epilogue longer than the main loop
         r[8 * j + i] = EPI == 3 ? up * fmaxf(gate, 0.f) : up * __fdividef(gate, 1.0f + __expf(-gate));
@@ -363,7 +384,7 @@ __device__ __forceinline__ void tc_store_chunk(const uint32_t (&v)[32], OutT* __
 }
 
 // EPI 0: store.  EPI 1: SwiGLU.  EPI 2: the QKV epilogue with heads of HD values (C is not written).  EPI 3: gated
-// like EPI 1, the gate a ReLU.
+// like EPI 1, the gate a ReLU.  EPI 4: gated, the gate and an optional bias in front of it from `qkv`.
 template <int BN, int EPI, typename OutT, int HD = 128>
 __global__ void __launch_bounds__(TcThreads<EPI>::THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
@@ -523,7 +544,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           uint32_t v[32];
           tmem_ld_32(tmem_acc + (uint32_t)c0, v);
           tmem_wait_ld();
-          if (row < M) tc_store_chunk<EPI == 2 ? 0 : EPI, OutT>(v, C, row, n0 + c0, N, ldc);
+          if (row < M) tc_store_chunk<EPI == 2 ? 0 : EPI, OutT>(v, C, row, n0 + c0, N, ldc, qkv);
         }
         tcgen05_fence_before();
         __syncwarp();
@@ -735,7 +756,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           uint32_t v[32];
           tmem_ld_32(tmem_acc + (uint32_t)c0, v);
           tmem_wait_ld();
-          if (row < M) tc_store_chunk<EPI == 2 ? 0 : EPI, OutT>(v, C, row, n0 + c0, N, ldc);
+          if (row < M) tc_store_chunk<EPI == 2 ? 0 : EPI, OutT>(v, C, row, n0 + c0, N, ldc, qkv);
         }
         tcgen05_fence_before();
         __syncwarp();
@@ -833,9 +854,9 @@ static int tc_pick_bn(int M, int N) {
 
 template <int EPI, typename OutT>
 static int gemm_tc_dispatch(const void* A, const void* W, void* C, int M, int N, int K, int ldc, int* status,
-                            cudaStream_t stream) {
-  if (tc_pick_bn(M, N) == 256) return gemm_tc_launch<256, EPI, OutT>(A, W, C, M, N, K, ldc, status, stream);
-  return gemm_tc_launch<128, EPI, OutT>(A, W, C, M, N, K, ldc, status, stream);
+                            cudaStream_t stream, const QkvEpilogue& e = QkvEpilogue{}) {
+  if (tc_pick_bn(M, N) == 256) return gemm_tc_launch<256, EPI, OutT>(A, W, C, M, N, K, ldc, status, stream, e);
+  return gemm_tc_launch<128, EPI, OutT>(A, W, C, M, N, K, ldc, status, stream, e);
 }
 
 }  // namespace q3
@@ -868,6 +889,23 @@ extern "C" int q3_gemm_tc_pair(const void* A, const void* W, void* C, int M, int
   if (swiglu) return q3::gemm_tc_pair_launch<1, bf16>(A, W, C, M, N, K, ldc, status, stream);
   if (out_f32) return q3::gemm_tc_pair_launch<0, float>(A, W, C, M, N, K, ldc, status, stream);
   return q3::gemm_tc_pair_launch<0, bf16>(A, W, C, M, N, K, ldc, status, stream);
+}
+
+// The gated product with a bias (float32 [N] in the order of W's rows, or null) in front of the gate: W's rows alternate
+// gate/up in blocks of eight, N a multiple of 16, C is [M, N / 2] bfloat16.  act: Q3_ACT_SILU, Q3_ACT_GELU_TANH or
+// Q3_ACT_LIMITED with its limit.  pair: by pairs of CTAs.
+extern "C" int q3_gemm_tc_gated(const void* A, const void* W, void* C, int M, int N, int K, int ldc, int act, const float* bias,
+                                float limit, int pair, int* status, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K <= 0 || K % 8 || N % 16 || (act != Q3_ACT_SILU && act != Q3_ACT_GELU_TANH && act != Q3_ACT_LIMITED)) return Q3_ERR_SIZE;
+  if ((uintptr_t)A % 16 || (uintptr_t)W % 16) return Q3_ERR_ALIGN;
+  q3::QkvEpilogue e{};
+  e.gate_bias = bias;
+  e.gate_act = act;
+  e.gate_limit = limit;
+  using bf16 = __nv_bfloat16;
+  if (pair) return q3::gemm_tc_pair_launch<4, bf16>(A, W, C, M, N, K, ldc, status, stream, e);
+  return q3::gemm_tc_dispatch<4, bf16>(A, W, C, M, N, K, ldc, status, stream, e);
 }
 
 // For the tests of the give-up path: see set_wait_test in tc_common.cuh.

@@ -4,6 +4,8 @@
 //   decayed   S <- decay_h S + k v^T;  o = S^T q                  (a fixed decay per head: retention, lightning attention)
 //   delta     g = exp(-exp(A_log_h) softplus(a + dt_bias_h)),  beta = sigmoid(b),  q and k brought to length one
 //             S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q                    (the gated delta rule)
+//   channel   o = (S + diag(u) k v^T)^T q;  S <- diag(w) S + k v^T     (a decay w per token and key channel, given by its
+//             logarithm; the token itself is read with a bonus u per head and channel, before it enters: RWKV's time mixing)
 //
 //   memory_scan    walks the tokens of every request in order.  A block owns one head of one request and a slice of the
 //                  Dv columns; L lanes share a column, each with 4 J of its rows in registers.  A chunk of tokens' q, k,
@@ -13,6 +15,8 @@
 //                  r = S_old^T q,  u = beta (v - g p),  o = g r + (k . q) u,  S = g S_old + k u^T.
 //                  The state is read at the start and written at the end, so a prompt in portions walks exactly as the
 //                  whole prompt does.  It is kept column by column, [slots, H, Dv, D].
+//   low_rank_decay the logarithms of the channel form's decays: -exp(W_2 tanh(low) + w_0) for the rows `low` that a first,
+//                  narrow projection left, all in float32.
 //   memory_out     o divided by the root mean square of its part of the row (one part, or one per head), times an
 //                  optional weight, times sigmoid or silu of a gate: the operand of the output projection.
 //   rotate_columns rotation of the first `dims` values of every head (value i with i + dims / 2), in place.
@@ -24,6 +28,7 @@
 namespace q3 {
 
 constexpr int LM_THREADS = 128, LM_WARPS = 4;
+enum MemoryRule { LM_DECAYED = 0, LM_DELTA = 1, LM_CHANNEL = 2 };
 
 // Where the operands of a step lie: x [T, ld] with q (G heads of D), k, v (H heads of Dv) at columns of it; for the
 // delta rule the pre-activations b and a (H each) at columns of `gates` [T, ldg].
@@ -35,6 +40,7 @@ struct MemoryIn {
   int ldg, b_col, a_col;
   const float *A_log, *dt_bias;     // delta [H]
   const float *decay, *decay_m1;    // decayed [H]: the decay and the decay minus one
+  const float *logw, *bonus;        // channel: the decays' logarithms [T, H * D], u [H, D]
   float q_scale;
   int act;                          // Q3_ACT_SILU or Q3_ACT_NONE, on q, k and v
   int vec;                          // rows and slices are made of aligned 16-byte pieces
@@ -50,7 +56,7 @@ __device__ __forceinline__ void lm_copy(T* dst, const T* src, int n, int vec, in
   }
 }
 
-template <typename T, int L, int J, int CPT, bool DELTA>
+template <typename T, int L, int J, int CPT, int RULE>
 __global__ void __launch_bounds__(LM_THREADS)
 memory_scan_kernel(MemoryIn<T> in, float* __restrict__ state, const int* __restrict__ q_start,
                    const int* __restrict__ slot_ids, int num_slots, float* __restrict__ out, int H, int G, int D, int Dv,
@@ -58,14 +64,15 @@ memory_scan_kernel(MemoryIn<T> in, float* __restrict__ state, const int* __restr
   constexpr int DP = 4 * L * J;                     // a row of q or k in shared memory, zeros beyond D
   constexpr int CHUNK = DP <= 128 ? 16 : 2048 / DP; // tokens of a chunk
   constexpr int COLS = (LM_THREADS / L) * CPT;      // columns of a block
-  constexpr bool EXACT = sizeof(T) == 4;
+  constexpr bool EXACT = sizeof(T) == 4, DELTA = RULE == LM_DELTA, CHANNEL = RULE == LM_CHANNEL;
   extern __shared__ __align__(16) unsigned char lm_smem[];
   float* q_s = reinterpret_cast<float*>(lm_smem);   // [CHUNK][DP]
   float* k_s = q_s + CHUNK * DP;
   float* v_s = k_s + CHUNK * DP;                    // [CHUNK][COLS]
   float* o_s = v_s + CHUNK * COLS;                  // [CHUNK][COLS]
-  float* g_s = o_s + CHUNK * COLS;                  // [CHUNK][4]: g, g - 1, beta, k . q
-  T* raw = reinterpret_cast<T*>(g_s + 4 * CHUNK);   // [2][q: CHUNK][DP] [k] [v: CHUNK][COLS]
+  float* g_s = o_s + CHUNK * COLS;                  // [CHUNK][4]: g, g - 1, beta, k . q; channel: q . (u k)
+  float* w_s = g_s + 4 * CHUNK;                     // channel: [CHUNK][DP] decays minus one, then [2][CHUNK][DP] logarithms
+  T* raw = reinterpret_cast<T*>(w_s + (CHANNEL ? 3 * CHUNK * DP : 0));  // [2][q: CHUNK][DP] [k] [v: CHUNK][COLS]
   constexpr int RAW = CHUNK * (2 * DP + COLS);
 
   const int b = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * COLS;
@@ -109,7 +116,7 @@ memory_scan_kernel(MemoryIn<T> in, float* __restrict__ state, const int* __restr
   if (DELTA) {
     rate = -expf(in.A_log[h]);
     bias = in.dt_bias[h];
-  } else {
+  } else if (!CHANNEL) {
     dec = in.decay[h];
     dec1 = in.decay_m1[h];
   }
@@ -126,6 +133,8 @@ memory_scan_kernel(MemoryIn<T> in, float* __restrict__ state, const int* __restr
       lm_copy(r + c * DP, row + in.q_col + hk * D, D, in.vec, lane, 32);
       lm_copy(r + (CHUNK + c) * DP, row + in.k_col + hk * D, D, in.vec, lane, 32);
       lm_copy(r + 2 * CHUNK * DP + c * COLS, row + in.v_col + h * Dv + col0, vn, in.vec, lane, 32);
+      if constexpr (CHANNEL)
+        lm_copy(w_s + (1 + buf) * CHUNK * DP + c * DP, in.logw + ((size_t)(c0 + c) * H + h) * D, D, in.vec, lane, 32);
     }
     cp_async_commit();
   };
@@ -164,6 +173,7 @@ memory_scan_kernel(MemoryIn<T> in, float* __restrict__ state, const int* __restr
           g_s[4 * c + 3] = kq * fq * fk;
         }
       }
+      [[maybe_unused]] float own = 0.f;
       for (int d = lane; d < DP; d += 32) {
         float qv = 0.f, kv = 0.f;
         if (d < D) {
@@ -176,6 +186,14 @@ memory_scan_kernel(MemoryIn<T> in, float* __restrict__ state, const int* __restr
         }
         q_s[c * DP + d] = qv * fq;
         k_s[c * DP + d] = kv * fk;
+        if constexpr (CHANNEL) {
+          w_s[c * DP + d] = d < D ? expm1f(w_s[(1 + buf) * CHUNK * DP + c * DP + d]) : 0.f;
+          if (d < D) own = fmaf(qv * fq, in.bonus[(size_t)h * D + d] * kv, own);
+        }
+      }
+      if constexpr (CHANNEL) {
+        own = warp_sum(own);
+        if (lane == 0) g_s[4 * c] = own;
       }
       for (int d = lane; d < COLS; d += 32) {
         float v = d < vn ? to_float(rv[d]) : 0.f;
@@ -231,6 +249,32 @@ memory_scan_kernel(MemoryIn<T> in, float* __restrict__ state, const int* __restr
             for (int e = 0; e < 4; ++e)
               S[i][j][e] = EXACT ? S[i][j][e] + fmaf(gs.y, S[i][j][e], kk[j][e] * u) : fmaf(gs.x, S[i][j][e], kk[j][e] * u);
         }
+      } else if constexpr (CHANNEL) {
+        float w1[J][4];
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+          const float4 wv = *reinterpret_cast<const float4*>(w_s + c * DP + 4 * (l + L * j));
+          w1[j][0] = wv.x, w1[j][1] = wv.y, w1[j][2] = wv.z, w1[j][3] = wv.w;
+        }
+        const float own = g_s[4 * c];
+#pragma unroll
+        for (int i = 0; i < CPT; ++i) {
+          float ra[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+          for (int j = 0; j < J; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              ra[e] = fmaf(S[i][j][e], qq[j][e], ra[e]);
+              S[i][j][e] += fmaf(w1[j][e], S[i][j][e], kk[j][e] * vv[i]);
+            }
+          o[i] = (ra[0] + ra[1]) + (ra[2] + ra[3]);
+        }
+#pragma unroll
+        for (int w = L >> 1; w > 0; w >>= 1)
+#pragma unroll
+          for (int i = 0; i < CPT; ++i) o[i] += __shfl_xor_sync(0xffffffffu, o[i], w);
+#pragma unroll
+        for (int i = 0; i < CPT; ++i) o[i] = fmaf(own, vv[i], o[i]);
       } else {
 #pragma unroll
         for (int i = 0; i < CPT; ++i) {
@@ -280,15 +324,15 @@ memory_scan_kernel(MemoryIn<T> in, float* __restrict__ state, const int* __restr
   }
 }
 
-template <typename T, int L, int J, int CPT, bool DELTA>
+template <typename T, int L, int J, int CPT, int RULE>
 static int memory_scan_launch(const MemoryIn<T>& in, float* state, const int* q_start, const int* slot_ids, int num_slots,
                               float* out, int B, int H, int G, int D, int Dv, int* status, cudaStream_t stream) {
   constexpr int DP = 4 * L * J, CHUNK = DP <= 128 ? 16 : 2048 / DP, COLS = (LM_THREADS / L) * CPT;
-  constexpr size_t smem = sizeof(float) * (size_t)(CHUNK * (2 * DP + 2 * COLS) + 4 * CHUNK) +
+  constexpr size_t smem = sizeof(float) * (size_t)(CHUNK * (2 * DP + 2 * COLS) + 4 * CHUNK + (RULE == LM_CHANNEL ? 3 * CHUNK * DP : 0)) +
                           2 * sizeof(T) * (size_t)CHUNK * (2 * DP + COLS);
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(memory_scan_kernel<T, L, J, CPT, DELTA>,
+    cudaError_t e = cudaFuncSetAttribute(memory_scan_kernel<T, L, J, CPT, RULE>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
@@ -297,22 +341,22 @@ static int memory_scan_launch(const MemoryIn<T>& in, float* state, const int* q_
   // 16-byte pieces: rows, columns, heads and slices all start on one
   constexpr int PER = 16 / sizeof(T);
   args.vec = (uintptr_t)in.x % 16 == 0 && in.ld % PER == 0 && in.q_col % PER == 0 && in.k_col % PER == 0 &&
-             in.v_col % PER == 0 && D % PER == 0 && Dv % PER == 0 && COLS % PER == 0;
-  launch(memory_scan_kernel<T, L, J, CPT, DELTA>, dim3((Dv + COLS - 1) / COLS, H, B), dim3(LM_THREADS), smem, stream, args,
+             in.v_col % PER == 0 && D % PER == 0 && Dv % PER == 0 && COLS % PER == 0 && (uintptr_t)in.logw % 16 == 0;
+  launch(memory_scan_kernel<T, L, J, CPT, RULE>, dim3((Dv + COLS - 1) / COLS, H, B), dim3(LM_THREADS), smem, stream, args,
          state, q_start, slot_ids, num_slots, out, H, G, D, Dv, status);
   return launch_status();
 }
 
-template <typename T, bool DELTA>
+template <typename T, int RULE>
 static int memory_scan_sizes(const MemoryIn<T>& in, float* state, const int* q_start, const int* slot_ids, int num_slots,
                              float* out, int B, int H, int G, int D, int Dv, int* status, cudaStream_t stream) {
 #define Q3_LM(L, J)                                                                                                     \
   {                                                                                                                     \
     const long long wide = (long long)B * H * ((Dv + 2 * (LM_THREADS / L) - 1) / (2 * (LM_THREADS / L)));               \
     if (wide >= 4LL * sm_count())                                                                                       \
-      return memory_scan_launch<T, L, J, 2, DELTA>(in, state, q_start, slot_ids, num_slots, out, B, H, G, D, Dv, status, \
+      return memory_scan_launch<T, L, J, 2, RULE>(in, state, q_start, slot_ids, num_slots, out, B, H, G, D, Dv, status, \
                                                    stream);                                                             \
-    return memory_scan_launch<T, L, J, 1, DELTA>(in, state, q_start, slot_ids, num_slots, out, B, H, G, D, Dv, status,  \
+    return memory_scan_launch<T, L, J, 1, RULE>(in, state, q_start, slot_ids, num_slots, out, B, H, G, D, Dv, status,  \
                                                  stream);                                                               \
   }
   if (D <= 32) Q3_LM(4, 2)
@@ -321,6 +365,58 @@ static int memory_scan_sizes(const MemoryIn<T>& in, float* state, const int* q_s
   if (D <= 256) Q3_LM(16, 4)
   Q3_LM(32, 4)
 #undef Q3_LM
+}
+
+// ---------------------------------------------------------------- decays from a low-rank projection
+// logw[t, c] = -exp(sum_r w2[c, r] tanh(low[t, r]) + w0[c]), at least LR_LEAST (whose exponential is zero in float32).
+// low: [T, ld]; w2: [C, R]; w0: [C]; logw: [T, C].  A block takes LR_T tokens and LR_C channels; a sum runs over r in order.
+constexpr int LR_T = 32, LR_C = 64, LR_R = 32, LR_THREADS = 256;
+constexpr float LR_LEAST = -104.f;
+
+__global__ void __launch_bounds__(LR_THREADS)
+low_rank_decay_kernel(const float* __restrict__ low, int ld, const float* __restrict__ w2, const float* __restrict__ w0,
+                      float* __restrict__ logw, int Ttot, int C, int R) {
+  __shared__ float a_s[LR_R][LR_T + 1], w_s[LR_R][LR_C + 1];
+  const int t0 = blockIdx.y * LR_T, c0 = blockIdx.x * LR_C;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;  // four channels tx + 16 j, two tokens ty + 16 i
+  auto weights = [&](int r0) {
+    for (int i = threadIdx.x; i < LR_C * LR_R; i += LR_THREADS) {
+      const int c = i / LR_R, r = i % LR_R;
+      w_s[r][c] = c0 + c < C && r0 + r < R ? w2[(size_t)(c0 + c) * R + r0 + r] : 0.f;
+    }
+  };
+  weights(0);  // they do not depend on the kernel before this one
+  pdl_wait();
+  pdl_launch_dependents();
+  float acc[2][4] = {};
+  for (int r0 = 0; r0 < R; r0 += LR_R) {
+    if (r0 > 0) {
+      __syncthreads();
+      weights(r0);
+    }
+    for (int i = threadIdx.x; i < LR_T * LR_R; i += LR_THREADS) {
+      const int t = i / LR_R, r = i % LR_R;
+      a_s[r][t] = t0 + t < Ttot && r0 + r < R ? tanhf(low[(size_t)(t0 + t) * ld + r0 + r]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int r = 0; r < LR_R; ++r) {
+      const float a0 = a_s[r][ty], a1 = a_s[r][ty + 16];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float w = w_s[r][tx + 16 * j];
+        acc[0][j] = fmaf(a0, w, acc[0][j]);
+        acc[1][j] = fmaf(a1, w, acc[1][j]);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = t0 + ty + 16 * i, c = c0 + tx + 16 * j;
+      if (t < Ttot && c < C) logw[(size_t)t * C + c] = fmaxf(-expf(acc[i][j] + w0[c]), LR_LEAST);
+    }
 }
 
 // ---------------------------------------------------------------- the norm and the gate behind a memory
@@ -425,15 +521,39 @@ extern "C" int q3_memory_scan(const void* x, int ld, int q_col, int k_col, int v
 #define Q3_LM_DTYPE(E)                                                                                                     \
   {                                                                                                                        \
     const q3::MemoryIn<E> in{(const E*)x, ld, q_col, k_col, v_col, (const E*)gates, ldg, b_col, a_col, A_log, dt_bias,     \
-                             decay, decay_m1, q_scale, act, 0};                                                            \
+                             decay, decay_m1, nullptr, nullptr, q_scale, act, 0};                                                            \
     if (decay)                                                                                                             \
-      return q3::memory_scan_sizes<E, false>(in, state, q_start, slot_ids, num_slots, out, B, H, G, D, Dv, status, stream); \
-    return q3::memory_scan_sizes<E, true>(in, state, q_start, slot_ids, num_slots, out, B, H, G, D, Dv, status, stream);   \
+      return q3::memory_scan_sizes<E, q3::LM_DECAYED>(in, state, q_start, slot_ids, num_slots, out, B, H, G, D, Dv, status, stream); \
+    return q3::memory_scan_sizes<E, q3::LM_DELTA>(in, state, q_start, slot_ids, num_slots, out, B, H, G, D, Dv, status, stream);   \
   }
   if (dtype == Q3_F32) Q3_LM_DTYPE(float)
   if (dtype == Q3_BF16) Q3_LM_DTYPE(__nv_bfloat16)
 #undef Q3_LM_DTYPE
   return Q3_ERR_DTYPE;
+}
+
+// The channel form (see the head of the file): x as above with one query/key head per value head; logw: float32 [T, H * D],
+// the logarithms of the decays; bonus: float32 [H, D].
+extern "C" int q3_channel_memory_scan(const void* x, int ld, int q_col, int k_col, int v_col, const float* logw,
+                                      const float* bonus, float* state, const int* q_start, const int* slot_ids, int num_slots,
+                                      float* out, int dtype, int B, int H, int D, int Dv, int* status, cudaStream_t stream) {
+  if (B <= 0) return 0;
+  if (H <= 0 || H > 65535 || B > 65535 || D <= 0 || D > 512 || Dv <= 0 || num_slots <= 0 || !logw || !bonus) return Q3_ERR_SIZE;
+  Q3_BY_DTYPE(dtype, {
+    const q3::MemoryIn<E> in{(const E*)x, ld, q_col, k_col, v_col, nullptr, 0, 0, 0, nullptr, nullptr, nullptr, nullptr, logw,
+                             bonus, 1.0f, Q3_ACT_NONE, 0};
+    return q3::memory_scan_sizes<E, q3::LM_CHANNEL>(in, state, q_start, slot_ids, num_slots, out, B, H, H, D, Dv, status, stream);
+  })
+}
+
+// low: float32 rows of ld values (the first R are read); w2: float32 [C, R]; w0: float32 [C]; logw: float32 [T, C].
+extern "C" int q3_low_rank_decay(const float* low, int ld, const float* w2, const float* w0, float* logw, int T, int C, int R,
+                                 cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (C <= 0 || R <= 0 || R > ld || T > 32 * 65535) return Q3_ERR_SIZE;
+  q3::launch(q3::low_rank_decay_kernel, dim3((C + q3::LR_C - 1) / q3::LR_C, (T + q3::LR_T - 1) / q3::LR_T), dim3(q3::LR_THREADS), 0,
+             stream, low, ld, w2, w0, logw, T, C, R);
+  return q3::launch_status();
 }
 
 // weight: float32 [n], [n / parts] with weight_shared, or null.  gate: Q3_ACT_SILU, or Q3_ACT_NONE for a sigmoid.

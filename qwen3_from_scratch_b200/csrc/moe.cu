@@ -5,7 +5,9 @@
 //                  with the largest s + bias[e] are chosen (ties: the lower index).  With `groups` > 1 the experts form
 //                  equal groups of neighbours and only experts of the `keep` groups with the largest best member can be
 //                  chosen.  Their weights are s * scale (the bias takes no part in the weights), divided by the sum
-//                  of the chosen s (+ 1e-20) with `renorm`.  One block per token.
+//                  of the chosen s (+ 1e-20) with `renorm`.  A bias of the logits themselves (`zbias`) is added before
+//                  anything else.  With `share` the router's matrix has one more row w_s, and share[t] =
+//                  sigmoid(w_s h): what a shared expert's output is multiplied by.  One block per token.
 //   moe_pair_up    for every (token, chosen expert) pair: act(W_up[e] h), a warp per output value; the pair's expert
 //                  weight is streamed once per pair.  For a few tokens (decoding) and the float32 run.
 //   moe_pair_down  out[t] = base[t] + sum_k weight[t, k] W_down[e_k] a[t, k]: a warp per output value, the chosen
@@ -13,11 +15,11 @@
 //
 // Gated experts (`gate_block` > 0): W_down (act(W_gate h) * (W_up h)); the stack `up` then holds 2 F rows per
 // expert, gate and up rows alternating in blocks of `gate_block` rows (gate_block = F: all gate rows, then all up
-// rows).  `in_wts` (or null): the router's weight multiplies what the expert reads (both of its first products)
+// rows); the limited form of a gate (gated_f) takes `limit`.  `in_wts` (or null): the router's weight multiplies what the expert reads (both of its first products)
 // instead of what it returns; the caller then passes ones as `wts` to the second kernel.
 //
 // Sums over a row are taken lane by lane in ascending order and then across the warp, so a token's result does not
-// depend on the batch.  The expert weights are stacked: up [E, F, W], down [E, W, F].
+// depend on the batch.  `base_wts` (or null): base[t] counts times base_wts[t].  The expert weights are stacked: up [E, F, W], down [E, W, F].
 #include "common.cuh"
 
 namespace q3 {
@@ -146,7 +148,8 @@ __device__ __forceinline__ void choose_experts(const Choice& c, float* score, un
 // wait in shared memory (the form for many tokens, W a multiple of 4).  The order of a dot product's additions is the same.
 template <typename T, int TOK>
 __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ bias,
-                                 int* __restrict__ ids, float* __restrict__ wts, int Ttot, int W, Choice c) {
+                                 const float* __restrict__ zbias, int* __restrict__ ids, float* __restrict__ wts,
+                                 float* __restrict__ share, int Ttot, int W, Choice c) {
   extern __shared__ __align__(16) float score[];  // [TOK][E] scores, [TOK][E] keys, [TOK][groups] flags, TOK > 1: [TOK][W] rows
   unsigned* key = reinterpret_cast<unsigned*>(score + TOK * c.E);
   unsigned* kept = key + TOK * c.E;
@@ -156,7 +159,15 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
   const int t0 = blockIdx.x * TOK;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   const T* row = h + (size_t)t0 * W;
-  auto leave = [&](int k, int e, float dot) { score[k * c.E + e] = c.softmax ? dot : 1.0f / (1.0f + expf(-dot)); };
+  const int rows_of_router = c.E + (share ? 1 : 0);
+  auto leave = [&](int k, int e, float dot) {
+    if (e == c.E) {  // the shared expert's row
+      if (t0 + k < Ttot) share[t0 + k] = sigmoid_f(dot);
+      return;
+    }
+    if (zbias) dot += zbias[e];
+    score[k * c.E + e] = c.softmax ? dot : 1.0f / (1.0f + expf(-dot));
+  };
   if constexpr (TOK > 1) {
     constexpr int PER = 4;
     const int live = min(TOK, Ttot - t0);
@@ -164,7 +175,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
     for (int i = threadIdx.x * PER; i < TOK * W; i += blockDim.x * PER)
       *reinterpret_cast<Pack*>(rows + i) = *reinterpret_cast<const Pack*>(row + (i < live * W ? i : i % W));
     __syncthreads();
-    for (int e = warp; e < c.E; e += nwarps) {
+    for (int e = warp; e < rows_of_router; e += nwarps) {
       const float* w = wr + (size_t)e * W;
       float dot[TOK];
 #pragma unroll
@@ -191,7 +202,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
   } else {
     // four values per lane and turn where the rows allow it, so that a warp has its loads in flight together
     const bool by4 = (W & 3) == 0 && ((uintptr_t)row & (4 * sizeof(T) - 1)) == 0 && ((uintptr_t)wr & 15) == 0;
-    for (int e = warp; e < c.E; e += nwarps) {
+    for (int e = warp; e < rows_of_router; e += nwarps) {
       const float* w = wr + (size_t)e * W;
       float dot = 0.f;
       if (by4) {
@@ -222,7 +233,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
 template <typename T>
 __global__ void moe_pair_up_kernel(const T* __restrict__ h, const T* __restrict__ up, const int* __restrict__ ids,
                                    T* __restrict__ a, int W, int F, int E, int top, int act, int gate_block,
-                                   const float* __restrict__ in_wts) {
+                                   const float* __restrict__ in_wts, float limit) {
   pdl_wait();
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31;
@@ -248,7 +259,7 @@ __global__ void moe_pair_up_kernel(const T* __restrict__ h, const T* __restrict_
     }
     dg = warp_sum(dg) * in_scale;
     du = warp_sum(du) * in_scale;
-    if (lane == 0) a[(size_t)pair * F + f] = from_float<T>(activate(dg, act) * du);
+    if (lane == 0) a[(size_t)pair * F + f] = from_float<T>(gated_f(dg, du, act, limit));
     return;
   }
   const T* w = up + ((size_t)e * F + f) * W;
@@ -261,8 +272,8 @@ __global__ void moe_pair_up_kernel(const T* __restrict__ h, const T* __restrict_
 // grid (T, ceil(W / warps)).  out[t, c] = base[t, c] + sum_k wts[t, k] sum_f down[e_k, c, f] a[t * top + k, f].
 template <typename T>
 __global__ void moe_pair_down_kernel(const T* __restrict__ a, const T* __restrict__ down, const int* __restrict__ ids,
-                                     const float* __restrict__ wts, const T* __restrict__ base, T* __restrict__ out, int W,
-                                     int F, int E, int top) {
+                                     const float* __restrict__ wts, const T* __restrict__ base,
+                                     const float* __restrict__ base_wts, T* __restrict__ out, int W, int F, int E, int top) {
   pdl_wait();
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31;
@@ -270,6 +281,7 @@ __global__ void moe_pair_down_kernel(const T* __restrict__ a, const T* __restric
   const int t = blockIdx.x;
   if (c >= W) return;
   float acc = base ? to_float(base[(size_t)t * W + c]) : 0.f;
+  if (base_wts) acc *= base_wts[t];
   for (int k = 0; k < top; ++k) {
     const int e = ids[(size_t)t * top + k];
     if (e < 0 || e >= E) continue;
@@ -291,9 +303,11 @@ __global__ void moe_pair_down_kernel(const T* __restrict__ a, const T* __restric
 
 // h: [T, W] in `dtype`; wr: float32 [E, W]; bias: float32 [E] or null; ids: int32 [T, top]; wts: float32 [T, top].
 // softmax: scores by softmax instead of a sigmoid; groups, keep: see the head of the file (1, 1: no groups); renorm: the
-// weights divided by the chosen scores' sum.
-extern "C" int q3_moe_route(const void* h, const float* wr, const float* bias, int* ids, float* wts, int dtype, int T, int W,
-                            int E, int top, float scale, int softmax, int groups, int keep, int renorm, cudaStream_t stream) {
+// weights divided by the chosen scores' sum.  zbias: float32 [E] or null, added to the logits.  share: float32 [T] or null; with
+// it wr is [E + 1, W] and share[t] receives the sigmoid of the last row's product.
+extern "C" int q3_moe_route(const void* h, const float* wr, const float* bias, const float* zbias, int* ids, float* wts,
+                            float* share, int dtype, int T, int W, int E, int top, float scale, int softmax, int groups,
+                            int keep, int renorm, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (W <= 0 || E <= 0 || top <= 0 || top > E || top > q3::MOE_MAX_TOP || E > 4096) return Q3_ERR_SIZE;
   if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups)) return Q3_ERR_SIZE;
@@ -313,34 +327,37 @@ extern "C" int q3_moe_route(const void* h, const float* wr, const float* bias, i
         if (err != cudaSuccess) return (int)err;
         configured = true;
       }
-      q3::launch(kernel, dim3((T + MANY - 1) / MANY), dim3(threads), smem_many, stream, (const E_*)h, wr, bias, ids, wts, T, W,
-                 choice);
+      q3::launch(kernel, dim3((T + MANY - 1) / MANY), dim3(threads), smem_many, stream, (const E_*)h, wr, bias, zbias, ids, wts, share, T,
+                 W, choice);
     })
     return q3::launch_status();
   }
   Q3_BY_DTYPE(dtype, {
     auto kernel = q3::moe_route_kernel<E_, 1>;
     q3::launch(kernel, dim3(T), dim3(E >= 16 ? 512 : (E >= 8 ? 256 : 128)), (size_t)(2 * E + groups + 3) * sizeof(float), stream,
-               (const E_*)h, wr, bias, ids, wts, T, W, choice);
+               (const E_*)h, wr, bias, zbias, ids, wts, share, T, W, choice);
   })
   return q3::launch_status();
 }
 
 // a: [T * top, F] = act(up[ids] h); out: [T, W] = base + sum_k wts down[ids] a.  act: a Q3_ACT_* code.
-// gate_block > 0: gated experts (see the head of the file); in_wts: float32 [T * top] or null.
+// gate_block > 0: gated experts (see the head of the file; only they take Q3_ACT_LIMITED, with its limit); in_wts: float32
+// [T * top] or null; base_wts: float32 [T] or null.
 extern "C" int q3_moe_pairs(const void* h, const void* up, const void* down, const int* ids, const float* wts,
                             const void* base, void* a, void* out, int dtype, int T, int W, int F, int E, int top, int act,
-                            int gate_block, const float* in_wts, cudaStream_t stream) {
+                            int gate_block, const float* in_wts, const float* base_wts, float limit, cudaStream_t stream) {
   if (gate_block < 0 || (gate_block > 0 && F % gate_block)) return Q3_ERR_SIZE;
   if (T <= 0) return 0;
-  if (W <= 0 || F <= 0 || E <= 0 || top <= 0 || (long long)T * top > 0x7fffffffll || F > 4 * 65535 || W > 4 * 65535 || act < 0 || act > Q3_ACT_RELU_SQ)
+  if (W <= 0 || F <= 0 || E <= 0 || top <= 0 || (long long)T * top > 0x7fffffffll || F > 4 * 65535 || W > 4 * 65535 || act < 0 || act > Q3_ACT_LIMITED ||
+      (act == Q3_ACT_LIMITED && gate_block == 0))
     return Q3_ERR_SIZE;
   const int warps = 4;
   Q3_BY_DTYPE(dtype, q3::launch(q3::moe_pair_up_kernel<E_>, dim3(T * top, (F + warps - 1) / warps), dim3(warps * 32), 0,
-                                stream, (const E_*)h, (const E_*)up, ids, (E_*)a, W, F, E, top, act, gate_block, in_wts))
+                                stream, (const E_*)h, (const E_*)up, ids, (E_*)a, W, F, E, top, act, gate_block, in_wts, limit))
   int code = q3::launch_status();
   if (code) return code;
   Q3_BY_DTYPE(dtype, q3::launch(q3::moe_pair_down_kernel<E_>, dim3(T, (W + warps - 1) / warps), dim3(warps * 32), 0, stream,
-                                (const E_*)a, (const E_*)down, ids, wts, (const E_*)base, (E_*)out, W, F, E, top))
+                                (const E_*)a, (const E_*)down, ids, wts, (const E_*)base, base_wts, (E_*)out, W, F, E,
+                                top))
   return q3::launch_status();
 }

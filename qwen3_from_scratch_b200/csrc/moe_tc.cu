@@ -15,7 +15,7 @@
 //                   the routing and a captured graph replays them.  The epilogue applies the activation; for gated
 //                   experts (gate and up rows alternating in blocks of 16 rows of a stack of 2 F) it multiplies the
 //                   activated gate columns of a 32-column piece by the piece's up columns and stores 16 values.
-//   moe_combine     out[t] = base[t] + sum_k weight[t, k] y[pos[t, k]], float32 sums in the router's order.
+//   moe_combine     out[t] = base[t] (times base_wts[t], where that is given) + sum_k weight[t, k] y[pos[t, k]], float32 sums in the router's order.
 //
 // Every wait on an mbarrier is bounded as in gemm_tc.cu: a wait that runs out sets the TIMEOUT bit of the status word,
 // every role leaves its loop, tensor memory is released and the block returns.
@@ -112,10 +112,11 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ h, const int
 // grid (tokens).  y: the sorted rows of the second product.
 __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ pos,
                                    const float* __restrict__ wts, const __nv_bfloat16* __restrict__ base,
-                                   __nv_bfloat16* __restrict__ out, int W, int top) {
+                                   const float* __restrict__ base_wts, __nv_bfloat16* __restrict__ out, int W, int top) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
+  const float share = base_wts ? base_wts[t] : 1.0f;
   for (int i = threadIdx.x; i < W / 8; i += blockDim.x) {
     float acc[8];
     if (base) {
@@ -124,8 +125,8 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const in
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 f = __bfloat1622float2(b2[j]);
-        acc[2 * j] = f.x;
-        acc[2 * j + 1] = f.y;
+        acc[2 * j] = f.x * share;
+        acc[2 * j + 1] = f.y * share;
       }
     } else {
 #pragma unroll
@@ -156,13 +157,13 @@ constexpr int MOE_GATED = 0x100;  // OR-ed into the activation code: the columns
 
 // 32 columns of one row: activation, rounding to bfloat16, store.
 __device__ __forceinline__ void moe_store_chunk(const uint32_t (&v)[32], __nv_bfloat16* C, int row, int col0, int N, int ldc,
-                                                int act) {
+                                                int act, float limit) {
   if (act & MOE_GATED) {  // columns col0 .. +15: gates, +16 .. +31: their up values; N = 2 ldc-columns, whole pieces
     if (col0 + 32 > N) return;
     __nv_bfloat16* dst = C + (size_t)row * ldc + (col0 >> 1);
     float g[16];
 #pragma unroll
-    for (int j = 0; j < 16; ++j) g[j] = activate(__uint_as_float(v[j]), act & 0xff) * __uint_as_float(v[16 + j]);
+    for (int j = 0; j < 16; ++j) g[j] = gated_f(__uint_as_float(v[j]), __uint_as_float(v[16 + j]), act & 0xff, limit);
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       uint4 pk;
@@ -200,7 +201,7 @@ template <int BN>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                    __nv_bfloat16* __restrict__ C, const int* __restrict__ meta, int max_tiles, int N, int K, int E, int ldc,
-                   int act, int* status) {
+                   int act, float limit, int* status) {
   using S = MoeShape<BN>;
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* tiles = smem_raw;
@@ -336,7 +337,7 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
         uint32_t v[32];
         tmem_ld_32(tmem_acc + (uint32_t)c0, v);
         tmem_wait_ld();
-        moe_store_chunk(v, C, row, n0 + c0, N, ldc, act);
+        moe_store_chunk(v, C, row, n0 + c0, N, ldc, act, limit);
       }
       tcgen05_fence_before();
       __syncwarp();
@@ -353,7 +354,7 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
 
 template <int BN>
 static int moe_grouped_launch(const void* A, const void* W, void* C, const int* meta, int map_tiles, int max_tiles, int N,
-                              int K, int E, int ldc, int act, int* status, cudaStream_t stream) {
+                              int K, int E, int ldc, int act, float limit, int* status, cudaStream_t stream) {
   using S = MoeShape<BN>;
   static bool configured = false;
   if (!configured) {
@@ -371,7 +372,7 @@ static int moe_grouped_launch(const void* A, const void* W, void* C, const int* 
   if (tiles > 0x7fffffffLL) return Q3_ERR_SIZE;
   const int grid = (int)(tiles < sm_count() ? tiles : sm_count());
   q3::launch(moe_grouped_kernel<BN>, dim3(grid), dim3(MOE_THREADS), S::SMEM_BYTES, stream, map_a, map_b, (__nv_bfloat16*)C,
-             meta, max_tiles, N, K, E, ldc, act, status);
+             meta, max_tiles, N, K, E, ldc, act, limit, status);
   return launch_status();
 }
 
@@ -382,19 +383,19 @@ extern "C" int q3_moe_tile_rows() { return q3::MOE_BM; }
 
 // The routed experts of T tokens (bfloat16) by sorted rows and two grouped products.  h: [T, W]; up: [E, F, W];
 // (gated: [E, 2 F, W], gate and up rows alternating in blocks of 16, F a multiple of 16); in_wts: [T, top] or null, the
-// weights of what the experts read (`wts` are those of what they return);
-// down: [E, W, F]; ids, wts: [T, top]; base: [T, W] or null; out: [T, W].  Scratch for max_tiles >= T * top / 128 + E
+// weights of what the experts read (`wts` are those of what they return); limit: of Q3_ACT_LIMITED (gated experts only);
+// down: [E, W, F]; ids, wts: [T, top]; base: [T, W] or null, with base_wts [T] or null; out: [T, W].  Scratch for max_tiles >= T * top / 128 + E
 // tiles: sorted_in [max_tiles * 128, W], sorted_act [.., F], sorted_out [.., W], pos int32 [T * top], src int32
 // [max_tiles * 128], meta int32 [1 + max_tiles].  W and F multiples of 8, all bases 16-byte aligned.
 extern "C" int q3_moe_grouped(const void* h, const void* up, const void* down, const int* ids, const float* wts,
                               const void* base, void* out, void* sorted_in, void* sorted_act, void* sorted_out, int* pos,
                               int* src, int* meta, int T, int W, int F, int E, int top, int max_tiles, int act, int gated,
-                              const float* in_wts, int* status, cudaStream_t stream) {
+                              const float* in_wts, const float* base_wts, float limit, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (gated && F % 16) return Q3_ERR_SIZE;
   if (W <= 0 || F <= 0 || E <= 0 || E > 4096 || top <= 0 || W % 8 || F % 8 || (long long)T * top > 0x3fffffffll ||
       max_tiles < (int)(((long long)T * top) / q3::MOE_BM) + E || (long long)E * (W > 2 * F ? W : 2 * F) > 0x7fffffffll ||
-      act < 0 || act > Q3_ACT_RELU_SQ)
+      act < 0 || act > Q3_ACT_LIMITED || (act == Q3_ACT_LIMITED && !gated))
     return Q3_ERR_SIZE;
   if ((uintptr_t)h % 16 || (uintptr_t)up % 16 || (uintptr_t)down % 16 || (uintptr_t)out % 16 || (uintptr_t)sorted_in % 16 ||
       (uintptr_t)sorted_act % 16 || (uintptr_t)sorted_out % 16 || (base && (uintptr_t)base % 16))
@@ -417,8 +418,8 @@ extern "C" int q3_moe_grouped(const void* h, const void* up, const void* down, c
     return ((t256 + sms - 1) / sms) * 256 <= ((t128 + sms - 1) / sms) * 128;
   };
   auto product = [&](const void* a, const void* wgt, void* c, int n, int k, int ldc, int activation) {
-    return wide(n) ? q3::moe_grouped_launch<256>(a, wgt, c, meta, map_tiles, max_tiles, n, k, E, ldc, activation, status, stream)
-                   : q3::moe_grouped_launch<128>(a, wgt, c, meta, map_tiles, max_tiles, n, k, E, ldc, activation, status, stream);
+    return wide(n) ? q3::moe_grouped_launch<256>(a, wgt, c, meta, map_tiles, max_tiles, n, k, E, ldc, activation, limit, status, stream)
+                   : q3::moe_grouped_launch<128>(a, wgt, c, meta, map_tiles, max_tiles, n, k, E, ldc, activation, limit, status, stream);
   };
   code = gated ? product(sorted_in, up, sorted_act, 2 * F, W, F, act | q3::MOE_GATED)
                : product(sorted_in, up, sorted_act, F, W, F, act);
@@ -426,6 +427,6 @@ extern "C" int q3_moe_grouped(const void* h, const void* up, const void* down, c
   code = product(sorted_act, down, sorted_out, W, F, W, Q3_ACT_NONE);
   if (code) return code;
   q3::launch(q3::moe_combine_kernel, dim3(T), dim3(128), 0, stream, (const bf16*)sorted_out, (const int*)pos, wts,
-             (const bf16*)base, (bf16*)out, W, top);
+             (const bf16*)base, base_wts, (bf16*)out, W, top);
   return q3::launch_status();
 }

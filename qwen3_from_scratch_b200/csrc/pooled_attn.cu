@@ -11,6 +11,9 @@
 //   pw_qkv_post      RMS norm of the whole q projection and of the whole k projection (one mean over all heads'
 //                    values, a weight per value), rotation of the first `dims` values of every head (pair i with
 //                    i + dims / 2, sines and cosines times `mag`), q to a buffer, k and v into the token pages
+//   head_qkv_post    the same between a projection and the attention for designs with a bias on the projections and a
+//                    norm per head: bias, RMS norm of every head of q and of k (one weight of D values per kind, shared
+//                    by the heads), rotation, q to a buffer, k and v into the token pages
 //   pool_blocks      the blocks that this step completed: their means into the block pages
 //   pw_attn_ref      a warp per (token, head), blocks first and then tokens, one by one in ascending order, float32
 //                    arithmetic: the float32 run's kernel, the fallback for every shape and the other kernels' oracle
@@ -92,6 +95,99 @@ __global__ void pw_qkv_post_kernel(const T* __restrict__ proj, int ld, int k_col
   for (int i = threadIdx.x; i < G * Dv; i += blockDim.x) {
     const int g = i / Dv, d = i - g * Dv;
     v_pages[(((size_t)page * G + g) * page_size + in_page) * Dv + d] = row[v_col + i];
+  }
+}
+
+// A warp per head vector of the token, V values per access.  proj: [T, ld] with q (H * D) at column 0 and, with has_kv, k
+// (G * D) at k_col and v (G * Dv) at v_col; bias: float32, by the same columns, or null; wq, wk: float32 [D] or null.
+template <typename T, int V>
+struct alignas(sizeof(T) * V) PwPack { T v[V]; };
+
+constexpr int HQ_WARPS = 8;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(HQ_WARPS * 32)
+head_qkv_post_kernel(const T* __restrict__ proj, int ld, int k_col, int v_col, int has_kv, int H, int G, int D, int Dv,
+                     const float* __restrict__ bias, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
+                     int dims, const float* __restrict__ freq, float mag, const int* __restrict__ positions,
+                     const int* __restrict__ tok_seq, const int* __restrict__ table, int stride, int page_size, int num_pages,
+                     T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, int* status) {
+  extern __shared__ float hq_smem[];  // [dims / 2] cosines, [dims / 2] sines, times mag; then per warp a head's values
+  constexpr int PER = PW_PER / V;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int pos = positions[t], b = tok_seq[t], half = dims >> 1;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, c;
+    sincosf((float)pos * freq[i], &sn, &c);
+    hq_smem[i] = c * mag;
+    hq_smem[half + i] = sn * mag;
+  }
+  float* head = hq_smem + ((dims + 3) & ~3) + warp * ((D + 3) & ~3);
+  int page = 0, in_page = 0;
+  bool write = has_kv != 0;
+  if (write) {
+    page = (pos < 0 || b < 0) ? -1 : table_page(table + (size_t)b * stride, pos / page_size, stride, status);
+    if (page < 0 || page >= num_pages) {
+      if (threadIdx.x == 0) atomicOr(status, (pos < 0 || b < 0) ? Q3_STATUS_BAD_POSITION : Q3_STATUS_BAD_PAGE);
+      write = false;
+    }
+    in_page = write ? pos % page_size : 0;
+  }
+  __syncthreads();
+  const int units = H + (has_kv ? 2 * G : 0);
+  for (int u = warp; u < units; u += HQ_WARPS) {
+    const bool is_q = u < H, is_v = u >= H + G;
+    const int g = is_q ? 0 : (is_v ? u - H - G : u - H), width = is_v ? Dv : D;
+    const int col = is_q ? u * D : (is_v ? v_col + g * Dv : k_col + g * D);
+    if (!is_q && !write) continue;
+    T* dst = is_q ? q_out + ((size_t)t * H + u) * D
+                  : (is_v ? v_pages + (((size_t)page * G + g) * page_size + in_page) * Dv
+                          : k_pages + (((size_t)page * G + g) * page_size + in_page) * D);
+    const float* w = is_q ? wq : (is_v ? nullptr : wk);
+    float x[PER][V], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+      const int i = (k * 32 + lane) * V;
+      if (i >= width) continue;
+      const PwPack<T, V> p = *reinterpret_cast<const PwPack<T, V>*>(proj + (size_t)t * ld + col + i);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        x[k][e] = to_float(p.v[e]);
+        if (bias) x[k][e] += bias[col + i + e];
+        ss = fmaf(x[k][e], x[k][e], ss);
+      }
+    }
+    const float r = w ? 1.0f / sqrtf(warp_sum(ss) / (float)D + eps) : 1.0f;
+    const bool turn = !is_v && dims > 0;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+      const int i = (k * 32 + lane) * V;
+      if (i >= width) continue;
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        if (w) x[k][e] *= r * w[i + e];
+        if (turn) head[i + e] = x[k][e];
+      }
+    }
+    __syncwarp();
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+      const int i = (k * 32 + lane) * V;
+      if (i >= width) continue;
+      PwPack<T, V> y;
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        const int d = i + e;
+        float v = x[k][e];
+        if (turn && d < dims)
+          v = d < half ? v * hq_smem[d] - head[d + half] * hq_smem[half + d] : v * hq_smem[d - half] + head[d - half] * hq_smem[d];
+        y.v[e] = from_float<T>(v);
+      }
+      *reinterpret_cast<PwPack<T, V>*>(dst + i) = y;
+    }
+    __syncwarp();  // the head's values have been read before the next head's are written
   }
 }
 
@@ -254,6 +350,35 @@ extern "C" int q3_pw_qkv_post(const void* proj, int ld, int k_col, int v_col, in
                                 (const E*)proj, ld, k_col, v_col, H, G, D, Dv, wq, wk, eps, dims, freq, mag, positions,
                                 tok_seq, table, stride, page_size, num_pages, (E*)q_out, (E*)k_pages, (E*)v_pages,
                                 write_cache, status))
+  return q3::launch_status();
+}
+
+// has_kv = 0: the projection holds queries only, and the pages are neither read nor written.
+extern "C" int q3_head_qkv_post(const void* proj, int ld, int k_col, int v_col, int has_kv, int H, int G, int D, int Dv,
+                                const float* bias, const float* wq, const float* wk, float eps, int dims, const float* freq,
+                                float mag, const int* positions, const int* tok_seq, const int* table, int stride,
+                                int page_size, int num_pages, void* q_out, void* k_pages, void* v_pages, int dtype, int T,
+                                int* status, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G || D <= 0 || D > 32 * q3::PW_PER || Dv <= 0 || Dv > 32 * q3::PW_PER || dims < 0 || dims > D ||
+      dims % 2 || page_size <= 0 || stride <= 0)
+    return Q3_ERR_SIZE;
+  const size_t smem = (((dims + 3) & ~3) + q3::HQ_WARPS * ((D + 3) & ~3)) * sizeof(float);
+  const bool by4 = D % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && k_col % 4 == 0 && v_col % 4 == 0 && (uintptr_t)proj % 16 == 0 &&
+                   (uintptr_t)q_out % 16 == 0 && (uintptr_t)k_pages % 16 == 0 && (uintptr_t)v_pages % 16 == 0;
+#define Q3_HQ(V)                                                                                                           \
+  Q3_BY_DTYPE(dtype, q3::launch(q3::head_qkv_post_kernel<E Q3_COMMA V>, dim3(T), dim3(q3::HQ_WARPS * 32), smem, stream,    \
+                                (const E*)proj, ld, k_col, v_col, has_kv, H, G, D, Dv, bias, wq, wk, eps, dims, freq, mag, \
+                                positions, tok_seq, table, stride, page_size, num_pages, (E*)q_out, (E*)k_pages,           \
+                                (E*)v_pages, status))
+#define Q3_COMMA ,
+  if (by4) {
+    Q3_HQ(4)
+  } else {
+    Q3_HQ(1)
+  }
+#undef Q3_HQ
+#undef Q3_COMMA
   return q3::launch_status();
 }
 

@@ -15,8 +15,8 @@ import torch
 from ..cache.manager import CacheLayout, layout_of
 from ..config.model_config import ModelConfig
 from ..kernels import ops
-from ..parts.base import (EMBEDDING_OUTPUT, EMBEDDING_SIDE, LAYER_REPEAT, NEXT_NORM_WEIGHT, STREAM_SUMSQ, ModelSpec, Runtime,
-                          StepContext)
+from ..parts.base import (EMBEDDING_OUTPUT, EMBEDDING_SIDE, LAYER_REPEAT, NEXT_NORM_WEIGHT, STREAM_SUMSQ, ModelSpec,
+                          PagedCacheSpec, Runtime, StepContext)
 from ..registry import build_model_spec, create_part, load_config
 from ..weights.loader import load_weights
 from ..weights.random_init import random_weights_on_device
@@ -33,6 +33,18 @@ def resolve_dtype(dtype) -> torch.dtype:
         return DTYPES[str(dtype).lower()]
     except KeyError:
         raise ValueError(f"dtype must be bfloat16 or float32, got '{dtype}'") from None
+
+
+def shared_need(a, b):
+    """What a cache has to keep for two layers that use it: pages of the same planes may differ in how far back the layers
+    read, and then keep what the one that reads farther needs.  None if the needs do not go together."""
+    if a == b:
+        return a
+    if not (isinstance(a, PagedCacheSpec) and isinstance(b, PagedCacheSpec)) or (a.planes, a.entry_tokens) != (b.planes, b.entry_tokens):
+        return None
+    if a.window is None or b.window is None:
+        return PagedCacheSpec(a.planes, None, a.entry_tokens)
+    return PagedCacheSpec(a.planes, max(a.window, b.window), a.entry_tokens, max(a.keep_first, b.keep_first))
 
 
 class Model:
@@ -64,14 +76,15 @@ class Model:
         return specs
 
     def cache_layout(self) -> CacheLayout:
-        """What every cache id of the run order has to hold, as its writer's mixer asks."""
+        """What every cache id of the run order has to hold, as its writer's mixer and the layers that read it ask."""
         needs: Dict[int, object] = {}
         for call in self.spec.order:
             if call.cache is None:
                 continue
             need = self.layers[call.layer].cache_spec()
             if call.cache in needs:
-                if needs[call.cache] != need:
+                need = shared_need(needs[call.cache], need)
+                if need is None:
                     raise ValueError(f"cache {call.cache} is used by layers with different needs")
                 if call.write_cache:
                     raise ValueError(f"cache {call.cache} has two writers in the run order")

@@ -84,7 +84,12 @@ _SIGNATURES = {
                   _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p],
     "q3_scale_add_rmsnorm": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_float,
                              _c_void_p],
-    "q3_gated_act": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "q3_gated_act": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_void_p],
+    "q3_gemm_skinny_gated": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float,
+                             _c_void_p],
+    "q3_gemm_skinny_groups": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "q3_gemm_tc_gated": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_int,
+                         _c_void_p, _c_void_p],
     "q3_token_shift": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                        _c_int, _c_int, _c_void_p, _c_void_p],
     "q3_causal_conv": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
@@ -152,6 +157,9 @@ _SIGNATURES = {
     "q3_pw_qkv_post": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_float,
                        _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p,
                        _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+    "q3_head_qkv_post": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p,
+                         _c_void_p, _c_float, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
+                         _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p],
     "q3_pool_blocks": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                        _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                        _c_void_p, _c_void_p],
@@ -167,14 +175,14 @@ _SIGNATURES = {
                        _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p],
     "q3_moe_grouped": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                        _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                       _c_int, _c_void_p, _c_void_p, _c_void_p],
+                       _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p],
     "q3_mingru_scan_chunked": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                                _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                _c_float, _c_void_p, _c_void_p],
-    "q3_moe_route": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-                     _c_float, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "q3_moe_route": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
+                     _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "q3_moe_pairs": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
-                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p],
     "q3_add_dyt": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                    _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "q3_side_gate": [_c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
@@ -183,9 +191,17 @@ _SIGNATURES = {
     "q3_mlstm_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p,
                       _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                       _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
-    "q3_sum_norm": [_c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_float,
-                    _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-                    _c_float, _c_void_p],
+    "q3_sum_norm": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p,
+                    _c_void_p, _c_void_p, _c_float, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
+                    _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p],
+    "q3_sum_mix": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_float, _c_void_p, _c_int, _c_void_p, _c_void_p,
+                   _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+    "q3_channel_memory_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
+                               _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+    "q3_channel_memory_scan_mma": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
+                                   _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
+                                   _c_void_p, _c_void_p],
+    "q3_low_rank_decay": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
     "q3_memory_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p,
                        _c_void_p, _c_void_p, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int,
                        _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
@@ -252,6 +268,10 @@ def library() -> ctypes.CDLL:
                 lib.q3_memory_chunk.restype = _c_int
                 lib.q3_memory_mma_takes.argtypes = [_c_int, _c_int]
                 lib.q3_memory_mma_takes.restype = _c_int
+                lib.q3_channel_chunk.argtypes = []
+                lib.q3_channel_chunk.restype = _c_int
+                lib.q3_channel_mma_takes.argtypes = [_c_int, _c_int]
+                lib.q3_channel_mma_takes.restype = _c_int
                 lib.q3_moe_tile_rows.argtypes = []
                 lib.q3_moe_tile_rows.restype = _c_int
                 lib.q3_sample_scratch_bytes.argtypes = [_c_int]
@@ -439,15 +459,15 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float
 
 
 def gemm_f32_nt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
-    """out[M, N] = a[M, K] @ w[N, K]^T in plain float32 (no tensor cores)."""
+    """out[M, N] = a[M, K] @ w[N, K]^T in plain float32 (no tensor cores).  ``out`` may be a column view of a wider buffer."""
     _check("gemm_f32_nt.a", a, torch.float32)
     _check("gemm_f32_nt.w", w, torch.float32)
-    _check("gemm_f32_nt.out", out, torch.float32)
     M, K = a.shape
     N = w.shape[0]
-    if w.shape[1] != K or tuple(out.shape) != (M, N):
-        raise KernelError(f"gemm_f32_nt: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
-    code = library().q3_gemm_f32_nt(a.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, K, K, N, _stream())
+    if (w.shape[1] != K or tuple(out.shape) != (M, N) or out.dtype != torch.float32 or not out.is_cuda
+            or (N > 1 and out.stride(1) != 1)):
+        raise KernelError(f"gemm_f32_nt: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} {out.dtype}")
+    code = library().q3_gemm_f32_nt(a.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, K, K, out.stride(0), _stream())
     _done("gemm_f32_nt", code, f"M {M} N {N} K {K}")
 
 
@@ -529,7 +549,8 @@ def attn_ref(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out:
     _done("attn_ref", code, f"heads {Hq}/{Hkv}, head_dim {D}")
 
 
-ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "none": 3, "relu_sq": 4}
+# "limited" is a form of a gate and its up value together (both held back by a limit): g sigmoid(1.702 g) (u + 1)
+ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "none": 3, "relu_sq": 4, "limited": 5}
 
 
 def activation_code(name: str, gate: bool = False) -> int:
@@ -538,16 +559,27 @@ def activation_code(name: str, gate: bool = False) -> int:
     return ACTIVATIONS[name]
 
 
-def gated_act(gate_up: torch.Tensor, out: torch.Tensor, interleave8: bool = False, activation: str = "silu") -> None:
+def _gate_bias(name: str, bias: Optional[torch.Tensor], columns: int) -> None:
+    if bias is not None:
+        _check(f"{name}.bias", bias, torch.float32)
+        if bias.numel() != columns:
+            raise KernelError(f"{name}: a bias of {bias.numel()} values for {columns} columns")
+
+
+def gated_act(gate_up: torch.Tensor, out: torch.Tensor, interleave8: bool = False, activation: str = "silu",
+              bias: Optional[torch.Tensor] = None, limit: float = 0.0) -> None:
     """out = up * act(gate); gate = first half of the columns and up = second half, or with
-    ``interleave8`` alternating blocks of eight columns (gate, up, gate, up, ...)."""
+    ``interleave8`` alternating blocks of eight columns (gate, up, gate, up, ...).  ``bias`` (float32, in the order of the
+    columns) is added first; ``limit``: of the "limited" form."""
     _check("gated_act.gate_up", gate_up)
     _check("gated_act.out", out, gate_up.dtype)
     T, two_i = gate_up.shape
     if two_i % 2 or tuple(out.shape) != (T, two_i // 2):
         raise KernelError(f"gated_act: gate_up {tuple(gate_up.shape)}, out {tuple(out.shape)}")
+    _gate_bias("gated_act", bias, two_i)
     code = library().q3_gated_act(gate_up.data_ptr(), out.data_ptr(), dtype_tag(out.dtype), T, two_i // 2,
-                                  1 if interleave8 else 0, activation_code(activation, gate=True), _stream())
+                                  1 if interleave8 else 0, activation_code(activation, gate=True), _ptr(bias), float(limit),
+                                  _stream())
     _done("gated_act", code, f"width {two_i // 2}")
 
 
@@ -564,9 +596,11 @@ def gemm_skinny_takes(rows: int, weight: torch.Tensor) -> bool:
 
 
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu_blocks: bool = False,
-                activation: str = "silu", plain_activation: Optional[str] = None) -> None:
+                activation: str = "silu", plain_activation: Optional[str] = None, bias: Optional[torch.Tensor] = None,
+                limit: float = 0.0) -> None:
     """out[T, N] = x[T, K] @ w[N, K]^T for T <= 16, bfloat16 in, out bfloat16 or float32.
-    ``swiglu_blocks``: w's rows alternate gate/up in blocks of eight and out is [T, N / 2] = up * act(gate).
+    ``swiglu_blocks``: w's rows alternate gate/up in blocks of eight and out is [T, N / 2] = up * act(gate), behind a
+    ``bias`` (float32 [N], in the order of w's rows) if one is given; ``limit``: of the "limited" form.
     ``plain_activation`` (without ``swiglu_blocks``): out = act(x w^T), the activation applied before the store."""
     _check("gemm_skinny.x", x, torch.bfloat16)
     _check("gemm_skinny.w", w, torch.bfloat16)
@@ -576,12 +610,36 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu_bloc
     want_cols = N // 2 if swiglu_blocks else N
     if w.shape[1] != K or tuple(out.shape) != (T, want_cols) or out.dtype not in (torch.bfloat16, torch.float32):
         raise KernelError(f"gemm_skinny: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} {out.dtype}")
+    if bias is not None and not swiglu_blocks:
+        raise KernelError("gemm_skinny: a bias only in front of a gate")
+    if swiglu_blocks and (bias is not None or activation == "limited"):
+        _gate_bias("gemm_skinny", bias, N)
+        if out.dtype != torch.bfloat16:
+            raise KernelError(f"gemm_skinny: a gated product leaves bfloat16, not {out.dtype}")
+        code = library().q3_gemm_skinny_gated(x.data_ptr(), w.data_ptr(), out.data_ptr(), T, N, K, want_cols,
+                                              activation_code(activation, gate=True), _ptr(bias), float(limit), _stream())
+        _done("gemm_skinny", code, f"T {T} N {N} K {K}")
+        return
     code = library().q3_gemm_skinny(x.data_ptr(), w.data_ptr(), out.data_ptr(), T, N, K, want_cols,
                                     1 if out.dtype == torch.float32 else 0,
                                     1 + activation_code(activation, gate=True) if swiglu_blocks else (
                                         -1 - activation_code(plain_activation, gate=True) if plain_activation else 0),
                                     _stream())
     _done("gemm_skinny", code, f"T {T} N {N} K {K}")
+
+
+def gemm_skinny_groups(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """Several few-rows products in one launch: x [n, T, K], w [n * rows, K] with ``rows`` a multiple of 16, and columns
+    i rows .. (i + 1) rows - 1 of out [T, n * rows] are x[i] times those rows of w.  T <= 16, bfloat16."""
+    _check("gemm_skinny_groups.x", x, torch.bfloat16)
+    _check("gemm_skinny_groups.w", w, torch.bfloat16)
+    _check("gemm_skinny_groups.out", out, torch.bfloat16)
+    n, T, K = x.shape
+    N = w.shape[0]
+    if w.shape[1] != K or N % n or tuple(out.shape) != (T, N):
+        raise KernelError(f"gemm_skinny_groups: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
+    code = library().q3_gemm_skinny_groups(x.data_ptr(), w.data_ptr(), out.data_ptr(), T, N, K, N // n, N, _stream())
+    _done("gemm_skinny_groups", code, f"T {T} N {N} K {K} in {n} groups")
 
 
 SUMSQ_ROWS = 16  # row pitch of the partial sums of squares that the fused few-rows products exchange
@@ -727,14 +785,22 @@ def gemm_tc_swiglu_pays(rows: int, weight: torch.Tensor) -> Optional[str]:
     return "single" if narrow and rows >= 128 else None
 
 
-GEMM_TC_GATES = {"silu": 1, "relu": 2}  # the gates that the tcgen05 product's epilogue applies
+GEMM_TC_GATES = {"silu": 1, "relu": 2}  # the gates with an epilogue of their own in the tcgen05 product
+GEMM_TC_BIASED_GATES = ("silu", "gelu_tanh", "limited")  # those of the epilogue that takes a bias and a limit
+
+
+def gemm_tc_gate_takes(activation: str, biased: bool) -> bool:
+    """Whether the tcgen05 product's epilogue applies this gate (behind a bias, if ``biased``)."""
+    return activation in GEMM_TC_BIASED_GATES or (activation in GEMM_TC_GATES and not biased)
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Tensor,
-            swiglu_blocks: bool = False, pair: bool = False, activation: str = "silu") -> None:
+            swiglu_blocks: bool = False, pair: bool = False, activation: str = "silu", bias: Optional[torch.Tensor] = None,
+            limit: float = 0.0) -> None:
     """out[M, N] = x[M, K] @ w[N, K]^T on the tcgen05 tensor cores (TMA-fed, accumulator in TMEM).
     ``swiglu_blocks``: w's rows alternate gate/up in blocks of eight and out is [M, N / 2] = up * act(gate),
-    ``activation`` one of ``GEMM_TC_GATES``.
+    ``activation`` one that ``gemm_tc_gate_takes``, behind a ``bias`` (float32 [N], in the order of w's rows) if one is
+    given; ``limit``: of the "limited" form.
     ``pair``: by pairs of CTAs on 256 x 256 tiles (the paired instruction) instead of single CTAs."""
     _check("gemm_tc.x", x, torch.bfloat16)
     _check("gemm_tc.w", w, torch.bfloat16)
@@ -744,6 +810,17 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.T
     want_cols = N // 2 if swiglu_blocks else N
     if w.shape[1] != K or tuple(out.shape) != (M, want_cols) or out.dtype not in (torch.bfloat16, torch.float32):
         raise KernelError(f"gemm_tc: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} {out.dtype}")
+    if bias is not None and not swiglu_blocks:
+        raise KernelError("gemm_tc: a bias only in front of a gate")
+    if swiglu_blocks and (bias is not None or activation not in GEMM_TC_GATES):
+        _gate_bias("gemm_tc", bias, N)
+        if out.dtype != torch.bfloat16:
+            raise KernelError(f"gemm_tc: a gated product leaves bfloat16, not {out.dtype}")
+        code = library().q3_gemm_tc_gated(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, want_cols,
+                                          activation_code(activation, gate=True), _ptr(bias), float(limit), 1 if pair else 0,
+                                          status.data_ptr(), _stream())
+        _done("gemm_tc", code, f"M {M} N {N} K {K}{' pair' if pair else ''}, {activation} gate")
+        return
     entry = library().q3_gemm_tc_pair if pair else library().q3_gemm_tc
     code = entry(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, want_cols,
                  1 if out.dtype == torch.float32 else 0, GEMM_TC_GATES[activation] if swiglu_blocks else 0,
@@ -1884,6 +1961,45 @@ def pw_qkv_post(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, heads: i
     _done("pw_qkv_post", code, f"heads {heads}/{kv_heads}, dim {dim}, vdim {vdim}, rotated {dims}")
 
 
+def head_qkv_post(proj: torch.Tensor, q_col: int, k_col: Optional[int], v_col: Optional[int], heads: int, kv_heads: int,
+                  dim: int, vdim: int, bias: Optional[torch.Tensor], q_norm: Optional[torch.Tensor],
+                  k_norm: Optional[torch.Tensor], eps: float, dims: int, freq: torch.Tensor, magnitude: float,
+                  positions: torch.Tensor, tok_seq: torch.Tensor, table: torch.Tensor, q_out: torch.Tensor,
+                  k_pages: torch.Tensor, v_pages: torch.Tensor, status: torch.Tensor) -> None:
+    """Like ``pw_qkv_post`` with a ``bias`` (float32, one value per column from ``q_col`` on, or None) on the projection and an
+    RMS norm per head (weights ``q_norm`` and ``k_norm`` [dim], shared by the heads, or None).  ``k_col`` and ``v_col`` None:
+    ``proj`` holds queries only and the pages stay as they are (a layer that reads the keys and values of another)."""
+    _check("head_qkv_post.proj", proj)
+    has_kv = k_col is not None
+    if has_kv != (v_col is not None):
+        raise KernelError("head_qkv_post: keys and values, or neither")
+    _check("head_qkv_post.q_out", q_out, proj.dtype)
+    _check("head_qkv_post.k_pages", k_pages, proj.dtype)
+    _check("head_qkv_post.v_pages", v_pages, proj.dtype)
+    for name, t in (("bias", bias), ("q_norm", q_norm), ("k_norm", k_norm), ("freq", freq)):
+        if t is not None:
+            _check(f"head_qkv_post.{name}", t, torch.float32)
+    for name, t in (("positions", positions), ("tok_seq", tok_seq), ("table", table)):
+        _check(f"head_qkv_post.{name}", t, torch.int32)
+    T, ld = proj.shape
+    k_at, v_at = (int(k_col), int(v_col)) if has_kv else (int(q_col), int(q_col))
+    ends = [q_col + heads * dim] + ([k_at + kv_heads * dim, v_at + kv_heads * vdim] if has_kv else [])
+    if (tuple(q_out.shape) != (T, heads, dim) or min(q_col, k_at - q_col, v_at - q_col) < 0 or max(ends) > ld
+            or (bias is not None and bias.numel() < max(ends) - q_col)
+            or any(w is not None and w.numel() != dim for w in (q_norm, k_norm)) or freq.numel() < dims // 2
+            or tuple(k_pages.shape[1:]) != (kv_heads, k_pages.shape[2], dim)
+            or tuple(v_pages.shape) != (k_pages.shape[0], kv_heads, k_pages.shape[2], vdim)):
+        raise KernelError(f"head_qkv_post: proj {tuple(proj.shape)}, q_out {tuple(q_out.shape)}, k pages "
+                          f"{tuple(k_pages.shape)}, v pages {tuple(v_pages.shape)}")
+    code = library().q3_head_qkv_post(proj.data_ptr() + int(q_col) * proj.element_size(), ld, k_at - int(q_col),
+                                      v_at - int(q_col), 1 if has_kv else 0, heads, kv_heads, dim, vdim, _ptr(bias),
+                                      _ptr(q_norm), _ptr(k_norm), float(eps), int(dims), freq.data_ptr(), float(magnitude),
+                                      positions.data_ptr(), tok_seq.data_ptr(), table.data_ptr(), table.shape[1],
+                                      k_pages.shape[2], k_pages.shape[0], q_out.data_ptr(), k_pages.data_ptr(),
+                                      v_pages.data_ptr(), dtype_tag(proj.dtype), T, status.data_ptr(), _stream())
+    _done("head_qkv_post", code, f"heads {heads}/{kv_heads}, dim {dim}, vdim {vdim}, rotated {dims}")
+
+
 def pool_blocks(k_pages: torch.Tensor, v_pages: torch.Tensor, pk_pages: torch.Tensor, pv_pages: torch.Tensor,
                 q_start: torch.Tensor, kv_len: torch.Tensor, table: torch.Tensor, ptable: torch.Tensor, num_seqs: int,
                 max_q_len: int, pool: int, status: torch.Tensor) -> None:
@@ -2084,38 +2200,52 @@ MOE_SCORES = {"sigmoid": 0, "softmax": 1}  # what makes scores of the router's l
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.Tensor, weights: torch.Tensor,
-              scale: float, score: str = "sigmoid", groups: int = 1, keep: int = 1, renormalise: bool = False) -> None:
+              scale: float, score: str = "sigmoid", groups: int = 1, keep: int = 1, renormalise: bool = False,
+              logit_bias: Optional[torch.Tensor] = None, share: Optional[torch.Tensor] = None) -> None:
     """Scores s = sigmoid(h router^T) (``score="softmax"``: softmax over the experts) in float32; ``ids`` [T, top] the
     experts with the largest s + bias, ``weights`` [T, top] their s * scale (``renormalise``: divided by the sum of the
     chosen s + 1e-20).  ``groups`` > 1: only experts of the ``keep`` groups of neighbours with the largest best member can
-    be chosen."""
+    be chosen.  ``logit_bias`` [E]: added to the logits before anything else.  ``share`` [T]: ``router`` then has one more
+    row, the sigmoid of whose product goes there (what a shared expert's output is multiplied by)."""
     _check("moe_route.h", h)
     _check("moe_route.router", router, torch.float32)
     _check("moe_route.ids", ids, torch.int32)
     _check("moe_route.weights", weights, torch.float32)
     T, W = h.shape
-    E = router.shape[0]
+    E = router.shape[0] - (0 if share is None else 1)
     top = ids.shape[1]
-    if bias is not None:
-        _check("moe_route.bias", bias, torch.float32)
-    if (router.shape[1] != W or tuple(ids.shape) != (T, top) or tuple(weights.shape) != (T, top)
-            or (bias is not None and bias.numel() != E)):
+    for name, t, n in (("bias", bias, E), ("logit_bias", logit_bias, E), ("share", share, T)):
+        if t is not None:
+            _check(f"moe_route.{name}", t, torch.float32)
+            if t.numel() != n:
+                raise KernelError(f"moe_route: {name} has {t.numel()} values for {n}")
+    if router.shape[1] != W or tuple(ids.shape) != (T, top) or tuple(weights.shape) != (T, top):
         raise KernelError(f"moe_route: h {tuple(h.shape)}, router {tuple(router.shape)}, ids {tuple(ids.shape)}")
-    code = library().q3_moe_route(h.data_ptr(), router.data_ptr(), _ptr(bias), ids.data_ptr(), weights.data_ptr(),
-                                  dtype_tag(h.dtype), T, W, E, top, float(scale), MOE_SCORES[score], int(groups), int(keep),
+    code = library().q3_moe_route(h.data_ptr(), router.data_ptr(), _ptr(bias), _ptr(logit_bias), ids.data_ptr(),
+                                  weights.data_ptr(), _ptr(share), dtype_tag(h.dtype), T, W, E, top, float(scale), MOE_SCORES[score], int(groups), int(keep),
                                   1 if renormalise else 0, _stream())
     _done("moe_route", code, f"experts {E}, top {top}")
 
 
+def _base_weights(name: str, base_weights: Optional[torch.Tensor], base: Optional[torch.Tensor]) -> None:
+    if base_weights is not None:
+        _check(f"{name}.base_weights", base_weights, torch.float32)
+        if base is None or base_weights.numel() != base.shape[0]:
+            raise KernelError(f"{name}: one weight for every row of a base")
+
+
 def moe_pairs(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
               base: Optional[torch.Tensor], act_buf: torch.Tensor, out: torch.Tensor, activation: str,
-              gate_block: int = 0, in_weights: Optional[torch.Tensor] = None) -> None:
+              gate_block: int = 0, in_weights: Optional[torch.Tensor] = None, base_weights: Optional[torch.Tensor] = None,
+              limit: float = 0.0) -> None:
     """out[t] = base[t] + sum_k weights[t, k] down[ids[t, k]] act(up[ids[t, k]] h[t]); up [E, F, W], down [E, W, F];
     ``act_buf`` [T * top, F] receives the activations.  Every (token, expert) pair streams its expert once.
     ``gate_block`` > 0: gated experts, act(gate h) * (up h), ``up`` being [E, 2 F, W] with gate and up rows alternating
     in blocks of so many rows.  ``in_weights`` [T, top]: what multiplies the expert's input (``weights`` still
-    multiply its output: ones, for a design that weighs the input only)."""
+    multiply its output: ones, for a design that weighs the input only).  ``base_weights`` [T]: what multiplies the rows of
+    ``base``.  ``limit``: of the "limited" form of a gate."""
     _check("moe_pairs.h", h)
+    _base_weights("moe_pairs", base_weights, base)
     for name, t in (("up", up), ("down", down), ("act_buf", act_buf), ("out", out)):
         _check(f"moe_pairs.{name}", t, h.dtype)
     _check("moe_pairs.ids", ids, torch.int32)
@@ -2134,7 +2264,8 @@ def moe_pairs(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.
                           f"{tuple(ids.shape)}, activations {tuple(act_buf.shape)}, out {tuple(out.shape)}")
     code = library().q3_moe_pairs(h.data_ptr(), up.data_ptr(), down.data_ptr(), ids.data_ptr(), weights.data_ptr(),
                                   _ptr(base), act_buf.data_ptr(), out.data_ptr(), dtype_tag(h.dtype), T, W, F, E, top,
-                                  activation_code(activation, gate=True), int(gate_block), _ptr(in_weights), _stream())
+                                  activation_code(activation, gate=True), int(gate_block), _ptr(in_weights),
+                                  _ptr(base_weights), float(limit), _stream())
     _done("moe_pairs", code, f"experts {E}, top {top}, inner {F}")
 
 
@@ -2185,9 +2316,12 @@ class MoeScratch:
 
 def moe_grouped(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
                 base: Optional[torch.Tensor], out: torch.Tensor, activation: str, scratch: MoeScratch,
-                status: torch.Tensor, gated: bool = False, in_weights: Optional[torch.Tensor] = None) -> None:
+                status: torch.Tensor, gated: bool = False, in_weights: Optional[torch.Tensor] = None,
+                base_weights: Optional[torch.Tensor] = None, limit: float = 0.0) -> None:
     """out = base + sum_k weights[:, k] * down[ids[:, k]] act(up[ids[:, k]] h) for many tokens (bfloat16): the pairs
-    sorted by expert into whole tiles, both products of all experts as one grouped tensor-core product each."""
+    sorted by expert into whole tiles, both products of all experts as one grouped tensor-core product each.
+    ``base_weights``, ``limit``: as in ``moe_pairs``."""
+    _base_weights("moe_grouped", base_weights, base)
     _check("moe_grouped.h", h, torch.bfloat16)
     _check("moe_grouped.up", up, torch.bfloat16)
     _check("moe_grouped.down", down, torch.bfloat16)
@@ -2216,21 +2350,23 @@ def moe_grouped(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torc
                                     _ptr(base), out.data_ptr(), scratch.sorted_in.data_ptr(), scratch.sorted_act.data_ptr(),
                                     scratch.sorted_out.data_ptr(), scratch.pos.data_ptr(), scratch.src.data_ptr(),
                                     scratch.meta.data_ptr(), T, W, F, E, top, cap, activation_code(activation, gate=True),
-                                    1 if gated else 0, _ptr(in_weights), status.data_ptr(), _stream())
+                                    1 if gated else 0, _ptr(in_weights), _ptr(base_weights), float(limit), status.data_ptr(),
+                                    _stream())
     _done("moe_grouped", code, f"experts {E}, top {top}, width {W}, ff {F}")
 
 
 def routed_experts(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
                    base: Optional[torch.Tensor], act_buf: torch.Tensor, out: torch.Tensor, activation: str,
                    scratch: Optional[MoeScratch] = None, status: Optional[torch.Tensor] = None, gate_block: int = 0,
-                   in_weights: Optional[torch.Tensor] = None) -> None:
+                   in_weights: Optional[torch.Tensor] = None, base_weights: Optional[torch.Tensor] = None,
+                   limit: float = 0.0) -> None:
     """The chosen experts of a step's tokens, by the kernels that suit dtype and shape: with ``scratch``, from
     ``MOE_GROUPED_FROM`` tokens on, the grouped tensor-core products; otherwise a pair at a time (``moe_pairs``)."""
     if scratch is not None and status is not None and h.shape[0] >= MOE_GROUPED_FROM:
         moe_grouped(h, up, down, ids, weights, base, out, activation, scratch, status, gated=gate_block > 0,
-                    in_weights=in_weights)
+                    in_weights=in_weights, base_weights=base_weights, limit=limit)
     else:
-        moe_pairs(h, up, down, ids, weights, base, act_buf, out, activation, gate_block, in_weights)
+        moe_pairs(h, up, down, ids, weights, base, act_buf, out, activation, gate_block, in_weights, base_weights, limit)
 
 
 # ------------------------------------------------------------------ Dynamic Tanh around sub-layers, a token's second embedding
@@ -2422,15 +2558,31 @@ def mlstm_out(o: torch.Tensor, proj: torch.Tensor, g_col: int, weight: torch.Ten
 SUM_NORM_TERMS = 3  # open terms that one pass over the stream takes
 
 
-def sum_norm(stream: torch.Tensor, terms, term_eps: float, weight: torch.Tensor, out: torch.Tensor, eps: float,
-             second=None, rows: Optional[torch.Tensor] = None) -> None:
+def _sum_term(name: str, term, dtype: torch.dtype, T: int, W: int):
+    delta, w, scale, bias = term if len(term) == 4 else (*term, None)
+    if delta is not None:
+        _check(f"{name}.delta", delta, dtype)
+        if tuple(delta.shape) != (T, W):
+            raise KernelError(f"{name}: stream {(T, W)}, term {tuple(delta.shape)}")
+    for what, t in (("term_weight", w), ("term_bias", bias)):
+        if t is not None:
+            _check(f"{name}.{what}", t, torch.float32)
+            if t.numel() != W:
+                raise KernelError(f"{name}: {what} {tuple(t.shape)} for width {W}")
+    return [_ptr(delta), _ptr(bias), _ptr(w), float(scale)]
+
+
+def sum_norm(stream: torch.Tensor, terms, term_eps: float, weight: Optional[torch.Tensor], out: Optional[torch.Tensor],
+             eps: float, second=None, rows: Optional[torch.Tensor] = None) -> None:
     """stream += sum of ``terms``, then out = stream / rms(stream) * weight.  A term is (delta [T, W], weight or None,
-    scale): with a weight delta / sqrt(mean(delta^2) + term_eps) * weight * scale, without one delta as it is.
+    scale, and optionally a bias that is added to delta first): with a weight delta / sqrt(mean(delta^2) + term_eps) *
+    weight * scale, without one delta as it is.  ``weight`` None: no norm, ``out`` (or None) receives the new rows.
     ``second``: (weight, out) of another norm of the same rows.  ``rows`` (int32): only these rows are worked out, into
     ``out`` [len(rows), W], and the stream stays as it is."""
     _check("sum_norm.stream", stream, torch.float32)
-    _check("sum_norm.out", out)
-    _check("sum_norm.weight", weight, torch.float32)
+    for name, t, dtype in (("out", out, None), ("weight", weight, torch.float32)):
+        if t is not None:
+            _check(f"sum_norm.{name}", t, dtype)
     T, W = stream.shape
     n = T
     if rows is not None:
@@ -2438,19 +2590,12 @@ def sum_norm(stream: torch.Tensor, terms, term_eps: float, weight: torch.Tensor,
         n = rows.numel()
     if len(terms) > SUM_NORM_TERMS:
         raise KernelError(f"sum_norm: {len(terms)} terms, the kernel takes {SUM_NORM_TERMS}")
-    if tuple(out.shape) != (n, W) or weight.numel() != W:
-        raise KernelError(f"sum_norm: stream {tuple(stream.shape)}, out {tuple(out.shape)}, weight {tuple(weight.shape)}")
+    if (out is not None and tuple(out.shape) != (n, W)) or (weight is not None and (weight.numel() != W or out is None)):
+        raise KernelError(f"sum_norm: stream {tuple(stream.shape)}, out and weight do not fit")
     args = []
-    for delta, w, scale in list(terms) + [(None, None, 1.0)] * (SUM_NORM_TERMS - len(terms)):
-        if delta is not None:
-            _check("sum_norm.delta", delta, out.dtype)
-            if tuple(delta.shape) != (T, W):
-                raise KernelError(f"sum_norm: stream {tuple(stream.shape)}, term {tuple(delta.shape)}")
-        if w is not None:
-            _check("sum_norm.term_weight", w, torch.float32)
-            if w.numel() != W:
-                raise KernelError(f"sum_norm: term weight {tuple(w.shape)} for width {W}")
-        args += [_ptr(delta), _ptr(w), float(scale)]
+    dtype = out.dtype if out is not None else (terms[0][0].dtype if terms else torch.float32)
+    for term in list(terms) + [(None, None, 1.0)] * (SUM_NORM_TERMS - len(terms)):
+        args += _sum_term("sum_norm", term, dtype, T, W)
     w2 = out2 = None
     if second is not None:
         w2, out2 = second
@@ -2458,12 +2603,35 @@ def sum_norm(stream: torch.Tensor, terms, term_eps: float, weight: torch.Tensor,
         _check("sum_norm.second", out2, out.dtype)
         if tuple(out2.shape) != (n, W) or w2.numel() != W:
             raise KernelError(f"sum_norm: second norm: out {tuple(out2.shape)}, weight {tuple(w2.shape)}")
-    code = library().q3_sum_norm(stream.data_ptr(), *args, len(terms), float(term_eps), weight.data_ptr(), out.data_ptr(),
-                                 _ptr(w2), _ptr(out2), _ptr(rows), n, dtype_tag(out.dtype), T, W, float(eps), _stream())
+    code = library().q3_sum_norm(stream.data_ptr(), *args, len(terms), float(term_eps), _ptr(weight), _ptr(out),
+                                 _ptr(w2), _ptr(out2), _ptr(rows), n, dtype_tag(dtype), T, W, float(eps), _stream())
     _done("sum_norm", code, f"rows {n}, width {W}")
 
 
-# ------------------------------------------------------------------ matrix memories: fixed decays, the gated delta rule
+def sum_mix(stream: torch.Tensor, term, term_eps: float, mu: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor,
+            tok_seq: torch.Tensor, slot_ids: torch.Tensor, num_seqs: int, out: torch.Tensor, status: torch.Tensor) -> None:
+    """For every row m of ``mu`` [M, W]: out[m, t] = x_t + (x_{t-1} - x_t) * mu[m], x the float32 stream and out [M, T, W].  What
+    lies before a portion's first token comes from ``state`` (float32 [slots, W]), which then receives the portion's last x.
+    ``term`` (as in ``sum_norm``, or None) goes into the stream first; only in a step of single tokens."""
+    _check("sum_mix.stream", stream, torch.float32)
+    _check("sum_mix.mu", mu, torch.float32)
+    _check("sum_mix.state", state, torch.float32)
+    _check("sum_mix.out", out)
+    for name, t in (("q_start", q_start), ("tok_seq", tok_seq), ("slot_ids", slot_ids)):
+        _check(f"sum_mix.{name}", t, torch.int32)
+    T, W = stream.shape
+    M = mu.shape[0]
+    if mu.shape[1] != W or tuple(out.shape) != (M, T, W) or state.dim() != 2 or state.shape[1] != W or tok_seq.numel() != T:
+        raise KernelError(f"sum_mix: stream {tuple(stream.shape)}, mu {tuple(mu.shape)}, out {tuple(out.shape)}, state "
+                          f"{tuple(state.shape)}")
+    delta, bias, weight, scale = _sum_term("sum_mix", term if term is not None else (None, None, 1.0), out.dtype, T, W)
+    code = library().q3_sum_mix(stream.data_ptr(), delta, bias, weight, scale, float(term_eps), mu.data_ptr(), M,
+                                state.data_ptr(), q_start.data_ptr(), tok_seq.data_ptr(), slot_ids.data_ptr(), state.shape[0],
+                                out.data_ptr(), dtype_tag(out.dtype), T, int(num_seqs), W, status.data_ptr(), _stream())
+    _done("sum_mix", code, f"{M} mixes, width {W}{', with a term' if delta else ''}, {T} tokens of {num_seqs} requests")
+
+
+# ------------------------------------------------------------------ matrix memories: fixed decays, the gated delta rule, decays per channel
 def memory_max_dim() -> int:
     """The largest key size per head that ``memory_scan`` takes."""
     if "memory max dim" not in _DEVICE_FACTS:
@@ -2488,6 +2656,82 @@ class DeltaGates:
 
     def __init__(self, proj: torch.Tensor, b_col: int, a_col: int, a_log: torch.Tensor, dt_bias: torch.Tensor):
         self.proj, self.b_col, self.a_col, self.a_log, self.dt_bias = proj, int(b_col), int(a_col), a_log, dt_bias
+
+
+class ChannelDecay:
+    """A decay per token and key channel, by its logarithm (``logw`` float32 [T, heads * dim]), and the bonus with which a token
+    reads itself (float32 [heads, dim])."""
+
+    def __init__(self, logw: torch.Tensor, bonus: torch.Tensor):
+        self.logw, self.bonus = logw, bonus
+
+
+def low_rank_decay(low: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor, logw: torch.Tensor) -> None:
+    """logw[t, c] = -exp(sum_r w2[c, r] tanh(low[t, r]) + w0[c]) in float32 (held at -104, whose exponential is zero):
+    the logarithms of decays that a low-rank projection makes.  ``low`` [T, any] (the first ``w2.shape[1]`` columns)."""
+    for name, t in (("low", low), ("w2", w2), ("w0", w0), ("logw", logw)):
+        _check(f"low_rank_decay.{name}", t, torch.float32)
+    T, ld = low.shape
+    C, R = w2.shape
+    if tuple(logw.shape) != (T, C) or w0.numel() != C or R > ld:
+        raise KernelError(f"low_rank_decay: low {tuple(low.shape)}, w2 {tuple(w2.shape)}, logw {tuple(logw.shape)}")
+    code = library().q3_low_rank_decay(low.data_ptr(), ld, w2.data_ptr(), w0.data_ptr(), logw.data_ptr(), T, C, R, _stream())
+    _done("low_rank_decay", code, f"{C} channels of rank {R}")
+
+
+def channel_matrix_form(dtype: torch.dtype, dim: int, vdim: int) -> bool:
+    """Whether the matrix form of a memory with a decay per channel takes these heads: bfloat16, keys and values alike of 32, 64
+    or 128 values."""
+    return dtype == torch.bfloat16 and bool(library()._lib.q3_channel_mma_takes(int(dim), int(vdim)))
+
+
+class ChannelScratch:
+    """What the matrix form of ``channel_memory_scan`` keeps between its kernels for at most ``max_tokens`` tokens of
+    ``max_seqs`` requests: a state and the summed log-decays per chunk."""
+
+    def __init__(self, alloc, max_tokens: int, max_seqs: int, heads: int, dim: int):
+        self.chunk = int(library()._lib.q3_channel_chunk())
+        self.max_tokens = int(max_tokens)
+        self.max_records = max_tokens // self.chunk + max_seqs + 1
+        self.records = alloc("memory.records", self.max_records * heads * dim * dim, dtype=torch.float32)
+        self.totals = alloc("memory.totals", self.max_records * heads * dim, dtype=torch.float32)
+
+
+def channel_memory_scan(x: torch.Tensor, q_col: int, k_col: int, v_col: int, rule: ChannelDecay, state: torch.Tensor,
+                        q_start: torch.Tensor, slot_ids: torch.Tensor, num_seqs: int, out: torch.Tensor, status: torch.Tensor,
+                        max_q_len: int = 1, scratch: Optional[ChannelScratch] = None) -> None:
+    """A matrix memory per head with a decay per token and key channel: o = (S + diag(u) k v^T)^T q, then S <- diag(w) S + k v^T.
+    ``x`` [T, any]: q, k (heads * dim each) and v (heads * vdim) from the given columns.  ``state`` float32 [slots, heads,
+    vdim, dim] is read and renewed; ``out`` float32 [T, heads * vdim].  With ``scratch`` and a portion of
+    ``MEMORY_CHUNKED_FROM`` tokens or more the step runs in the matrix form (bfloat16 only)."""
+    _check("channel_memory_scan.x", x)
+    for name, t in (("state", state), ("out", out), ("logw", rule.logw), ("bonus", rule.bonus)):
+        _check(f"channel_memory_scan.{name}", t, torch.float32)
+    for name, t in (("q_start", q_start), ("slot_ids", slot_ids)):
+        _check(f"channel_memory_scan.{name}", t, torch.int32)
+    T, ld = x.shape
+    slots, H, Dv, D = state.shape
+    if (tuple(out.shape) != (T, H * Dv) or tuple(rule.logw.shape) != (T, H * D) or rule.bonus.numel() != H * D
+            or min(q_col, k_col, v_col) < 0 or max(q_col + H * D, k_col + H * D, v_col + H * Dv) > ld):
+        raise KernelError(f"channel_memory_scan: x {tuple(x.shape)}, state {tuple(state.shape)}, out {tuple(out.shape)}, "
+                          f"log-decays {tuple(rule.logw.shape)}")
+    if scratch is not None and max_q_len >= MEMORY_CHUNKED_FROM and ld % 8 == 0 and (q_col | k_col | v_col) % 8 == 0:
+        _check("channel_memory_scan.x", x, torch.bfloat16)
+        if (T > scratch.max_tokens or num_seqs + T // scratch.chunk + 1 > scratch.max_records or D != Dv
+                or scratch.records.numel() < scratch.max_records * H * D * D):
+            raise KernelError(f"channel_memory_scan: the scratch was made for {scratch.max_tokens} tokens, the step has {T}")
+        code = library().q3_channel_memory_scan_mma(x.data_ptr(), ld, int(q_col), int(k_col), int(v_col), rule.logw.data_ptr(),
+                                                    rule.bonus.data_ptr(), state.data_ptr(), q_start.data_ptr(),
+                                                    slot_ids.data_ptr(), slots, out.data_ptr(), scratch.records.data_ptr(),
+                                                    scratch.totals.data_ptr(), T, int(num_seqs), int(max_q_len), H, D,
+                                                    status.data_ptr(), _stream())
+        _done("channel_memory_scan_mma", code, f"heads {H}, dim {D}")
+        return
+    code = library().q3_channel_memory_scan(x.data_ptr(), ld, int(q_col), int(k_col), int(v_col), rule.logw.data_ptr(),
+                                            rule.bonus.data_ptr(), state.data_ptr(), q_start.data_ptr(), slot_ids.data_ptr(),
+                                            slots, out.data_ptr(), dtype_tag(x.dtype), int(num_seqs), H, D, Dv,
+                                            status.data_ptr(), _stream())
+    _done("channel_memory_scan", code, f"heads {H}, dim {D}, vdim {Dv}")
 
 
 MEMORY_CHUNKED_FROM = 32  # the longest portion of a step from which the matrix form runs

@@ -3,7 +3,7 @@ k, an optional position encoding and an optional sliding window), sigmoid attent
 softmax attention through a latent (one latent vector and one rotated key part per token, shared by the heads; with
 optional output gates and an optional sink in the softmax), softmax attention over a window and pooled blocks, and
 softmax attention over a window that also keeps a request's first tokens, or over all tokens with a bias by distance and
-a sink.
+a sink (or with biases on the projections, a norm per head, a fixed sink, the keys and values of another layer).
 
 Reference: models/self_attn.py:300-386 (packed [T, hidden] input, merged QKV, head norm then
 rotation, keys/values written to pages, causal attention over the cache, output projection),
@@ -23,7 +23,7 @@ import torch
 
 from ..kernels import ops
 from ..registry import create_part, register_part
-from .base import CachePlane, KVCacheSpec, Mixer, PagedCacheSpec, PartSpec, Runtime, StepContext, WeightSpec
+from .base import (CachePlane, KVCacheSpec, Mixer, PagedCacheSpec, PartSpec, PendingTerm, Runtime, StepContext, WeightSpec)
 from .linear import Linear
 
 
@@ -500,6 +500,13 @@ class KeptWindowAttention(Mixer):
     stored size says what B is ("rows" only sizes random weights); at load it becomes one value per head and distance up
     to the distance from which the last row is read.  None: no bias.  It does not go with kept first tokens.
     ``sink``: the learned logits ``<name>.sink`` [H]; nothing is scored or weighted by them and ``scale`` is not applied.
+    ``fixed_sink``: the same with one given logit for all heads and no tensor (0: a one in the denominator).
+
+    ``proj_bias``: the four projections have biases (``<name>.q.b`` and so on), added in float32 before anything else; the
+    output's is left open (``forward`` returns a ``PendingTerm``).  ``qk_norm_eps``: every head of q and of k goes through an
+    RMS norm over ``dim`` before the rotation, with one weight for all heads (``<name>.q.norm``, ``<name>.k.norm`` [dim]).
+    ``shares_kv``: the layer has no tensors for keys and values; its entry of the run order names the cache of a layer that
+    has (of the same head counts, sizes and rotation) and does not write it.
 
     One paged cache (planes ``k`` and ``v``), of which the manager keeps the pages of the last ``window`` tokens and those
     of the first ``keep_first`` (all pages without a window).  The attention kernels are those of the window with pooled blocks, run with blocks of
@@ -508,13 +515,23 @@ class KeptWindowAttention(Mixer):
     part's own."""
 
     graph_capturable = True
-    splittable = True
-    NAMES = {"q": "q", "k": "k", "v": "v", "gate": "g", "out": "o", "bias": "rel", "sink": "sink"}
+    NAMES = {"q": "q", "k": "k", "v": "v", "gate": "g", "out": "o", "bias": "rel", "sink": "sink", "q_bias": "q.b",
+             "k_bias": "k.b", "v_bias": "v.b", "out_bias": "o.b", "q_norm": "q.norm", "k_norm": "k.norm"}
 
     def __init__(self, name: str, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float,
                  window: Optional[int] = None, keep_first: int = 0, position: Optional[PartSpec] = None, gate: bool = True,
-                 names: Optional[Dict[str, str]] = None, bias: Optional[dict] = None, sink: bool = False):
+                 names: Optional[Dict[str, str]] = None, bias: Optional[dict] = None, sink: bool = False,
+                 fixed_sink: Optional[float] = None, proj_bias: bool = False, qk_norm_eps: Optional[float] = None,
+                 shares_kv: bool = False):
         super().__init__(name)
+        self.fixed_sink = None if fixed_sink is None else float(fixed_sink)
+        self.proj_bias, self.shares_kv = bool(proj_bias), bool(shares_kv)
+        self.qk_norm_eps = None if qk_norm_eps is None else float(qk_norm_eps)
+        if sink and self.fixed_sink is not None:
+            raise ValueError(f"attention {name}: a learned sink or a fixed one")
+        if self.proj_bias and gate:
+            raise ValueError(f"attention {name}: output gates beside biases on the projections are not built")
+        self.splittable = not self.proj_bias  # the output's bias stays open, which merged products have no place for
         self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
         if self.num_heads % self.num_kv_heads:
             raise ValueError(f"{self.num_heads} query heads are not a multiple of {self.num_kv_heads} kv heads")
@@ -532,7 +549,12 @@ class KeptWindowAttention(Mixer):
 
     def weight_specs(self) -> List[WeightSpec]:
         t, w, H, G, D, Dv = self.tensors, self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim
-        return [WeightSpec(t["q"], (H * D, w)), WeightSpec(t["k"], (G * D, w)), WeightSpec(t["v"], (G * Dv, w))] + (
+        own = [("q", H * D)] + ([] if self.shares_kv else [("k", G * D), ("v", G * Dv)])
+        vectors = [(f"{k}_bias", n, "normal") for k, n in own + [("out", w)]] if self.proj_bias else []
+        if self.qk_norm_eps is not None:
+            vectors += [(f"{k}_norm", D, "one_plus_normal") for k, _ in own if k != "v"]
+        return [WeightSpec(t[k], (n, w)) for k, n in own] + [
+            WeightSpec(t[k], (n,), kind="vector", init=init) for k, n, init in vectors] + (
             [WeightSpec(t["gate"], (H * Dv, w))] if self.has_gate else []) + (
             [WeightSpec(t["bias"], (int(self.bias["rows"]), H), kind="vector", init="normal", free_dims=(0,))] if self.bias else []) + (
             [WeightSpec(t["sink"], (H,), kind="vector", init="normal")] if self.has_sink else []) + [
@@ -546,7 +568,8 @@ class KeptWindowAttention(Mixer):
     # ------------------------------------------------------------------ the two products and what lies between
     def input_weight(self, weights: Dict[str, torch.Tensor]) -> torch.Tensor:
         t = self.tensors
-        parts = [weights.pop(t[k]) for k in (("q", "k", "v", "gate") if self.has_gate else ("q", "k", "v"))]
+        keys = ["q"] + ([] if self.shares_kv else ["k", "v"]) + (["gate"] if self.has_gate else [])
+        parts = [weights.pop(t[k]) for k in keys]
         dtype = torch.float32 if any(p.dtype == torch.float32 for p in parts) else parts[0].dtype
         return torch.cat([p.to(dtype) for p in parts], dim=0)  # columns of the product: q, k, v, gates
 
@@ -563,12 +586,22 @@ class KeptWindowAttention(Mixer):
         if self.position is not None:
             self.position.setup(rt, weights)
             self.freq, self.magnitude, self.dims = self.position.frequencies()
-        self.dist_bias, self.sink = None, weights[self.tensors["sink"]] if self.has_sink else None
+        t = self.tensors
+        self.dist_bias, self.sink = None, weights[t["sink"]] if self.has_sink else None
+        if self.fixed_sink is not None:
+            self.sink = torch.full((self.num_heads,), self.fixed_sink, dtype=torch.float32, device=rt.device)
+        self.in_bias = self.out_bias = None
+        if self.proj_bias:
+            self.in_bias = torch.cat([weights[t[f"{k}_bias"]] for k in (("q",) if self.shares_kv else ("q", "k", "v"))]).contiguous()
+            self.out_bias = weights[t["out_bias"]]
+        normed = self.qk_norm_eps is not None
+        self.q_norm = weights[t["q_norm"]] if normed else None
+        self.k_norm = weights[t["k_norm"]] if normed and not self.shares_kv else None
         if self.bias:
             table = weights[self.tensors["bias"]]  # [rows, heads]
             index = torch.tensor(distance_buckets(table.shape[0], float(self.bias["most"])), device=rt.device)
             self.dist_bias = table[index].t().contiguous()
-        elif self.has_sink:  # the kernels take a sink beside a bias: one of zeros
+        elif self.sink is not None:  # the kernels take a sink beside a bias: one of zeros
             self.dist_bias = torch.zeros(self.num_heads, 1, dtype=torch.float32, device=rt.device)
         self._q = rt.shared("kwattn.q", rt.max_tokens, self.num_heads, self.dim)
         self._partial = None
@@ -590,8 +623,16 @@ class KeptWindowAttention(Mixer):
         status = self.rt.status
         q = self._q[:T]
         k_col, v_col = column + H * D, column + (H + G) * D
-        ops.pw_qkv_post(proj, column, k_col, v_col, H, G, D, Dv, None, None, 0.0, self.dims, self.freq, self.magnitude,
-                        ctx.positions, ctx.tok_seq, table, q, k_pages, v_pages, write_cache, status)
+        if self.shares_kv and write_cache:
+            raise ValueError(f"attention {self.name}: it has no keys and values of its own to write")
+        if self.proj_bias or self.qk_norm_eps is not None or self.shares_kv:
+            own = write_cache and not self.shares_kv
+            ops.head_qkv_post(proj, column, k_col if own else None, v_col if own else None, H, G, D, Dv, self.in_bias, self.q_norm,
+                              self.k_norm, self.qk_norm_eps or 0.0, self.dims, self.freq, self.magnitude, ctx.positions,
+                              ctx.tok_seq, table, q, k_pages, v_pages, status)
+        else:
+            ops.pw_qkv_post(proj, column, k_col, v_col, H, G, D, Dv, None, None, 0.0, self.dims, self.freq, self.magnitude,
+                            ctx.positions, ctx.tok_seq, table, q, k_pages, v_pages, write_cache, status)
         window, first = (ops.NO_WINDOW, 0) if self.window is None else (self.window, self.keep_first)
         # the kept first tokens are "blocks" of one token read from the token pages, at most keep_first of them
         ops.pooled_window_attention(q, k_pages, v_pages, k_pages, v_pages, ctx, table, table, out, window, 1,
@@ -600,7 +641,8 @@ class KeptWindowAttention(Mixer):
         if self.has_gate:
             ops.sigmoid_gate(out, proj, v_col + G * Dv)
 
-    def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool):
         o = self._o[: x.shape[0]]
         self.core(self.in_proj(x), 0, ctx, cache_id, write_cache, o, 1.0)
-        return self.out_proj(o)
+        y = self.out_proj(o)
+        return y if self.out_bias is None else PendingTerm(y, bias=self.out_bias)

@@ -267,12 +267,14 @@ class PendingNormed:
 
 @dataclass
 class PendingTerm:
-    """Something that still has to be added to the residual stream: ``delta`` as it is, or (with a ``weight``) brought to
-    unit root mean square over its row, times the weight, times ``scale``."""
+    """Something that still has to be added to the residual stream: ``delta`` (with a ``bias``: delta + bias) as it is, or
+    (with a ``weight``) brought to unit root mean square over its row, times the weight, times ``scale``.  A mixer or
+    feed-forward whose last projection has a bias returns its output as such a term, the bias still to be added."""
 
     delta: torch.Tensor  # [T, W] in the compute dtype
     weight: Optional[torch.Tensor] = None  # float32 [W]
     scale: float = 1.0
+    bias: Optional[torch.Tensor] = None  # float32 [W]
 
 
 @dataclass
@@ -285,11 +287,13 @@ class PendingSum:
 
     @staticmethod
     def of(*parts) -> "PendingSum":
-        """The sum of sub-layer outputs, each a tensor or a ``PendingSum``."""
+        """The sum of sub-layer outputs, each a tensor, a ``PendingTerm`` without a weight or a ``PendingSum``."""
         terms, eps = [], None
         for p in parts:
             if not isinstance(p, PendingSum):
-                terms.append(PendingTerm(p))
+                if isinstance(p, PendingTerm) and p.weight is not None:
+                    raise ValueError("a term to be normed comes in a PendingSum, with its epsilon")
+                terms.append(p if isinstance(p, PendingTerm) else PendingTerm(p))
                 continue
             if any(t.weight is not None for t in p.terms):
                 if eps is not None and eps != p.eps:
@@ -297,6 +301,10 @@ class PendingSum:
                 eps = p.eps
             terms += p.terms
         return PendingSum(tuple(terms), 0.0 if eps is None else eps)
+
+    def kernel_terms(self):
+        """The terms as ``ops.sum_norm`` takes them."""
+        return [(t.delta, t.weight, t.scale, t.bias) for t in self.terms]
 
 
 @dataclass
@@ -367,6 +375,12 @@ class Mixer(Part):
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
         raise NotImplementedError
+
+    #: A mixer that reads the float32 residual stream itself (it mixes a token's row with the row before, say) may set this
+    #: and offer ``forward_stream(stream, pending, ctx, cache_id, write_cache)``: like ``forward``, but it first brings
+    #: what is still open (``pending``: a ``PendingSum`` or None) into the stream.  For blocks without a norm in front of
+    #: their mixer.
+    reads_stream = False
 
     #: A mixer that is one product of its input, a core and one product to its output may set this and offer the three
     #: methods below; the ``parallel`` mixer then runs it beside others on one merged input product and one merged

@@ -1,8 +1,8 @@
 """The arrangements of norms, mixer and feed-forward around the residual stream: the norm before each
 sub-layer (``pre_norm``), the norm after each sub-layer's sum (``post_norm``), the norm before each sub-layer
 of a model that keeps several residual streams per token (``hyper_pre_norm``), a norm on both sides of each
-sub-layer (``sandwich_norm``), and both sub-layers side by side on the same stream (``parallel_pre_norm``, at the end of
-the file).
+sub-layer (``sandwich_norm``), both sub-layers side by side on the same stream (``parallel_pre_norm``), and a norm on the
+sub-layers' outputs alone (``output_norm``, at the end of the file).
 
 Pre-norm residual block: h = x + mixer(norm1(x)); y = h + feed_forward(norm2(h)).
 
@@ -22,7 +22,7 @@ import torch
 from ..registry import create_part, register_part
 from ..kernels import ops
 from .base import (EMBEDDING_OUTPUT, EMBEDDING_SIDE, LAYER_REPEAT, NEXT_NORM_WEIGHT, STREAM_SUMSQ, Block, PartSpec, PendingNormed,
-                   PendingStreamWrite, PendingSum, Runtime, StateSpec, StepContext, WeightSpec)
+                   PendingStreamWrite, PendingSum, PendingTerm, Runtime, StateSpec, StepContext, WeightSpec)
 from .linear import Linear
 
 
@@ -487,3 +487,86 @@ class ParallelPreNormBlock(Block):
             return PendingSum.of(self.mixer.forward(self.norm1.add_norm(stream, pending), ctx, cache_id, write_cache))
         x, y = self.norm1.add_norm_pair(stream, pending, self.norm2)
         return PendingSum.of(self.mixer.forward(x, ctx, cache_id, write_cache), self.feed_forward.forward(y))
+
+
+@register_part("block", "output_norm")
+class OutputNormBlock(Block):
+    """A norm on each sub-layer's output and nowhere else; the sub-layers read the stream itself:
+
+        x <- x + norm1(mixer(x)) * s1;   x <- x + norm2(feed_forward(x)) * s2
+
+    The norms are RMS norms, s1 and s2 (``layer_scale``; without it ones) the tensors ``<name>.<scale1>`` and ``.<scale2>``
+    [width], multiplied into the norms' weights at load.  A sub-layer's output is left open (``PendingSum``: what its norm and
+    scale make of it, and the bias of its last projection if it has one); the next kernel over the stream closes it and
+    leaves the rows in the compute dtype for the next projection.  A mixer that reads the float32 stream
+    (``Mixer.reads_stream``) closes what is open before it itself.  ``feed_forward`` (and ``norm2``) may be None."""
+
+    def __init__(self, name: str, width: int, norm1: PartSpec, mixer: PartSpec, norm2: Optional[PartSpec] = None,
+                 feed_forward: Optional[PartSpec] = None, layer_scale: bool = False, names: Optional[Dict[str, str]] = None):
+        super().__init__(name)
+        n = {"norm1": "norm1", "mixer": "mixer", "norm2": "norm2", "feed_forward": "feed_forward", "scale1": "scale1",
+             "scale2": "scale2"}
+        n.update(names or {})
+        self.width, self.layer_scale = int(width), bool(layer_scale)
+        if self.width <= 0:
+            raise ValueError(f"block {name}: needs the stream's width")
+        self.norm1 = create_part("norm", norm1, name=f"{name}.{n['norm1']}")
+        self.mixer = create_part("mixer", mixer, name=f"{name}.{n['mixer']}")
+        self.norm2 = self.feed_forward = None
+        if feed_forward is not None:
+            if norm2 is None:
+                raise ValueError(f"block {name}: a feed-forward needs the norm behind it")
+            self.norm2 = create_part("norm", norm2, name=f"{name}.{n['norm2']}")
+            self.feed_forward = create_part("feed_forward", feed_forward, name=f"{name}.{n['feed_forward']}")
+        for norm in self._norms():
+            if not (hasattr(norm, "eps") and hasattr(norm, "add_norm_pair")):
+                raise ValueError(f"block {name}: {type(norm).__name__} cannot be left open behind a sub-layer")
+        self.scales = [f"{name}.{n['scale1']}", f"{name}.{n['scale2']}"][: len(self._norms())] if self.layer_scale else []
+
+    def _norms(self):
+        return [p for p in (self.norm1, self.norm2) if p is not None]
+
+    def _parts(self):
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.feed_forward) if p is not None]
+
+    @property
+    def graph_capturable(self) -> bool:
+        return all(p.graph_capturable for p in self._parts())
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [s for p in self._parts() for s in p.weight_specs()] + [
+            WeightSpec(t, (self.width,), kind="vector", init="one_plus_normal") for t in self.scales]
+
+    def setup(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
+        super().setup(rt, weights)
+        for part in self._parts():
+            part.setup(rt, weights)
+        self.out_weights = [norm.weight * weights[self.scales[i]] if self.scales else norm.weight
+                            for i, norm in enumerate(self._norms())]
+        self._x = rt.shared("block.rows", rt.max_tokens, self.width)
+
+    def _close(self, stream: torch.Tensor, pending: Optional[PendingSum]) -> torch.Tensor:
+        """What is open goes into the stream; its rows in the compute dtype (in a float32 run the stream itself)."""
+        terms = [] if pending is None else pending.kernel_terms()
+        out = None if self.rt.dtype == torch.float32 else self._x[: stream.shape[0]]
+        if terms or out is not None:
+            ops.sum_norm(stream, terms, 0.0 if pending is None else pending.eps, None, out, 0.0)
+        return stream if out is None else out
+
+    def _open(self, which: int, y) -> PendingSum:
+        """A sub-layer's output behind its norm and scale."""
+        delta, bias = (y.delta, y.bias) if isinstance(y, PendingTerm) else (y, None)
+        return PendingSum((PendingTerm(delta, self.out_weights[which], bias=bias),), self._norms()[which].eps)
+
+    def forward(self, stream: torch.Tensor, pending, ctx: StepContext, cache_id: Optional[int],
+                write_cache: bool) -> PendingSum:
+        if pending is not None and not isinstance(pending, PendingSum):
+            pending = PendingSum.of(pending)
+        if self.mixer.reads_stream:
+            y = self.mixer.forward_stream(stream, pending, ctx, cache_id, write_cache)
+        else:
+            y = self.mixer.forward(self._close(stream, pending), ctx, cache_id, write_cache)
+        pending = self._open(0, y)
+        if self.feed_forward is None:
+            return pending
+        return self._open(1, self.feed_forward.forward(self._close(stream, pending)))

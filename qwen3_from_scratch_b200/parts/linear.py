@@ -11,7 +11,7 @@ product even in a bfloat16 run.
 
 from __future__ import annotations
 
-from typing import Optional
+from typing import Optional, Sequence
 
 import torch
 
@@ -109,4 +109,47 @@ class Linear:
             return wide
         out = self._out[:rows]
         out.copy_(wide)
+        return out
+
+
+class GroupedLinear:
+    """Several projections with inputs of their own (each ``[T, in_features]``) and one output ``[T, sum of rows]``, the
+    projections' results side by side.  With up to 16 rows in bfloat16 (and projections of equal sizes in multiples of 16
+    rows) one launch streams all the weights; otherwise a product per projection stores into its columns."""
+
+    def __init__(self, weights: Sequence[torch.Tensor], rt: Runtime, tag: str):
+        self.rows = [w.shape[0] for w in weights]
+        self.in_features = weights[0].shape[1]
+        if any(w.dim() != 2 or w.shape[1] != self.in_features for w in weights):
+            raise ValueError(f"projections side by side read rows of one width, got {[tuple(w.shape) for w in weights]}")
+        self.full_precision = any(w.dtype == torch.float32 for w in weights)
+        dtype = torch.float32 if self.full_precision else weights[0].dtype
+        self.weight = torch.cat([w.to(dtype) for w in weights], dim=0).contiguous()
+        self.out_features = sum(self.rows)
+        self.out_dtype = rt.dtype
+        self._out = rt.shared(f"{tag}.out", rt.max_tokens, self.out_features, dtype=rt.dtype)
+        self._out32 = self._out
+        if self.full_precision and rt.dtype != torch.float32:
+            self._out32 = rt.shared(f"{tag}.out32", rt.max_tokens, self.out_features, dtype=torch.float32)
+        self.one_launch = len(set(self.rows)) == 1 and self.rows[0] % 16 == 0
+
+    def __call__(self, x: torch.Tensor) -> torch.Tensor:
+        """``x``: [projections, T, in_features], contiguous."""
+        n, T, K = x.shape
+        if n != len(self.rows) or K != self.in_features:
+            raise ValueError(f"{len(self.rows)} projections of rows of {self.in_features} values, got {tuple(x.shape)}")
+        out = self._out[:T]
+        if self.one_launch and ops.gemm_skinny_takes(T, self.weight) and x.dtype == torch.bfloat16:
+            ops.gemm_skinny_groups(x, self.weight, out)
+            return out
+        wide, at = self._out32[:T], 0
+        for i, rows in enumerate(self.rows):
+            w, y = self.weight[at:at + rows], wide[:, at:at + rows]
+            if self.full_precision:
+                ops.gemm_f32_nt(x[i].float(), w, y)
+            else:
+                torch.mm(x[i], w.t(), out=y)
+            at += rows
+        if wide is not out and self.full_precision and self.out_dtype != torch.float32:
+            out.copy_(wide)
         return out

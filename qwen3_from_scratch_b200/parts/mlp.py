@@ -1,6 +1,7 @@
-"""Gated feed-forward: y = (up(x) * act(gate(x))) W_down^T, no biases.  ``swiglu`` is the form with the SiLU
+"""Gated feed-forward: y = (up(x) * act(gate(x))) W_down^T.  ``swiglu`` is the form with the SiLU
 gate and the checkpoint's ``gate_proj`` / ``up_proj`` / ``down_proj`` names; ``gated_mlp`` takes the gate's
-activation (``silu``, ``relu``, ``gelu_tanh``) and the tensors' names as parameters.
+activation (``silu``, ``relu``, ``gelu_tanh``, ``limited``), the tensors' names and whether the projections have biases
+as parameters.
 
 Reference: models/feedback.py:14-34.  The gate and up weights are merged into one [2I, H] weight at load, so
 one product feeds the gate kernel.
@@ -14,10 +15,11 @@ import torch
 
 from ..kernels import ops
 from ..registry import create_part, register_part
-from .base import FeedForward, PartSpec, Runtime, StreamNorm, WeightSpec
+from .base import FeedForward, PartSpec, PendingTerm, Runtime, StreamNorm, WeightSpec
 from .linear import Linear
 
-_DEFAULT_NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
+_DEFAULT_NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight",
+                  "gate_bias": "gate_proj.bias", "up_bias": "up_proj.bias", "down_bias": "down_proj.bias"}
 
 
 @register_part("feed_forward", "gated_mlp")
@@ -25,9 +27,15 @@ class GatedMLP(FeedForward):
     graph_capturable = True
 
     def __init__(self, name: str, hidden_size: int, intermediate_size: int, activation: str = "silu",
-                 names: Optional[Dict[str, str]] = None):
-        """``names``: what follows the part's name (and a dot) in the names of its gate, up and down tensors."""
+                 names: Optional[Dict[str, str]] = None, bias: bool = False, limit: float = 0.0):
+        """``names``: what follows the part's name (and a dot) in the names of its gate, up and down tensors.  ``bias``: all
+        three projections have one; the last one is left open (``forward`` returns a ``PendingTerm``).  The activation
+        ``limited`` takes gate and up value together, both held back by ``limit`` (the gate from above only):
+        g sigmoid(1.702 g) (u + 1)."""
         super().__init__(name)
+        self.has_bias, self.limit = bool(bias), float(limit)
+        if activation == "limited" and self.limit <= 0:
+            raise ValueError(f"feed-forward {name}: the limit must be positive, got {self.limit}")
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         ops.activation_code(activation, gate=True)
         self.activation = activation
@@ -37,9 +45,12 @@ class GatedMLP(FeedForward):
 
     def weight_specs(self) -> List[WeightSpec]:
         h, i = self.hidden_size, self.intermediate_size
-        return [WeightSpec(self.tensors["gate"], (i, h)),
-                WeightSpec(self.tensors["up"], (i, h)),
-                WeightSpec(self.tensors["down"], (h, i))]
+        specs = [WeightSpec(self.tensors["gate"], (i, h)),
+                 WeightSpec(self.tensors["up"], (i, h)),
+                 WeightSpec(self.tensors["down"], (h, i))]
+        if self.has_bias:
+            specs += [WeightSpec(self.tensors[f"{k}_bias"], (n,), kind="vector") for k, n in (("gate", i), ("up", i), ("down", h))]
+        return specs
 
     def setup(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
         super().setup(rt, weights)
@@ -55,6 +66,14 @@ class GatedMLP(FeedForward):
         else:
             merged = torch.cat([gate.to(dtype), up.to(dtype)], dim=0)
         del gate, up
+        self.gate_up_bias = self.down_bias = None
+        if self.has_bias:  # in the order of the merged rows
+            gb, ub = weights[self.tensors["gate_bias"]], weights[self.tensors["up_bias"]]
+            if self.blocks_of_eight:
+                self.gate_up_bias = torch.cat([gb.view(-1, 8), ub.view(-1, 8)], dim=1).reshape(-1).contiguous()
+            else:
+                self.gate_up_bias = torch.cat([gb, ub]).contiguous()
+            self.down_bias = weights[self.tensors["down_bias"]]
         self.gate_up = Linear(merged, rt, tag="ffn.gate_up")
         self.down = Linear(weights.pop(self.tensors["down"]), rt, tag="ffn.down")
         self._act = rt.shared("ffn.act", rt.max_tokens, self.intermediate_size)
@@ -65,7 +84,7 @@ class GatedMLP(FeedForward):
     fuses_stream = True
 
     def can_fuse_stream(self, rows: int) -> bool:
-        return (self.fused_gate and self.activation == "silu" and self.gate_up.takes_stream_norm(rows)
+        return (self.fused_gate and not self.has_bias and self.activation == "silu" and self.gate_up.takes_stream_norm(rows)
                 and self.down.can_add_into_stream(rows))
 
     def forward(self, x, into_stream=None, next_norm_weight=None):
@@ -76,18 +95,22 @@ class GatedMLP(FeedForward):
             ops.gemm_skinny_normed(x.scaled, x.sumsq, x.parts, x.eps, self.gate_up.weight, act, swiglu_blocks=True)
         elif self.fused_gate and ops.gemm_skinny_takes(rows, self.gate_up.weight):
             # decoding: stream the weight once, activation applied before the store
-            ops.gemm_skinny(x, self.gate_up.weight, act, swiglu_blocks=True, activation=self.activation)
-        elif (self.fused_gate and self.activation in ops.GEMM_TC_GATES
+            ops.gemm_skinny(x, self.gate_up.weight, act, swiglu_blocks=True, activation=self.activation,
+                            bias=self.gate_up_bias, limit=self.limit)
+        elif (self.fused_gate and ops.gemm_tc_gate_takes(self.activation, self.has_bias)
               and ops.gemm_tc_swiglu_pays(rows, self.gate_up.weight) and ops.gemm_tc_takes(x, self.gate_up.weight)):
             # prompt portions: the engine's tcgen05 product with the activation in its epilogue, so the
             # [T, 2I] gate/up product never goes to memory
             ops.gemm_tc(x, self.gate_up.weight, act, self.rt.status, swiglu_blocks=True,
-                        pair=ops.gemm_tc_swiglu_pays(rows, self.gate_up.weight) == "pair", activation=self.activation)
+                        pair=ops.gemm_tc_swiglu_pays(rows, self.gate_up.weight) == "pair", activation=self.activation,
+                        bias=self.gate_up_bias, limit=self.limit)
         else:
-            ops.gated_act(self.gate_up(x), act, interleave8=self.blocks_of_eight, activation=self.activation)
+            ops.gated_act(self.gate_up(x), act, interleave8=self.blocks_of_eight, activation=self.activation,
+                          bias=self.gate_up_bias, limit=self.limit)
         if into_stream is not None:
             return self.down.into_stream(act, into_stream, next_norm_weight)
-        return self.down(act)
+        y = self.down(act)
+        return y if self.down_bias is None else PendingTerm(y, bias=self.down_bias)
 
 
 @register_part("feed_forward", "swiglu")
@@ -150,22 +173,31 @@ class RoutedExperts(FeedForward):
 
     ``score="softmax"``: s = softmax(W_router h) over all experts.  ``groups`` = (count, keep): the experts form ``count`` equal
     groups of neighbours, a group's score is the largest in it, and only experts of the ``keep`` best groups can be chosen.
-    ``renormalise``: the chosen experts' s are divided by their sum (+ 1e-20).
+    ``renormalise``: the chosen experts' s are divided by their sum (+ 1e-20).  ``router_bias``: a bias of the logits, the
+    tensor ``<name>.<router_bias>`` [E], added before anything else.  ``activation="limited"`` (gated experts): see
+    ``GatedMLP``, with ``limit``.
 
     The correction takes part in the choice only.  ``shared``: a feed-forward
-    (any registered one) that every token goes through, added to the sum, or None.  Tensors: ``<name>.<router>``
+    (any registered one) that every token goes through, added to the sum, or None; with ``shared_gate`` it is multiplied by
+    sigmoid(W_sg h), one number per token (``<name>.<shared>.<shared_gate>`` [1, width]).  Tensors: ``<name>.<router>``
     [E, width], ``<name>.<correction>`` [E] (absent with ``correction=False``), ``<name>.<expert><e>.<up>`` [ff, width]
     and ``.<down>`` [width, ff], and the shared part's under ``<name>.<shared>``."""
 
     graph_capturable = True
     NAMES = {"router": "router", "correction": "correction", "expert": "e", "up": "up", "down": "down", "gate": "gate",
-             "shared": "shared"}
+             "shared": "shared", "router_bias": "router.b", "shared_gate": "sg"}
 
     def __init__(self, name: str, hidden_size: int, experts: int, top: int, expert_ff: int, router_scale: float = 1.0,
                  activation: str = "relu_sq", correction: bool = True, shared: Optional[PartSpec] = None,
                  names: Optional[Dict[str, str]] = None, gated: bool = False, weigh: str = "output",
-                 score: str = "sigmoid", groups: Optional[Tuple[int, int]] = None, renormalise: bool = False):
+                 score: str = "sigmoid", groups: Optional[Tuple[int, int]] = None, renormalise: bool = False,
+                 limit: float = 0.0, router_bias: bool = False, shared_gate: bool = False):
         super().__init__(name)
+        self.limit, self.has_router_bias, self.has_shared_gate = float(limit), bool(router_bias), bool(shared_gate)
+        if activation == "limited" and (not gated or self.limit <= 0):
+            raise ValueError(f"feed-forward {name}: limited experts are gated and have a positive limit, got {self.limit}")
+        if self.has_shared_gate and shared is None:
+            raise ValueError(f"feed-forward {name}: a gate of the shared expert needs a shared expert")
         if score not in ops.MOE_SCORES:
             raise ValueError(f"feed-forward {name}: scores are made by {' or '.join(ops.MOE_SCORES)}, got {score!r}")
         self.score, self.renormalise = score, bool(renormalise)
@@ -187,6 +219,10 @@ class RoutedExperts(FeedForward):
         self.n = n
         self.shared = None if shared is None else create_part("feed_forward", shared, name=f"{name}.{n['shared']}")
 
+    @property
+    def _shared_gate(self) -> str:
+        return f"{self.name}.{self.n['shared']}.{self.n['shared_gate']}"
+
     def _expert(self, e: int, which: str) -> str:
         return f"{self.name}.{self.n['expert']}{e}.{self.n[which]}"
 
@@ -195,6 +231,10 @@ class RoutedExperts(FeedForward):
         specs = [WeightSpec(f"{self.name}.{self.n['router']}", (self.experts, w), kind="vector", init="normal")]
         if self.has_correction:
             specs.append(WeightSpec(f"{self.name}.{self.n['correction']}", (self.experts,), kind="vector", init="normal"))
+        if self.has_router_bias:
+            specs.append(WeightSpec(f"{self.name}.{self.n['router_bias']}", (self.experts,), kind="vector", init="normal"))
+        if self.has_shared_gate:
+            specs.append(WeightSpec(self._shared_gate, (1, w), kind="vector", init="normal"))
         for e in range(self.experts):
             if self.gated:
                 specs.append(WeightSpec(self._expert(e, "gate"), (f, w)))
@@ -205,6 +245,9 @@ class RoutedExperts(FeedForward):
         super().setup(rt, weights)
         self.router = weights[f"{self.name}.{self.n['router']}"]
         self.correction = weights[f"{self.name}.{self.n['correction']}"] if self.has_correction else None
+        self.router_bias = weights[f"{self.name}.{self.n['router_bias']}"] if self.has_router_bias else None
+        if self.has_shared_gate:  # one more row of the router's matrix
+            self.router = torch.cat([self.router, weights[self._shared_gate]], dim=0).contiguous()
         # the experts' matrices in two stacks, in the compute dtype: up [E, ff, width], down [E, width, ff]
         self.gate_block = ops.moe_gate_block(self.expert_ff) if self.gated else 0
         if self.gated:
@@ -222,6 +265,7 @@ class RoutedExperts(FeedForward):
         T = rt.max_tokens
         self._ids = rt.shared("moe.ids", T, self.top, dtype=torch.int32)
         self._weights = rt.shared("moe.weights", T, self.top, dtype=torch.float32)
+        self._share = rt.shared("moe.share", T, dtype=torch.float32) if self.has_shared_gate else None
         self._act = rt.shared("moe.act", T * self.top, self.expert_ff)
         self._out = rt.shared("moe.out", T, self.hidden_size)
         self._status = rt.status
@@ -234,11 +278,13 @@ class RoutedExperts(FeedForward):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         T = x.shape[0]
         ids, wts = self._ids[:T], self._weights[:T]
+        share = None if self._share is None else self._share[:T]
         ops.moe_route(x, self.router, self.correction, ids, wts, self.router_scale, self.score, self.groups, self.keep,
-                      self.renormalise)
+                      self.renormalise, logit_bias=self.router_bias, share=share)
         base = self.shared.forward(x) if self.shared is not None else None
         out = self._out[:T]
         ops.routed_experts(x, self.up, self.down, ids, self._ones[:T] if self.weigh_input else wts, base,
                            self._act[: T * self.top], out, self.activation, scratch=self._grouped, status=self._status,
-                           gate_block=self.gate_block, in_weights=wts if self.weigh_input else None)
+                           gate_block=self.gate_block, in_weights=wts if self.weigh_input else None, base_weights=share,
+                           limit=self.limit)
         return out

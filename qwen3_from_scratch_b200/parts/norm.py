@@ -53,7 +53,7 @@ class RMSNorm(Norm):
 
     @staticmethod
     def _terms(pending: Optional[PendingSum]):
-        return [] if pending is None else [(t.delta, t.weight, t.scale) for t in pending.terms]
+        return [] if pending is None else pending.kernel_terms()
 
     def add_norm_pair(self, stream: torch.Tensor, pending, other: "RMSNorm"):
         """This norm and ``other`` (with the same epsilon) of the same rows, in one pass: (this one's output, the other's)."""

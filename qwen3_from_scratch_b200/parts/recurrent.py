@@ -15,6 +15,7 @@
                     (see the class).
 ``decayed_memory``  a matrix memory with a fixed decay per head and no softmax (retention, lightning attention).
 ``gated_delta``     a matrix memory with the gated delta rule.
+``time_mixing``     a matrix memory with a decay per key channel, each operand from a mix of a token with the one before.
 
 The first two keep two things per request, named in ``cache_spec()``: ``state`` (float32) and ``conv`` (the last
 taps - 1 inputs of the short convolution, float32).  A new request's slot is zero.  The projections are
@@ -31,8 +32,8 @@ import torch
 
 from ..kernels import ops
 from ..registry import create_part, register_part
-from .base import Mixer, PartSpec, Runtime, StateSpec, StepContext, WeightSpec
-from .linear import Linear
+from .base import Mixer, PartSpec, PendingSum, Runtime, StateSpec, StepContext, WeightSpec
+from .linear import GroupedLinear, Linear
 
 
 class _NamedTensors:
@@ -618,3 +619,98 @@ class GatedDelta(Mixer, _NamedTensors):
                         self._scratch)
         ops.memory_out(o, proj, g_col, self.norm_weight, self.norm_eps, "silu", gated, H)
         return self.out_proj(gated)
+
+
+@register_part("mixer", "time_mixing")
+class TimeMixing(Mixer, _NamedTensors):
+    """The time mixing of RWKV-6 (Peng et al., "Eagle and Finch: RWKV with Matrix-Valued States and Dynamic Recurrence"), with
+    one learned mix per operand.  With h the input, h' the input of the token before (zeros for the first), H heads of ``dim``:
+
+        m_s = h + (h' - h) mu_s                                             for s in r, k, v, g, w
+        r = W_r m_r;  k = W_k m_k;  v = W_v m_v
+        logw = -exp(W_w2 tanh(W_w1 m_w) + w0)                               (per head and key channel)
+        o = (S + diag(u) k v^T)^T r;   S <- diag(exp(logw)) S + k v^T       (per head: the token itself with the bonus u)
+        out = W_o (unit_rms_per_head(o) * norm * silu(W_g m_g))
+
+    The rank of the decay's projection is what the stored W_w1 and W_w2 say (``rank`` only sizes random weights).  Per request
+    it keeps ``state`` (S value by value, float32) and ``shift`` (the last h, float32); a new request's slots are zero.  The
+    mixes, everything about the decays, the state and the norm are float32 in every run; only the operands of the
+    projections are rounded to the compute dtype.  ``names``: the tensors' names after the part's own."""
+
+    graph_capturable = True
+    reads_stream = True
+    MIXES = ("r", "k", "v", "g", "w")
+    NAMES = {"mu_r": "mu.r", "mu_k": "mu.k", "mu_v": "mu.v", "mu_g": "mu.g", "mu_w": "mu.w", "r": "r", "k": "k", "v": "v",
+             "g": "g", "w1": "w1", "w2": "w2", "w0": "w0", "u": "u", "norm": "norm", "out": "o"}
+
+    def __init__(self, name: str, hidden_size: int, num_heads: int, dim: int, norm_eps: float, rank: int = 32,
+                 names: Optional[Dict[str, str]] = None):
+        super().__init__(name)
+        self.hidden_size, self.num_heads, self.dim, self.norm_eps = int(hidden_size), int(num_heads), int(dim), float(norm_eps)
+        self.rank = int(rank)
+        self._name_tensors(name, self.NAMES, names)
+
+    def weight_specs(self) -> List[WeightSpec]:
+        t, w, n = self.tensors, self.hidden_size, self.num_heads * self.dim
+        return [WeightSpec(t[f"mu_{s}"], (w,), kind="vector", init="normal") for s in self.MIXES] + [
+            WeightSpec(t[s], (n, w)) for s in "rkvg"] + [
+            WeightSpec(t["w1"], (self.rank, w), free_dims=(0,)),
+            WeightSpec(t["w2"], (n, self.rank), kind="vector", init="normal", free_dims=(1,)),
+            WeightSpec(t["w0"], (n,), kind="vector", init="normal"),
+            WeightSpec(t["u"], (self.num_heads, self.dim), kind="vector", init="normal"),
+            WeightSpec(t["norm"], (n,), kind="vector", init="one_plus_normal"),
+            WeightSpec(t["out"], (w, n))]
+
+    def cache_spec(self):
+        return {"state": StateSpec((self.num_heads, self.dim, self.dim), "float32"),
+                "shift": StateSpec((self.hidden_size,), "float32")}
+
+    def setup(self, rt: Runtime, weights: Dict[str, torch.Tensor]) -> None:
+        super().setup(rt, weights)
+        if self.dim > ops.memory_max_dim():
+            raise ValueError(f"mixer {self.name}: keys of {self.dim} values exceed the {ops.memory_max_dim()} the scan takes")
+        t, n, T = self.tensors, self.num_heads * self.dim, rt.max_tokens
+        self.mu = torch.stack([weights[t[f"mu_{s}"]] for s in self.MIXES]).contiguous()
+        self.proj = GroupedLinear([weights.pop(t[s]) for s in "rkvg"], rt, tag="tmix.proj")  # columns: r, k, v, g
+        w1 = weights.pop(t["w1"])
+        self.w2, self.w0 = weights[t["w2"]], weights[t["w0"]]
+        if w1.shape[0] != self.w2.shape[1]:
+            raise ValueError(f"mixer {self.name}: {t['w1']} leaves {w1.shape[0]} values, {t['w2']} reads {self.w2.shape[1]}")
+        self.low = Linear(_stack_rows([w1]), rt, tag="tmix.low", out_dtype=torch.float32)
+        self.bonus, self.norm_weight = weights[t["u"]], weights[t["norm"]]
+        self.out_proj = Linear(weights.pop(t["out"]), rt, tag="tmix.out")
+        self._mix = rt.shared("tmix.mix", len(self.MIXES) * T * self.hidden_size)
+        self._x32 = None
+        self._logw = rt.shared("tmix.logw", T, n, dtype=torch.float32)
+        self._o = rt.shared("memory.o", T, n, dtype=torch.float32)
+        self._gated = rt.shared("tmix.gated", T, n)
+        self._scratch = None
+        if ops.channel_matrix_form(rt.dtype, self.dim, self.dim) and T >= ops.MEMORY_CHUNKED_FROM:
+            self._scratch = ops.ChannelScratch(rt.shared, T, rt.max_seqs, self.num_heads, self.dim)
+
+    def forward_stream(self, stream: torch.Tensor, pending: Optional[PendingSum], ctx: StepContext, cache_id: Optional[int],
+                       write_cache: bool) -> torch.Tensor:
+        T, W = stream.shape
+        terms = [] if pending is None else pending.kernel_terms()
+        eps = 0.0 if pending is None else pending.eps
+        if terms and (len(terms) > 1 or ctx.max_q_len > 1):  # a portion's rows are read by their neighbours: close them first
+            ops.sum_norm(stream, terms, eps, None, None, 0.0)
+            terms = []
+        mix = self._mix[: len(self.MIXES) * T * W].view(len(self.MIXES), T, W)
+        ops.sum_mix(stream, terms[0] if terms else None, eps, self.mu, ctx.state(cache_id, "shift"), ctx.q_start, ctx.tok_seq,
+                    ctx.slot_ids, ctx.num_seqs, mix, self.rt.status)
+        n = self.num_heads * self.dim
+        proj = self.proj(mix[:4])
+        logw, o, gated = self._logw[:T], self._o[:T], self._gated[:T]
+        ops.low_rank_decay(self.low(mix[4]), self.w2, self.w0, logw)
+        ops.channel_memory_scan(proj, 0, n, 2 * n, ops.ChannelDecay(logw, self.bonus), ctx.state(cache_id, "state"), ctx.q_start,
+                                ctx.slot_ids, ctx.num_seqs, o, self.rt.status, ctx.max_q_len, self._scratch)
+        ops.memory_out(o, proj, 3 * n, self.norm_weight, self.norm_eps, "silu", gated, self.num_heads)
+        return self.out_proj(gated)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache_id: Optional[int], write_cache: bool) -> torch.Tensor:
+        if self._x32 is None:
+            self._x32 = self.rt.shared("tmix.x32", self.rt.max_tokens, self.hidden_size, dtype=torch.float32)
+        stream = self._x32[: x.shape[0]]
+        stream.copy_(x)
+        return self.forward_stream(stream, None, ctx, cache_id, write_cache)

@@ -105,3 +105,27 @@ class RotaryStretched(PositionEncoding):
     def frequencies(self) -> Tuple[torch.Tensor, float, int]:
         """(float32 frequencies [dims / 2] on the device, magnitude, dims)."""
         return self.freq, self.magnitude, self.dims
+
+
+@register_part("position", "rotary_banded")
+class RotaryBanded(RotaryStretched):
+    """Rotate-half rotation whose frequencies are stretched by wavelength, in the manner of Llama 3.1: with
+    f_i = base^(-2i / dims) and n_i = original * f_i / (2 pi), the turns that pair i makes within the ``original`` context,
+
+        freq_i = f_i                                  where n_i > high
+        freq_i = f_i / factor                         where n_i < low
+        freq_i = (1 - s) f_i / factor + s f_i         between, s = (n_i - low) / (high - low)
+
+    The frequencies are evaluated in float64 on the host and kept in float32 (see ``RotaryStretched``)."""
+
+    def __init__(self, name: str, dims: int, base: float, scaling: Optional[dict] = None):
+        super().__init__(name, dims, base)
+        if scaling:
+            factor, original = float(scaling["factor"]), float(scaling["original"])
+            low, high = float(scaling["low"]), float(scaling["high"])
+            if not (factor > 0 and original > 0 and high > low):
+                raise ValueError(f"rotation {name}: scaling needs a positive factor and context and high above low, got {scaling}")
+            for i, f in enumerate(self._freq):
+                s = (original * f / (2.0 * math.pi) - low) / (high - low)
+                s = min(max(s, 0.0), 1.0)
+                self._freq[i] = (1.0 - s) * f / factor + s * f
