@@ -1,5 +1,5 @@
-"""``bench.py --arch binupel|bikadra|dogidra|zasalix|domelix``: another design beside Qwen3 (Zasalix: beside Dogidra,
-Domelix: beside Zasalix, the closest of the other designs) at equal layer sizes (random weights drawn on
+"""``bench.py --arch binupel|bikadra|dogidra|zasalix|domelix|zasitar``: another design beside Qwen3 (Zasalix: beside Dogidra,
+Domelix: beside Zasalix, Zasitar: beside Domelix, the closest of the other designs) at equal layer sizes (random weights drawn on
 the device): a prompt step of 2,048 tokens and decode steps at two batch sizes, each replayed on the device
 between CUDA events, and every kernel of one eagerly launched step timed by events of its own, with the bytes
 or flops it must move and the fraction of the measured copy bandwidth or bf16 throughput that this makes.
@@ -11,7 +11,8 @@ and a span of two layers twice; a Zasalix model repeats the pattern latent atten
 attention that keeps the first tokens beside a matrix memory with routed gated experts, a matrix memory alone with
 routed gated experts, the last two as a span that runs twice; a Domelix model repeats the pattern full attention with a
 distance bias beside lightning attention, the gated delta rule, retention, each with routed gated experts chosen within
-groups; the Qwen3 model has as many layer runs of the same width, heads, head size and
+groups; a Zasitar model repeats the pattern time mixing with routed limited experts and a shared one, windowed attention with
+a dense feed-forward, windowed attention on the keys of the layer before with routed experts; the Qwen3 model has as many layer runs of the same width, heads, head size and
 (active) feed-forward width.
 """
 
@@ -123,6 +124,28 @@ def domelix_config(s):
     pattern = [par, delta, ret]
     return {"architecture": "Domelix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
             "layers": [pattern[i % 3] for i in range(s["layers"])]}
+
+
+def zasitar_config(s):
+    """Time mixing with heads of 64 over the width; attention over 1,024 tokens (heads as the other models', half of each
+    rotated), and a layer that reads its keys and values; 16 experts of a quarter of the dense width, three per token, and a
+    shared one of the same width, or the dense feed-forward."""
+    moe = {"kind": "moe", "expert": {"ff": s["ff"] // 4, "limit": 7.0}, "router": {"experts": 16, "top": 3},
+           "shared": {"ff": s["ff"] // 4, "limit": 7.0}}
+    dense = {"kind": "dense", "ff": s["ff"]}
+
+    def att(mlp, **more):
+        return {"type": "attention", "mlp": mlp,
+                "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+                          "mask": {"size": 1024},
+                          "rot": {"base": 500000.0, "dims": s["dim"] // 2,
+                                  "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}, **more}}
+
+    layers = []
+    for i in range(s["layers"]):
+        layers.append([{"type": "wkv", "mixer": {"heads": s["width"] // 64, "dim": 64}, "mlp": moe}, att(dense),
+                       att(moe, kv_from=i - 1)][i % 3])
+    return {"architecture": "Zasitar", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "layers": layers}
 
 
 def qwen3_config(s):
@@ -270,7 +293,24 @@ class KernelClock:
         if name == "sum_norm":
             stream, terms, out = a[0], a[1], a[4]
             n = size(stream) * (2 if terms and k.get("rows") is None else 1) + sum(size(t[0]) for t in terms)
-            return "bytes", n + size(out) * (2 if k.get("second") is not None else 1)
+            return "bytes", n + (size(out) if out is not None else 0) * (2 if k.get("second") is not None else 1)
+        if name == "sum_mix":
+            stream, term, mix = a[0], a[1], a[9]
+            return "bytes", size(stream) * (2 if term is not None else 1) + (size(term[0]) if term is not None else 0) + size(mix)
+        if name == "channel_memory_scan":
+            # q, k, v, the log-decays and the result once, and the state in and out
+            x, rule, state, out = a[0], a[4], a[5], a[9]
+            H, Dv, D = state.shape[1], state.shape[2], state.shape[3]
+            seqs = 1 if sc["kind"] == "prefill" else sc["batch"]
+            return "bytes", x.shape[0] * H * (2 * D + Dv) * x.element_size() + size(rule.logw) + size(out) + 2 * seqs * H * D * Dv * 4
+        if name == "low_rank_decay":
+            return "bytes", size(a[0]) + size(a[1]) + size(a[3])
+        if name == "gemm_skinny_groups":
+            return "bytes", size(a[1])
+        if name == "head_qkv_post":
+            proj, has_kv, heads, kv_heads, dim, vdim = a[0], a[2] is not None, a[4], a[5], a[6], a[7]
+            n = proj.shape[0] * proj.element_size()
+            return "bytes", 2 * n * (heads * dim + (kv_heads * (dim + vdim) if has_kv else 0))
         if name == "mlstm_out":
             o, out = a[0], a[5]
             return "bytes", size(o) + 2 * out.numel() * out.element_size()
@@ -321,6 +361,12 @@ class KernelClock:
             if sc["kind"] == "prefill":
                 return "flops", 2 * H * (D + Dv) * sum(seen(i) for i in range(sc["tokens"]))
             return "bytes", sc["batch"] * seen(sc["context"] - 1) * G * (D + Dv) * k_pages.element_size() + 2 * size(q)
+        if name == "window_attention":
+            q, k_pages, window = a[0], a[1], a[6]
+            if sc["kind"] == "prefill":
+                return "flops", 4 * q.shape[1] * q.shape[2] * sum(min(i + 1, window) for i in range(sc["tokens"]))
+            row = 2 * k_pages.shape[1] * k_pages.shape[3] * k_pages.element_size()
+            return "bytes", sc["batch"] * min(sc["context"], window) * row + 2 * size(q)
         if name == "mingru_scan":
             out = a[10]
             return "bytes", 4 * out.numel() * out.element_size()
@@ -361,7 +407,8 @@ class KernelClock:
                      "latent_q_post", "gate_heads", "latent_attention", "ssd_scan", "gated_group_norm", "add_layernorm",
                      "add_layernorm_conv1", "input_conv", "stream_concat", "pw_qkv_post", "pool_blocks", "pooled_window_attention",
                      "mingru_scan", "moe_route", "routed_experts", "add_dyt", "add_unit_rms", "side_gate", "sigmoid_gate",
-                     "mlstm_scan", "mlstm_out", "memory_scan", "memory_out", "rotate_columns", "sum_norm"):
+                     "mlstm_scan", "mlstm_out", "memory_scan", "memory_out", "rotate_columns", "sum_norm",
+                     "sum_mix", "channel_memory_scan", "low_rank_decay", "gemm_skinny_groups", "head_qkv_post", "window_attention"):
             self.wrap(ops, name, name)
         real_mm = torch.mm
         clock = self
@@ -376,6 +423,21 @@ class KernelClock:
 
         self.saved.append((torch, "mm", real_mm))
         torch.mm = mm
+        real_bmm = torch.bmm
+
+        def bmm(x, wt, **k):
+            start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            start.record()
+            out = real_bmm(x, wt, **k)
+            end.record()
+            w = wt.transpose(1, 2)
+            rows, columns = x.shape[1], w.reshape(-1, w.shape[2])
+            clock.pending.append(("library product", start, end,
+                                  clock.work("library product", (x.new_empty(rows, 0), columns), {})))
+            return out
+
+        self.saved.append((torch, "bmm", real_bmm))
+        torch.bmm = bmm
         return self
 
     def __exit__(self, *exc):
@@ -449,11 +511,11 @@ def compare(args, peaks, sample_clocks):
     sampler = sample_clocks()
     t0 = time.time()
     other = {"binupel": binupel_config, "bikadra": bikadra_config, "dogidra": dogidra_config,
-             "zasalix": zasalix_config, "domelix": domelix_config}[args.arch]
-    # what the design stands beside: Qwen3, or for Zasalix and Domelix the closest of the other designs (a windowed
-    # attention beside a recurrence, routed experts; an attention beside a matrix memory, matrix memories alone, gated experts)
-    beside, beside_config = {"zasalix": ("dogidra", dogidra_config),
-                             "domelix": ("zasalix", zasalix_config)}.get(args.arch, ("qwen3", qwen3_config))
+             "zasalix": zasalix_config, "domelix": domelix_config, "zasitar": zasitar_config}[args.arch]
+    # what the design stands beside: Qwen3, or for the last three the closest of the other designs (a windowed attention
+    # beside a recurrence, routed experts; an attention beside a matrix memory, matrix memories alone, gated experts)
+    beside, beside_config = {"zasalix": ("dogidra", dogidra_config), "domelix": ("zasalix", zasalix_config),
+                             "zasitar": ("domelix", domelix_config)}.get(args.arch, ("qwen3", qwen3_config))
     out = {"arch": args.arch, "beside": beside, "sizes": dict(size, name=args.arch_size), "dtype": "bf16",
            "data": "synthetic tokens, random weights drawn on the device", "steps": args.steps, "warmup": args.warmup,
            "peaks": peaks, "timing": "CUDA events around each replay of the step; 256 MB written between replays",

@@ -106,6 +106,7 @@ struct DecodeQkv {
   __nv_bfloat16* v_pages;
   int write_kv;              // 0: another layer wrote this cache; only the query is made
   int angles_early;          // cos_sin is older than the launch before this one
+  const float* sink;         // float32 [Hq]: exp(sink) joins the denominator; or null
 };
 
 // BLOCKS: blocks per SM the kernel is compiled for.  Three (128 registers) give a large grid half as many
@@ -450,6 +451,13 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       }
     }
     const int head = hk * g + r;
+    if (fq.sink != nullptr && split == 0) {  // the sink: one more exponential in the denominator, in the first range's share
+      const float s2 = fq.sink[head] * 1.4426950408889634f, top = fmaxf(big, s2);
+      const float keep = big == -INFINITY ? 0.f : exp2f(big - top);
+      acc *= keep;
+      den = fmaf(den, keep, exp2f(s2 - top));
+      big = top;
+    }
     if (num_splits == 1) {
       out[((size_t)tq * Hq + head) * D + d] = __float2bfloat16_rn(den > 0.f ? acc / den : 0.f);
     } else {
@@ -527,6 +535,25 @@ extern "C" int q3_attn_decode_tma(const void* q, const void* k_pages, const void
   return q3::attn_decode_tma_launch<128>(q, k_pages, v_pages, out, partial, q_start, kv_len, block_table,
                                          table_stride, page_size, num_pages, B, Hq, Hkv, scale, window, num_splits,
                                          status, stream);
+}
+
+// The same with a sink (float32 [Hq]): exp(sink) joins the softmax's denominator.  The scale must be positive.
+extern "C" int q3_attn_decode_tma_sink(const void* q, const void* k_pages, const void* v_pages, void* out, float* partial,
+                                       const int* q_start, const int* kv_len, const int* block_table, int table_stride,
+                                       int page_size, int num_pages, int B, int Hq, int Hkv, int D, float scale, int window,
+                                       int num_splits, const float* sink, int* status, cudaStream_t stream) {
+  if (B <= 0) return 0;
+  if (Hkv <= 0 || Hq % Hkv || Hq / Hkv > 16 || (D != 64 && D != 128) || page_size <= 0 || page_size % 16 ||
+      num_splits < 1 || table_stride <= 0 || B > 65535 || Hkv > 65535 || !(scale > 0.f))
+    return Q3_ERR_SIZE;
+  if ((uintptr_t)q % 16 || (uintptr_t)k_pages % 16 || (uintptr_t)v_pages % 16) return Q3_ERR_ALIGN;
+  q3::DecodeQkv fq{};
+  fq.sink = sink;
+  if (D == 64)
+    return q3::attn_decode_tma_launch<64>(q, k_pages, v_pages, out, partial, q_start, kv_len, block_table, table_stride,
+                                          page_size, num_pages, B, Hq, Hkv, scale, window, num_splits, status, stream, fq);
+  return q3::attn_decode_tma_launch<128>(q, k_pages, v_pages, out, partial, q_start, kv_len, block_table, table_stride,
+                                         page_size, num_pages, B, Hq, Hkv, scale, window, num_splits, status, stream, fq);
 }
 
 // The same with the work of q3_qkv_post for a step in which every row brings one token (see DecodeQkv):

@@ -1,5 +1,6 @@
 // Paged causal attention for prompt portions on the fifth-generation tensor cores (tcgen05),
-// bfloat16, head size 64 or 128, pages of 8 to 64 tokens, no window.
+// bfloat16, head size 64 or 128, pages of 8 to 64 tokens; optionally over a sliding window and with a sink (a logit per head
+// in the denominator only).
 //
 // A block owns 128 query rows of one kv head (rows are (token, head-in-group) pairs as in
 // attn_prefill.cu) and walks the keys in tiles of 128:
@@ -59,14 +60,17 @@ __device__ __forceinline__ uint32_t sw128_offset(int row, int col) {
 // SIGMOID: the weights are not normalised over the keys (attn_sigmoid.cu): a visible key gets
 // sigmoid(s * scale + head_bias[h]), there is no maximum, no denominator and nothing to rescale, and the finished
 // row is multiplied by gate[t, h].  The "softmax" threads then only turn scores into weights.
-template <int D, bool SIGMOID = false>
+// WINDOW: a row at position p reads the keys n with p - window < n <= p, so a block's tiles start at the one that holds the
+// oldest key of its first row (pages wholly before that key may have been given back and are left out; their rows of V are
+// zeroed, as those past the end are), and exp(sink[h]) joins the finished row's denominator.
+template <int D, bool SIGMOID = false, bool WINDOW = false>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out,
                const int* __restrict__ q_start, const int* __restrict__ kv_len,
                const int* __restrict__ block_table, int table_stride, int page_size, int num_pages, int Hq,
                int Hkv, float scale_log2, int* status, const float* __restrict__ head_bias = nullptr,
-               const float* __restrict__ gate = nullptr) {
+               const float* __restrict__ gate = nullptr, int window = 0, const float* __restrict__ sink = nullptr) {
   using S = AttnTcShape<D>;
   constexpr int ATOMS = S::ATOMS;
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -105,7 +109,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
   }
   const int last_row = min(total_rows, row0 + AT_BM) - 1;
   const int pos_first = past + row0 / g, pos_last = past + last_row / g;
-  const int n_tiles = pos_last / AT_BN + 1;
+  const int lo_key = WINDOW ? max(0, pos_first - window + 1) : 0;  // the oldest key that any row reads
+  const int tile0 = lo_key / AT_BN;                                // tile j of the block is tile tile0 + j of the sequence
+  const int n_tiles = pos_last / AT_BN + 1 - tile0;
   const int* table = block_table + (size_t)b * table_stride;
 
   if (warp == AT_LOAD_WARP && lane == 0) tma_prefetch_map(&map_k);
@@ -185,9 +191,13 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
     uint64_t* full = is_v ? v_full : k_full;
     uint64_t* empty = is_v ? v_empty : k_empty;
     const int pages_per_tile = AT_BN / page_size;
+    auto has_page = [&](int j) {  // whether the lane has a page of tile j to bring in
+      const int first = (tile0 + j) * AT_BN + lane * page_size;
+      return lane < pages_per_tile && first < len && (!WINDOW || first + page_size > lo_key);
+    };
     auto page_id = [&](int j) -> int {  // lane's page of tile j, or -1 if the tile has no such page
-      if (lane >= pages_per_tile || j >= n_tiles || j * AT_BN + lane * page_size >= len) return -1;
-      return table_page(table, (j * AT_BN) / page_size + lane, table_stride, status);
+      if (j >= n_tiles || !has_page(j)) return -1;
+      return table_page(table, ((tile0 + j) * AT_BN) / page_size + lane, table_stride, status);
     };
     int page = page_id(0), page_next = page_id(1);
     bool ok = true;
@@ -195,7 +205,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
       const int st = j & 1;
       const uint32_t use = (uint32_t)j >> 1;
       const int page_after = page_id(j + 2);
-      const bool wanted = lane < pages_per_tile && j * AT_BN + lane * page_size < len;
+      const bool wanted = has_page(j);
       if (wanted && (page < 0 || page >= num_pages)) {
         if (!is_v) atomicOr(status, Q3_STATUS_BAD_PAGE);
         page = -1;
@@ -292,11 +302,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
       uint32_t sv[32];
       tmem_ld_32(tmem_s + st * AT_BN + part * AT_PART + lane_base, sv);
       tmem_wait_ld();
-      const int base_n = j * AT_BN + part * AT_PART;
+      const int tile_n = (tile0 + j) * AT_BN;  // the tile's first key
+      const int base_n = tile_n + part * AT_PART;
       if constexpr (SIGMOID) {
         // a thread's packed weights go where another thread's scores were: all scores are in registers first
         asm volatile("bar.sync 1, %0;" ::"n"(AT_SOFTMAX) : "memory");
-        const bool diagonal = j * AT_BN + AT_BN - 1 > pos_first;
+        const bool diagonal = tile_n + AT_BN - 1 > pos_first;
         uint32_t pk[16];
 #pragma unroll
         for (int e = 0; e < 16; ++e) {
@@ -313,10 +324,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
         tmem_wait_st();
       } else {
       float mx = -INFINITY;
-      if (j * AT_BN + AT_BN - 1 > pos_first) {  // the diagonal: keys beyond this row's position are hidden
+      // the diagonal: keys beyond this row's position are hidden; the window's start: keys before it
+      if (tile_n + AT_BN - 1 > pos_first || (WINDOW && tile_n < pos_last - window + 1)) {
 #pragma unroll
         for (int c = 0; c < 32; ++c) {
-          const float v = (base_n + c <= my_pos) ? __uint_as_float(sv[c]) : -INFINITY;
+          const bool seen = base_n + c <= my_pos && (!WINDOW || base_n + c > my_pos - window);
+          const float v = seen ? __uint_as_float(sv[c]) : -INFINITY;
           sv[c] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -369,9 +382,16 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
       l += sum;
       }  // softmax
       // keys past the end of the sequence in the last tile: their V rows were not loaded; zero them
-      if (j * AT_BN + AT_BN > len) {
+      if (WINDOW && j == 0 && lo_key - tile_n >= page_size) {  // and those of pages before the window
+        const int missing = (lo_key - tile_n) / page_size * page_size;
+        for (int e = soft_tid; e < missing * (D / 8); e += AT_SOFTMAX) {
+          const int key = e / (D / 8), c = e % (D / 8);
+          *reinterpret_cast<uint4*>(v_s + (c / 8) * (AT_BN * 128) + sw128_offset(key, (c % 8) * 8)) = make_uint4(0, 0, 0, 0);
+        }
+      }
+      if (tile_n + AT_BN > len) {
         ok = ok && mbar_wait(v_full + st, ((uint32_t)j >> 1) & 1, &abort_flag);
-        const int first_bad = len - j * AT_BN;
+        const int first_bad = len - tile_n;
         for (int e = soft_tid; e < (AT_BN - first_bad) * (D / 8); e += AT_SOFTMAX) {
           const int key = first_bad + e / (D / 8), c = e % (D / 8);
           *reinterpret_cast<uint4*>(v_s + st * S::V_BYTES + (c / 8) * (AT_BN * 128) + sw128_offset(key, (c % 8) * 8)) =
@@ -403,6 +423,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
       float total = 0.f;
 #pragma unroll
       for (int o = 0; o < AT_PARTS; ++o) total += xchg[o * AT_BM + rr];
+      if (WINDOW && sink && valid_row) total += exp2f(fmaf(sink[hk * g + R % g], 1.4426950408889634f, -m_ref));
       float inv = total > 0.f ? 1.0f / total : 0.f;
       if (SIGMOID) inv = (gate && valid_row) ? gate[(size_t)(qs + R / g) * Hq + hk * g + R % g] : 1.f;
       // The output tile goes through shared memory (where the query tile was: every product that read
@@ -454,15 +475,16 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant_
 #undef abort_flag
 }
 
-template <int D, bool SIGMOID = false>
+template <int D, bool SIGMOID = false, bool WINDOW = false>
 static int attn_tc_launch(const void* q, const void* k_pages, const void* v_pages, void* out, const int* q_start,
                           const int* kv_len, const int* block_table, int table_stride, int page_size, int num_pages,
                           int B, int max_q_len, int Hq, int Hkv, float scale, int* status, cudaStream_t stream,
-                          const float* head_bias = nullptr, const float* gate = nullptr) {
+                          const float* head_bias = nullptr, const float* gate = nullptr, int window = 0,
+                          const float* sink = nullptr) {
   using S = AttnTcShape<D>;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel<D, SIGMOID>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel<D, SIGMOID, WINDOW>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          (int)S::SMEM_BYTES);
     if (e != cudaSuccess) return (int)e;
     configured = true;
@@ -477,9 +499,9 @@ static int attn_tc_launch(const void* q, const void* k_pages, const void* v_page
   const long long tiles = ((long long)max_q_len * g + AT_BM - 1) / AT_BM;
   if (tiles > 65535) return Q3_ERR_SIZE;
   dim3 grid(Hkv, (unsigned)tiles, B);
-  q3::launch(attn_tc_kernel<D, SIGMOID>, grid, dim3(AT_THREADS), S::SMEM_BYTES, stream, map_k, map_v,
+  q3::launch(attn_tc_kernel<D, SIGMOID, WINDOW>, grid, dim3(AT_THREADS), S::SMEM_BYTES, stream, map_k, map_v,
              (const __nv_bfloat16*)q, (__nv_bfloat16*)out, q_start, kv_len, block_table, table_stride, page_size, num_pages,
-             Hq, Hkv, scale * 1.4426950408889634f, status, head_bias, gate);
+             Hq, Hkv, scale * 1.4426950408889634f, status, head_bias, gate, window, sink);
   return launch_status();
 }
 
@@ -505,6 +527,27 @@ extern "C" int q3_attn_tc(const void* q, const void* k_pages, const void* v_page
                                   num_pages, B, max_q_len, Hq, Hkv, scale, status, stream);
   return q3::attn_tc_launch<128>(q, k_pages, v_pages, out, q_start, kv_len, block_table, table_stride, page_size,
                                  num_pages, B, max_q_len, Hq, Hkv, scale, status, stream);
+}
+
+// The same over a sliding window (the keys n with p - window < n <= p; pages before it may have been given back) with a sink
+// (float32 [Hq] or null).  Limits as q3_attn_tc, and a positive scale.
+extern "C" int q3_attn_tc_window(const void* q, const void* k_pages, const void* v_pages, void* out, const int* q_start,
+                                 const int* kv_len, const int* block_table, int table_stride, int page_size, int num_pages,
+                                 int B, int max_q_len, int Hq, int Hkv, int D, float scale, int window, const float* sink,
+                                 int* status, cudaStream_t stream) {
+  if (B <= 0 || max_q_len <= 0) return 0;
+  if (Hkv <= 0 || Hq % Hkv || (D != 64 && D != 128) || table_stride <= 0 || B > 65535 || Hkv > 65535 || window <= 0 ||
+      !(scale > 0.f) || (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64))
+    return Q3_ERR_SIZE;
+  if ((uintptr_t)q % 16 || (uintptr_t)k_pages % 16 || (uintptr_t)v_pages % 16 || (uintptr_t)out % 16)
+    return Q3_ERR_ALIGN;
+  if (D == 64)
+    return q3::attn_tc_launch<64, false, true>(q, k_pages, v_pages, out, q_start, kv_len, block_table, table_stride, page_size,
+                                               num_pages, B, max_q_len, Hq, Hkv, scale, status, stream, nullptr, nullptr,
+                                               window, sink);
+  return q3::attn_tc_launch<128, false, true>(q, k_pages, v_pages, out, q_start, kv_len, block_table, table_stride, page_size,
+                                              num_pages, B, max_q_len, Hq, Hkv, scale, status, stream, nullptr, nullptr,
+                                              window, sink);
 }
 
 // The same kernel with sigmoid weights (see attn_sigmoid.cu): head_bias float32 [Hq] or null, gate float32

@@ -37,6 +37,14 @@ __device__ __forceinline__ float2 cm_pair(const __nv_bfloat16* p) {  // two neig
   return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
 }
 
+// The logarithms are kept in units of the base-2 exponential.
+constexpr float CM_LOG2E = 1.4426950408889634f;
+__device__ __forceinline__ float cm_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 struct ChannelMma {
   const __nv_bfloat16* x;  // [T, ld]: q, k (H heads of D), v (H heads of D) at columns
   int ld, q_col, k_col, v_col;
@@ -46,7 +54,7 @@ struct ChannelMma {
   const int *q_start, *slot_ids;
   float* state;    // [slots, H, D, D]: value by value, the keys' channels side by side
   float* records;  // per chunk [H, D, D]: chunk j of request b is record q_start[b] / CC + b + j
-  float* totals;   // per chunk [H, D]: b_last
+  float* totals;   // per chunk [H, D]: b_last (base 2)
   float* out;      // [T, H, D]
   int* status;
 };
@@ -88,7 +96,7 @@ channel_chunk_state_kernel(ChannelMma in) {
 #pragma unroll
     for (int i = 0; i < PT; ++i) {
       const int t = part * PT + i;
-      lw[i] = t < len ? in.logw[((size_t)(t0 + t) * H + h) * D + d] : 0.f;
+      lw[i] = t < len ? CM_LOG2E * in.logw[((size_t)(t0 + t) * H + h) * D + d] : 0.f;
       kv[i] = t < len ? __bfloat162float(in.x[(size_t)(t0 + t) * in.ld + in.k_col + h * D + d]) : 0.f;
     }
 #pragma unroll
@@ -100,7 +108,7 @@ channel_chunk_state_kernel(ChannelMma in) {
     if (part == 0) in.totals[((size_t)(start / CC + b + blockIdx.y) * H + h) * D + d] = after + total;
 #pragma unroll
     for (int i = PT - 1; i >= 0; --i) {
-      const float v = kv[i] * __expf(after);
+      const float v = kv[i] * cm_exp2(after);
       const __nv_bfloat16 hi = __float2bfloat16_rn(v);
       k_hi[(part * PT + i) * PN + d] = hi;
       k_lo[(part * PT + i) * PN + d] = __float2bfloat16_rn(v - __bfloat162float(hi));
@@ -167,10 +175,10 @@ __global__ void channel_chunk_carry_kernel(ChannelMma in, int D) {
     for (int k = 0; k < AHEAD; ++k)
       if (j0 + k < chunks) {
         *reinterpret_cast<float4*>(rec + (size_t)k * all) = S;
-        S.x = fmaf(__expf(keep[k].x), S.x, reached[k].x);
-        S.y = fmaf(__expf(keep[k].y), S.y, reached[k].y);
-        S.z = fmaf(__expf(keep[k].z), S.z, reached[k].z);
-        S.w = fmaf(__expf(keep[k].w), S.w, reached[k].w);
+        S.x = fmaf(cm_exp2(keep[k].x), S.x, reached[k].x);
+        S.y = fmaf(cm_exp2(keep[k].y), S.y, reached[k].y);
+        S.z = fmaf(cm_exp2(keep[k].z), S.z, reached[k].z);
+        S.w = fmaf(cm_exp2(keep[k].w), S.w, reached[k].w);
       }
   }
   *reinterpret_cast<float4*>(in.state + (size_t)slot * all + e) = S;
@@ -222,7 +230,7 @@ channel_chunk_output_kernel(ChannelMma in) {
 #pragma unroll
     for (int i = 0; i < CP; ++i) {
       const int t = part * CP + i;
-      lw[i] = t < len ? in.logw[((size_t)(t0 + t) * H + h) * D + d] : 0.f;
+      lw[i] = t < len ? CM_LOG2E * in.logw[((size_t)(t0 + t) * H + h) * D + d] : 0.f;
     }
     float* dst = sums + part * (CP + 1) * PB + d;
 #pragma unroll
@@ -261,7 +269,7 @@ channel_chunk_output_kernel(ChannelMma in) {
         const int row = gid + (r & 1) * 8, d = kk * 16 + 2 * tid4 + (r >> 1) * 8;
         const float2 q = cm_pair(qs + (part * CP + row) * PN + d);
         const float2 e = *reinterpret_cast<const float2*>(mine + row * PB + d);
-        cm_split_pack(q.x * __expf(e.x), q.y * __expf(e.y), qh[r], ql[r]);
+        cm_split_pack(q.x * cm_exp2(e.x), q.y * cm_exp2(e.y), qh[r], ql[r]);
       }
 #pragma unroll
       for (int i = 0; i < CPARTS - 1; ++i) {
@@ -275,7 +283,7 @@ channel_chunk_output_kernel(ChannelMma in) {
           const float2 e = *reinterpret_cast<const float2*>(sums + (i * (CP + 1) + hf * 8 + gid + 1) * PB + d);
           const float2 from = *reinterpret_cast<const float2*>(starts + i * D + d);
           const float2 to = *reinterpret_cast<const float2*>(starts + part * D + d);
-          cm_split_pack(k.x * __expf(to.x - from.x - e.x), k.y * __expf(to.y - from.y - e.y), kh[r], kl[r]);
+          cm_split_pack(k.x * cm_exp2(to.x - from.x - e.x), k.y * cm_exp2(to.y - from.y - e.y), kh[r], kl[r]);
         }
         mma_bf16(g[i], qh, kh[0], kh[1]);
         mma_bf16(g[i], qh, kl[0], kl[1]);
@@ -306,8 +314,8 @@ channel_chunk_output_kernel(ChannelMma in) {
         const float4 bs = *reinterpret_cast<const float4*>(mine + (s + 1) * PB + d);
         const bool own = s == t;
         // beyond the diagonal the exponent would be positive: held at zero, the sum is not used
-        const float w0 = own ? u.x : __expf(fminf(bt.x - bs.x, 0.f)), w1 = own ? u.y : __expf(fminf(bt.y - bs.y, 0.f));
-        const float w2 = own ? u.z : __expf(fminf(bt.z - bs.z, 0.f)), w3 = own ? u.w : __expf(fminf(bt.w - bs.w, 0.f));
+        const float w0 = own ? u.x : cm_exp2(fminf(bt.x - bs.x, 0.f)), w1 = own ? u.y : cm_exp2(fminf(bt.y - bs.y, 0.f));
+        const float w2 = own ? u.z : cm_exp2(fminf(bt.z - bs.z, 0.f)), w3 = own ? u.w : cm_exp2(fminf(bt.w - bs.w, 0.f));
         acc[j] = fmaf(q0.x * k0.x, w0, acc[j]);
         acc[j] = fmaf(q0.y * k0.y, w1, acc[j]);
         acc[j] = fmaf(q1.x * k1.x, w2, acc[j]);
@@ -370,7 +378,7 @@ channel_chunk_output_kernel(ChannelMma in) {
         const float2 q = cm_pair(qs + (part * CP + row) * PN + d);
         const float2 e = *reinterpret_cast<const float2*>(mine + row * PB + d);
         const float2 f = *reinterpret_cast<const float2*>(starts + part * D + d);
-        cm_split_pack(q.x * __expf(e.x + f.x), q.y * __expf(e.y + f.y), qh[r], ql[r]);
+        cm_split_pack(q.x * cm_exp2(e.x + f.x), q.y * cm_exp2(e.y + f.y), qh[r], ql[r]);
       }
 #pragma unroll
       for (int np = 0; np < NTW / 2; ++np) {

@@ -369,72 +369,125 @@ static int memory_scan_sizes(const MemoryIn<T>& in, float* state, const int* q_s
 
 // ---------------------------------------------------------------- decays from a low-rank projection
 // logw[t, c] = -exp(sum_r w2[c, r] tanh(low[t, r]) + w0[c]), at least LR_LEAST (whose exponential is zero in float32).
-// low: [T, ld]; w2: [C, R]; w0: [C]; logw: [T, C].  A block takes LR_T tokens and LR_C channels; a sum runs over r in order.
-constexpr int LR_T = 32, LR_C = 64, LR_R = 32, LR_THREADS = 256;
+// low: [T, ld]; w2t: [R, C]; w0: [C]; logw: [T, C].  Every sum runs over r in order, so that a token's decays do not depend on how
+// many there are.  For many tokens a block takes TT of them and TC channels, a thread 4 x 4; for a few, a warp per token and
+// LF_C channels, with all of their weights in shared memory.
+constexpr int LR_R = 32, LR_TT = 64, LR_TC = 64, LR_THREADS = LR_TT * LR_TC / 16;
+constexpr int LF_T = 8, LF_C = 32, LF_MAX_R = 256;
 constexpr float LR_LEAST = -104.f;
 
+__device__ __forceinline__ float log_decay_of(float sum, float w0) { return fmaxf(-expf(sum + w0), LR_LEAST); }
+
 __global__ void __launch_bounds__(LR_THREADS)
-low_rank_decay_kernel(const float* __restrict__ low, int ld, const float* __restrict__ w2, const float* __restrict__ w0,
+low_rank_decay_kernel(const float* __restrict__ low, int ld, const float* __restrict__ w2t, const float* __restrict__ w0,
                       float* __restrict__ logw, int Ttot, int C, int R) {
-  __shared__ float a_s[LR_R][LR_T + 1], w_s[LR_R][LR_C + 1];
-  const int t0 = blockIdx.y * LR_T, c0 = blockIdx.x * LR_C;
-  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;  // four channels tx + 16 j, two tokens ty + 16 i
+  __shared__ __align__(16) float a_s[LR_R][LR_TT + 4], w_s[LR_R][LR_TC + 4];
+  const int t0 = blockIdx.y * LR_TT, c0 = blockIdx.x * LR_TC;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;  // channels 4 tx .. 4 tx + 3, tokens 4 ty .. 4 ty + 3
   auto weights = [&](int r0) {
-    for (int i = threadIdx.x; i < LR_C * LR_R; i += LR_THREADS) {
-      const int c = i / LR_R, r = i % LR_R;
-      w_s[r][c] = c0 + c < C && r0 + r < R ? w2[(size_t)(c0 + c) * R + r0 + r] : 0.f;
+#pragma unroll
+    for (int i = threadIdx.x; i < LR_TC * LR_R; i += LR_THREADS) {
+      const int c = i % LR_TC, r = i / LR_TC;
+      w_s[r][c] = c0 + c < C && r0 + r < R ? w2t[(size_t)(r0 + r) * C + c0 + c] : 0.f;
     }
   };
   weights(0);  // they do not depend on the kernel before this one
   pdl_wait();
   pdl_launch_dependents();
-  float acc[2][4] = {};
+  float acc[4][4] = {};
   for (int r0 = 0; r0 < R; r0 += LR_R) {
     if (r0 > 0) {
       __syncthreads();
       weights(r0);
     }
-    for (int i = threadIdx.x; i < LR_T * LR_R; i += LR_THREADS) {
+#pragma unroll
+    for (int i = threadIdx.x; i < LR_TT * LR_R; i += LR_THREADS) {
       const int t = i / LR_R, r = i % LR_R;
       a_s[r][t] = t0 + t < Ttot && r0 + r < R ? tanhf(low[(size_t)(t0 + t) * ld + r0 + r]) : 0.f;
     }
     __syncthreads();
 #pragma unroll 8
     for (int r = 0; r < LR_R; ++r) {
-      const float a0 = a_s[r][ty], a1 = a_s[r][ty + 16];
+      const float4 w = *reinterpret_cast<const float4*>(&w_s[r][4 * tx]);
+      const float4 av = *reinterpret_cast<const float4*>(&a_s[r][4 * ty]);
+      const float a[4] = {av.x, av.y, av.z, av.w};
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float w = w_s[r][tx + 16 * j];
-        acc[0][j] = fmaf(a0, w, acc[0][j]);
-        acc[1][j] = fmaf(a1, w, acc[1][j]);
+      for (int i = 0; i < 4; ++i) {
+        acc[i][0] = fmaf(a[i], w.x, acc[i][0]);
+        acc[i][1] = fmaf(a[i], w.y, acc[i][1]);
+        acc[i][2] = fmaf(a[i], w.z, acc[i][2]);
+        acc[i][3] = fmaf(a[i], w.w, acc[i][3]);
       }
     }
   }
+  const int c = c0 + 4 * tx;
+  if (c >= C) return;
+  const bool by4 = (C & 3) == 0;
+  float off[4];
 #pragma unroll
-  for (int i = 0; i < 2; ++i)
+  for (int j = 0; j < 4; ++j) off[j] = c + j < C ? w0[c + j] : 0.f;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int t = t0 + ty + 16 * i, c = c0 + tx + 16 * j;
-      if (t < Ttot && c < C) logw[(size_t)t * C + c] = fmaxf(-expf(acc[i][j] + w0[c]), LR_LEAST);
+  for (int i = 0; i < 4; ++i) {
+    const int t = t0 + 4 * ty + i;
+    if (t >= Ttot) continue;
+    float* dst = logw + (size_t)t * C + c;
+    const float4 v = make_float4(log_decay_of(acc[i][0], off[0]), log_decay_of(acc[i][1], off[1]), log_decay_of(acc[i][2], off[2]),
+                                 log_decay_of(acc[i][3], off[3]));
+    if (by4) {
+      *reinterpret_cast<float4*>(dst) = v;
+    } else {
+      const float e[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < C) dst[j] = e[j];
     }
+  }
+}
+
+__global__ void __launch_bounds__(LF_T * 32)
+low_rank_decay_few_kernel(const float* __restrict__ low, int ld, const float* __restrict__ w2t, const float* __restrict__ w0,
+                          float* __restrict__ logw, int Ttot, int C, int R) {
+  extern __shared__ float lf_smem[];  // [R][LF_C] weights, [LF_T][R] inputs
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c = blockIdx.x * LF_C + lane, t = blockIdx.y * LF_T + warp;
+  float* w_s = lf_smem;
+  float* a_s = lf_smem + R * LF_C + warp * R;
+#pragma unroll 8
+  for (int r = warp; r < R; r += LF_T) w_s[r * LF_C + lane] = c < C ? w2t[(size_t)r * C + c] : 0.f;
+  const float off = c < C ? w0[c] : 0.f;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (t < Ttot)
+    for (int r = lane; r < R; r += 32) a_s[r] = tanhf(low[(size_t)t * ld + r]);
+  __syncthreads();
+  if (t >= Ttot || c >= C) return;
+  float acc = 0.f;
+#pragma unroll 8
+  for (int r = 0; r < R; ++r) acc = fmaf(a_s[r], w_s[r * LF_C + lane], acc);
+  logw[(size_t)t * C + c] = log_decay_of(acc, off);
 }
 
 // ---------------------------------------------------------------- the norm and the gate behind a memory
-// A unit (a warp, or with WHOLE a block) per (token, part), V values per access.  o: float32 [T, n]; gates at g_col of
+// A unit (LANES lanes of a warp, or with WHOLE a block) per (token, part), V values per access.  o: float32 [T, n]; gates at g_col of
 // proj; weight [n] (w_stride = width of a part), [width] shared by the parts (w_stride = 0), or null.
 template <typename T, int V>
 struct alignas(sizeof(T) * V) LmPack { T v[V]; };
 
-template <typename T, int V, bool WHOLE>
+template <typename T, int V, bool WHOLE, int LANES = 32>
 __global__ void memory_out_kernel(const float* __restrict__ o, const T* __restrict__ proj, int ld, int g_col,
                                   const float* __restrict__ w, int w_stride, float eps, int gate, T* __restrict__ out,
                                   int ldo, int n, int parts, int units) {
   __shared__ float red[32];
   pdl_wait();
   pdl_launch_dependents();
-  const int unit = WHOLE ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (unit >= units) return;
-  const int first = WHOLE ? threadIdx.x : threadIdx.x & 31, step = WHOLE ? blockDim.x : 32;
+  int unit = WHOLE ? blockIdx.x : blockIdx.x * (blockDim.x / LANES) + threadIdx.x / LANES;
+  const bool live = unit < units;
+  if (WHOLE || LANES == 32) {
+    if (!live) return;
+  } else {
+    unit = min(unit, units - 1);  // lanes of one warp stay together for the sum
+  }
+  const int first = WHOLE ? threadIdx.x : threadIdx.x % LANES, step = WHOLE ? blockDim.x : LANES;
   const int t = unit / parts, part = unit - t * parts, width = n / parts, c0 = part * width;
   const float* row = o + (size_t)t * n + c0;
   const T* gr = proj + (size_t)t * ld + g_col + c0;
@@ -447,7 +500,13 @@ __global__ void memory_out_kernel(const float* __restrict__ o, const T* __restri
 #pragma unroll
     for (int e = 0; e < V; ++e) ss = fmaf(x.v[e], x.v[e], ss);
   }
-  ss = WHOLE ? block_sum(ss, red) : warp_sum(ss);
+  if (WHOLE) {
+    ss = block_sum(ss, red);
+  } else {
+#pragma unroll
+    for (int w = LANES / 2; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+    if (!live) return;
+  }
   const float inv = 1.0f / sqrtf(ss / (float)width + eps);
 #pragma unroll 4
   for (int i = first * V; i < width; i += step * V) {
@@ -546,13 +605,18 @@ extern "C" int q3_channel_memory_scan(const void* x, int ld, int q_col, int k_co
   })
 }
 
-// low: float32 rows of ld values (the first R are read); w2: float32 [C, R]; w0: float32 [C]; logw: float32 [T, C].
-extern "C" int q3_low_rank_decay(const float* low, int ld, const float* w2, const float* w0, float* logw, int T, int C, int R,
+// low: float32 rows of ld values (the first R are read); w2t: float32 [R, C]; w0: float32 [C]; logw: float32 [T, C].
+extern "C" int q3_low_rank_decay(const float* low, int ld, const float* w2t, const float* w0, float* logw, int T, int C, int R,
                                  cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (C <= 0 || R <= 0 || R > ld || T > 32 * 65535) return Q3_ERR_SIZE;
-  q3::launch(q3::low_rank_decay_kernel, dim3((C + q3::LR_C - 1) / q3::LR_C, (T + q3::LR_T - 1) / q3::LR_T), dim3(q3::LR_THREADS), 0,
-             stream, low, ld, w2, w0, logw, T, C, R);
+  if (C <= 0 || R <= 0 || R > ld || T > q3::LF_T * 65535) return Q3_ERR_SIZE;
+  if ((uintptr_t)logw % 16) return Q3_ERR_ALIGN;
+  if (T <= 128 && R <= q3::LF_MAX_R)
+    q3::launch(q3::low_rank_decay_few_kernel, dim3((C + q3::LF_C - 1) / q3::LF_C, (T + q3::LF_T - 1) / q3::LF_T), dim3(q3::LF_T * 32),
+               (size_t)R * (q3::LF_C + q3::LF_T) * sizeof(float), stream, low, ld, w2t, w0, logw, T, C, R);
+  else
+    q3::launch(q3::low_rank_decay_kernel, dim3((C + q3::LR_TC - 1) / q3::LR_TC, (T + q3::LR_TT - 1) / q3::LR_TT), dim3(q3::LR_THREADS),
+               0, stream, low, ld, w2t, w0, logw, T, C, R);
   return q3::launch_status();
 }
 
@@ -571,17 +635,20 @@ extern "C" int q3_memory_out(const float* o, const void* proj, int ld, int g_col
   // a block per part where parts are long, else a warp per part
   const bool whole = width >= 512;
   const int threads = whole ? (width >= 2048 ? 512 : 256) : 128;
-  const unsigned grid = (unsigned)(whole ? units : (units + 3) / 4);
-#define Q3_MEMORY_OUT(V, WHOLE)                                                                                         \
+  const int lanes = !by4 || whole || width > 64 ? 32 : (width > 32 ? 16 : 8);  // short parts: several to a warp
+  const unsigned grid = (unsigned)(whole ? units : (units * lanes + threads - 1) / threads);
+#define Q3_MEMORY_OUT(V, WHOLE, LANES)                                                                                         \
   Q3_BY_DTYPE(dtype, {                                                                                                   \
-    auto kernel = q3::memory_out_kernel<E, V, WHOLE>;                                                                    \
+    auto kernel = q3::memory_out_kernel<E, V, WHOLE, LANES>;                                                                    \
     q3::launch(kernel, dim3(grid), dim3(threads), 0, stream, o, (const E*)proj, ld, g_col, weight, shared, eps, gate, (E*)out, \
                ldo, n, parts, (int)units);                                                                               \
   })
-  if (by4 && whole) { Q3_MEMORY_OUT(4, true) }
-  else if (by4) { Q3_MEMORY_OUT(4, false) }
-  else if (whole) { Q3_MEMORY_OUT(1, true) }
-  else { Q3_MEMORY_OUT(1, false) }
+  if (by4 && whole) { Q3_MEMORY_OUT(4, true, 32) }
+  else if (by4 && lanes == 16) { Q3_MEMORY_OUT(4, false, 16) }
+  else if (by4 && lanes == 8) { Q3_MEMORY_OUT(4, false, 8) }
+  else if (by4) { Q3_MEMORY_OUT(4, false, 32) }
+  else if (whole) { Q3_MEMORY_OUT(1, true, 32) }
+  else { Q3_MEMORY_OUT(1, false, 32) }
 #undef Q3_MEMORY_OUT
   return q3::launch_status();
 }

@@ -7,7 +7,9 @@
 //                  chosen.  Their weights are s * scale (the bias takes no part in the weights), divided by the sum
 //                  of the chosen s (+ 1e-20) with `renorm`.  A bias of the logits themselves (`zbias`) is added before
 //                  anything else.  With `share` the router's matrix has one more row w_s, and share[t] =
-//                  sigmoid(w_s h): what a shared expert's output is multiplied by.  One block per token.
+//                  sigmoid(w_s h): what a shared expert's output is multiplied by.  A block per token or per eight; in
+//                  bfloat16, up to MR_MAX_ROWS rows of the router, per sixteen on the tensor cores: the router's float32
+//                  numbers as three bfloat16 ones whose sum they are, so that every product is exact and the sums float32.
 //   moe_pair_up    for every (token, chosen expert) pair: act(W_up[e] h), a warp per output value; the pair's expert
 //                  weight is streamed once per pair.  For a few tokens (decoding) and the float32 run.
 //   moe_pair_down  out[t] = base[t] + sum_k weight[t, k] W_down[e_k] a[t, k]: a warp per output value, the chosen
@@ -20,7 +22,7 @@
 //
 // Sums over a row are taken lane by lane in ascending order and then across the warp, so a token's result does not
 // depend on the batch.  `base_wts` (or null): base[t] counts times base_wts[t].  The expert weights are stacked: up [E, F, W], down [E, W, F].
-#include "common.cuh"
+#include "attn_mma.cuh"
 
 namespace q3 {
 
@@ -229,6 +231,88 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
                    wts + (size_t)(t0 + k) * c.top, lane);
 }
 
+// Sixteen tokens to a block; the eight warps share the sum over W, in groups of 32 values of which lane t of a row takes
+// k = 8 t .. 8 t + 7 (see gemm_skinny.cu), and meet in shared memory in order.  W a multiple of 8.
+constexpr int MR_TOK = 16, MR_WARPS = 8, MR_MAX_ROWS = 40;
+
+template <int NT>  // tiles of eight router rows
+__global__ void __launch_bounds__(MR_WARPS * 32)
+moe_route_mma_kernel(const __nv_bfloat16* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ bias,
+                     const float* __restrict__ zbias, int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ share,
+                     int Ttot, int W, Choice c) {
+  extern __shared__ __align__(16) float score[];  // [16][E] scores, [16][E] keys, [16][groups] flags
+  __shared__ float part[MR_WARPS][MR_TOK][8 * NT + 1];
+  unsigned* key = reinterpret_cast<unsigned*>(score + MR_TOK * c.E);
+  unsigned* kept = key + MR_TOK * c.E;
+  const int t0 = blockIdx.x * MR_TOK, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, gid = lane >> 2, tid4 = lane & 3;
+  const int rows = c.E + (share ? 1 : 0);
+  const int groups32 = (W + 31) / 32, per = (groups32 + MR_WARPS - 1) / MR_WARPS;
+  const int g_lo = warp * per, g_hi = min(groups32, g_lo + per);
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  pdl_wait();
+  pdl_launch_dependents();
+  const __nv_bfloat16* x_lo = h + (size_t)min(t0 + gid, Ttot - 1) * W;
+  const __nv_bfloat16* x_hi = h + (size_t)min(t0 + gid + 8, Ttot - 1) * W;
+#pragma unroll 2
+  for (int g = g_lo; g < g_hi; ++g) {
+    const int k = g * 32 + 8 * tid4;
+    const bool in = k < W;
+    const uint4 lo = in ? *reinterpret_cast<const uint4*>(x_lo + k) : make_uint4(0, 0, 0, 0);
+    const uint4 hi = in ? *reinterpret_cast<const uint4*>(x_hi + k) : make_uint4(0, 0, 0, 0);
+    const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      const int e = nt * 8 + gid;
+      float w[8];
+      if (in && e < rows) {
+        const float4 u = *reinterpret_cast<const float4*>(wr + (size_t)e * W + k);
+        const float4 v = *reinterpret_cast<const float4*>(wr + (size_t)e * W + k + 4);
+        w[0] = u.x, w[1] = u.y, w[2] = u.z, w[3] = u.w, w[4] = v.x, w[5] = v.y, w[6] = v.z, w[7] = v.w;
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) w[i] = 0.f;
+      }
+#pragma unroll
+      for (int piece = 0; piece < 3; ++piece) {  // the upper eight bits, the middle, the lower
+        uint32_t b[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const __nv_bfloat162 p = __floats2bfloat162_rn(w[2 * i], w[2 * i + 1]);
+          const float2 f = __bfloat1622float2(p);
+          b[i] = *reinterpret_cast<const uint32_t*>(&p);
+          w[2 * i] -= f.x;
+          w[2 * i + 1] -= f.y;
+        }
+        mma_bf16(acc[nt], a0, b[0], b[1]);
+        mma_bf16(acc[nt], a1, b[2], b[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) part[warp][gid + 8 * (j >> 1)][nt * 8 + 2 * tid4 + (j & 1)] = acc[nt][j];
+  __syncthreads();
+  for (int i = threadIdx.x; i < MR_TOK * rows; i += MR_WARPS * 32) {
+    const int k = i / rows, e = i - k * rows;
+    float dot = 0.f;
+#pragma unroll
+    for (int w = 0; w < MR_WARPS; ++w) dot += part[w][k][e];
+    if (e == c.E) {
+      if (t0 + k < Ttot) share[t0 + k] = sigmoid_f(dot);
+      continue;
+    }
+    if (zbias) dot += zbias[e];
+    score[k * c.E + e] = c.softmax ? dot : sigmoid_f(dot);
+  }
+  __syncthreads();
+  for (int k = warp; k < MR_TOK && t0 + k < Ttot; k += MR_WARPS)
+    choose_experts(c, score + k * c.E, key + k * c.E, kept + k * c.groups, bias, ids + (size_t)(t0 + k) * c.top,
+                   wts + (size_t)(t0 + k) * c.top, lane);
+}
+
 // grid (pairs, ceil(F / warps)).  a[pair, f] = act(sum_i up[e, f, i] h[t, i]), t = pair / top.
 template <typename T>
 __global__ void moe_pair_up_kernel(const T* __restrict__ h, const T* __restrict__ up, const int* __restrict__ ids,
@@ -313,6 +397,19 @@ extern "C" int q3_moe_route(const void* h, const float* wr, const float* bias, c
   if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups)) return Q3_ERR_SIZE;
   if ((size_t)(2 * E + groups + 3) * sizeof(float) > 48 * 1024) return Q3_ERR_SIZE;
   const q3::Choice choice{E, top, softmax, groups, keep, renorm, scale};
+  const int rows = E + (share ? 1 : 0);
+  if (dtype == Q3_BF16 && rows <= q3::MR_MAX_ROWS && W % 8 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)wr % 16 == 0) {
+    auto go = [&](auto kernel) {
+      q3::launch(kernel, dim3((T + q3::MR_TOK - 1) / q3::MR_TOK), dim3(q3::MR_WARPS * 32),
+                 (size_t)q3::MR_TOK * (2 * E + groups) * sizeof(float), stream, (const __nv_bfloat16*)h, wr, bias, zbias, ids, wts,
+                 share, T, W, choice);
+      return q3::launch_status();
+    };
+    if (rows <= 8) return go(q3::moe_route_mma_kernel<1>);
+    if (rows <= 16) return go(q3::moe_route_mma_kernel<2>);
+    if (rows <= 24) return go(q3::moe_route_mma_kernel<3>);
+    return go(q3::moe_route_mma_kernel<5>);
+  }
   // many tokens: eight to a block, so that the experts' rows are read an eighth as often
   constexpr int MANY = 8;
   const size_t es = dtype == Q3_F32 ? 4 : 2;

@@ -105,7 +105,9 @@ struct alignas(sizeof(T) * V) PwPack { T v[V]; };
 
 constexpr int HQ_WARPS = 8;
 
-template <typename T, int V>
+// PER: accesses of a lane per head (heads of up to 32 V PER values).  LANES: with one access per head and halves of a rotation in
+// multiples of V, a value's partner comes from another lane's registers; else through shared memory.
+template <typename T, int V, int PER, bool LANES>
 __global__ void __launch_bounds__(HQ_WARPS * 32)
 head_qkv_post_kernel(const T* __restrict__ proj, int ld, int k_col, int v_col, int has_kv, int H, int G, int D, int Dv,
                      const float* __restrict__ bias, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
@@ -113,10 +115,25 @@ head_qkv_post_kernel(const T* __restrict__ proj, int ld, int k_col, int v_col, i
                      const int* __restrict__ tok_seq, const int* __restrict__ table, int stride, int page_size, int num_pages,
                      T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, int* status) {
   extern __shared__ float hq_smem[];  // [dims / 2] cosines, [dims / 2] sines, times mag; then per warp a head's values
-  constexpr int PER = PW_PER / V;
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  auto place = [&](int u, int& col, int& width) {  // a head's columns of the projection
+    const bool is_q = u < H, is_v = u >= H + G;
+    width = is_v ? Dv : D;
+    col = is_q ? u * D : (is_v ? v_col + (u - H - G) * Dv : k_col + (u - H) * D);
+  };
+  PwPack<T, V> next[PER];
+  auto fetch = [&](int u) {  // a head ahead, so that its loads are in flight while the head before is worked on
+    int col, width;
+    place(u, col, width);
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+      const int i = (k * 32 + lane) * V;
+      if (i < width) next[k] = *reinterpret_cast<const PwPack<T, V>*>(proj + (size_t)t * ld + col + i);
+    }
+  };
+  if (warp < H) fetch(warp);
   const int pos = positions[t], b = tok_seq[t], half = dims >> 1;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float sn, c;
@@ -136,12 +153,13 @@ head_qkv_post_kernel(const T* __restrict__ proj, int ld, int k_col, int v_col, i
     in_page = write ? pos % page_size : 0;
   }
   __syncthreads();
-  const int units = H + (has_kv ? 2 * G : 0);
+  const int units = H + (write ? 2 * G : 0);
+  if (warp >= H && warp < units) fetch(warp);
   for (int u = warp; u < units; u += HQ_WARPS) {
     const bool is_q = u < H, is_v = u >= H + G;
-    const int g = is_q ? 0 : (is_v ? u - H - G : u - H), width = is_v ? Dv : D;
-    const int col = is_q ? u * D : (is_v ? v_col + g * Dv : k_col + g * D);
-    if (!is_q && !write) continue;
+    const int g = is_q ? 0 : (is_v ? u - H - G : u - H);
+    int col, width;
+    place(u, col, width);
     T* dst = is_q ? q_out + ((size_t)t * H + u) * D
                   : (is_v ? v_pages + (((size_t)page * G + g) * page_size + in_page) * Dv
                           : k_pages + (((size_t)page * G + g) * page_size + in_page) * D);
@@ -151,25 +169,48 @@ head_qkv_post_kernel(const T* __restrict__ proj, int ld, int k_col, int v_col, i
     for (int k = 0; k < PER; ++k) {
       const int i = (k * 32 + lane) * V;
       if (i >= width) continue;
-      const PwPack<T, V> p = *reinterpret_cast<const PwPack<T, V>*>(proj + (size_t)t * ld + col + i);
+      PwPack<float, V> bv{};
+      if (bias) bv = *reinterpret_cast<const PwPack<float, V>*>(bias + col + i);
 #pragma unroll
       for (int e = 0; e < V; ++e) {
-        x[k][e] = to_float(p.v[e]);
-        if (bias) x[k][e] += bias[col + i + e];
+        x[k][e] = to_float(next[k].v[e]) + bv.v[e];
         ss = fmaf(x[k][e], x[k][e], ss);
       }
     }
+    if (u + HQ_WARPS < units) fetch(u + HQ_WARPS);
     const float r = w ? 1.0f / sqrtf(warp_sum(ss) / (float)D + eps) : 1.0f;
     const bool turn = !is_v && dims > 0;
 #pragma unroll
     for (int k = 0; k < PER; ++k) {
       const int i = (k * 32 + lane) * V;
       if (i >= width) continue;
+      PwPack<float, V> wv;
+      if (w) wv = *reinterpret_cast<const PwPack<float, V>*>(w + i);
 #pragma unroll
       for (int e = 0; e < V; ++e) {
-        if (w) x[k][e] *= r * w[i + e];
-        if (turn) head[i + e] = x[k][e];
+        if (w) x[k][e] *= r * wv.v[e];
+        if (!LANES && turn) head[i + e] = x[k][e];
       }
+    }
+    if constexpr (LANES) {  // PER = 1: lane l holds the values V l .. V l + V - 1
+      const int d0 = lane * V;
+      const bool lower = d0 < half, turns = turn && d0 < dims;
+      PwPack<float, V> cv{}, sv{};
+      if (turns) {
+        cv = *reinterpret_cast<const PwPack<float, V>*>(hq_smem + (lower ? d0 : d0 - half));
+        sv = *reinterpret_cast<const PwPack<float, V>*>(hq_smem + (lower ? half + d0 : d0));
+      }
+      const int partner = (lower ? lane + half / V : lane - half / V) & 31;
+      PwPack<T, V> y;
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        float v = d0 < width ? x[0][e] : 0.f;
+        const float o = __shfl_sync(0xffffffffu, v, partner);
+        if (turns) v = lower ? v * cv.v[e] - o * sv.v[e] : v * cv.v[e] + o * sv.v[e];
+        y.v[e] = from_float<T>(v);
+      }
+      if (d0 < width) *reinterpret_cast<PwPack<T, V>*>(dst + d0) = y;
+      continue;
     }
     __syncwarp();
 #pragma unroll
@@ -365,17 +406,21 @@ extern "C" int q3_head_qkv_post(const void* proj, int ld, int k_col, int v_col, 
     return Q3_ERR_SIZE;
   const size_t smem = (((dims + 3) & ~3) + q3::HQ_WARPS * ((D + 3) & ~3)) * sizeof(float);
   const bool by4 = D % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && k_col % 4 == 0 && v_col % 4 == 0 && (uintptr_t)proj % 16 == 0 &&
-                   (uintptr_t)q_out % 16 == 0 && (uintptr_t)k_pages % 16 == 0 && (uintptr_t)v_pages % 16 == 0;
-#define Q3_HQ(V)                                                                                                           \
-  Q3_BY_DTYPE(dtype, q3::launch(q3::head_qkv_post_kernel<E Q3_COMMA V>, dim3(T), dim3(q3::HQ_WARPS * 32), smem, stream,    \
+                   (uintptr_t)q_out % 16 == 0 && (uintptr_t)k_pages % 16 == 0 && (uintptr_t)v_pages % 16 == 0 &&
+                   (uintptr_t)bias % 16 == 0 && (uintptr_t)wq % 16 == 0 && (uintptr_t)wk % 16 == 0;
+  const int most = D > Dv ? D : Dv;
+#define Q3_HQ(V, PER, LANES)                                                                                               \
+  Q3_BY_DTYPE(dtype, q3::launch(q3::head_qkv_post_kernel<E Q3_COMMA V Q3_COMMA PER Q3_COMMA LANES>, dim3(T), dim3(q3::HQ_WARPS * 32), smem, stream, \
                                 (const E*)proj, ld, k_col, v_col, has_kv, H, G, D, Dv, bias, wq, wk, eps, dims, freq, mag, \
                                 positions, tok_seq, table, stride, page_size, num_pages, (E*)q_out, (E*)k_pages,           \
                                 (E*)v_pages, status))
 #define Q3_COMMA ,
-  if (by4) {
-    Q3_HQ(4)
+  if (by4 && most <= 128 && dims % 8 == 0) {
+    Q3_HQ(4, 1, true)
+  } else if (by4) {
+    Q3_HQ(4, 4, false)
   } else {
-    Q3_HQ(1)
+    Q3_HQ(1, 16, false)
   }
 #undef Q3_HQ
 #undef Q3_COMMA

@@ -194,6 +194,11 @@ _SIGNATURES = {
     "q3_sum_norm": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p,
                     _c_void_p, _c_void_p, _c_float, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                     _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p],
+    "q3_attn_tc_window": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
+                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p],
+    "q3_attn_decode_tma_sink": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
+                                _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p,
+                                _c_void_p, _c_void_p],
     "q3_sum_mix": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_float, _c_void_p, _c_int, _c_void_p, _c_void_p,
                    _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "q3_channel_memory_scan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
@@ -993,11 +998,12 @@ def _attn_common(name, q, k_pages, v_pages, out, q_start, kv_len, block_table):
 def attn_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor,
                 partial: Optional[torch.Tensor], q_start: torch.Tensor, kv_len: torch.Tensor,
                 block_table: torch.Tensor, num_seqs: int, scale: float, window: int, num_splits: int,
-                status: torch.Tensor, loader: str = "cp_async", raw_qkv=None) -> None:
+                status: torch.Tensor, loader: str = "cp_async", raw_qkv=None, sink: Optional[torch.Tensor] = None) -> None:
     """Split-KV tensor-core attention for the first ``num_seqs`` rows, one query token each.
     ``raw_qkv = (qkv, q_weight, k_weight, eps, cos_sin, write_kv)`` (TMA loader only): ``q`` only gives the
     shape; the kernel norms and rotates the query from the raw projection ``qkv[T, (Hq + 2 Hkv) D]`` itself
     and makes, stores and uses the new key and value (the work of ``qkv_post`` for these tokens).
+    ``sink`` (float32 [Hq], TMA loader only, a positive scale): exp(sink) joins the softmax's denominator.
     ``loader``: ``"cp_async"`` (every warp copies its own tiles) or ``"tma"`` (a loader warp feeds a
     ring of stages through TMA; head size 64 / 128 and pages that are multiples of 16 only)."""
     T, Hq, D, num_pages, Hkv, page_size = _attn_common("attn_decode", q, k_pages, v_pages, out, q_start, kv_len,
@@ -1029,6 +1035,16 @@ def attn_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, o
             block_table.data_ptr(), block_table.shape[1], page_size, num_pages, num_seqs, Hq, Hkv, D, float(scale),
             int(window), int(num_splits), status.data_ptr(), _stream())
         _done("attn_decode", code, f"heads {Hq}/{Hkv}, head_dim {D}, page {page_size}, raw projection")
+        return
+    if sink is not None:
+        if loader != "tma":
+            raise KernelError("attn_decode: only the kernel with the TMA loader takes a sink")
+        _dist_args("attn_decode", None, sink, Hq)
+        code = library().q3_attn_decode_tma_sink(
+            q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), _ptr(partial), q_start.data_ptr(),
+            kv_len.data_ptr(), block_table.data_ptr(), block_table.shape[1], page_size, num_pages, num_seqs, Hq, Hkv, D,
+            float(scale), int(window), int(num_splits), sink.data_ptr(), status.data_ptr(), _stream())
+        _done("attn_decode", code, f"heads {Hq}/{Hkv}, head_dim {D}, page {page_size}, with a sink")
         return
     fn = library().q3_attn_decode_tma if loader == "tma" else library().q3_attn_decode
     code = fn(q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
@@ -1071,6 +1087,68 @@ def attn_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: 
                                 page_size, num_pages, num_seqs, int(max_q_len), Hq, Hkv, D, float(scale),
                                 status.data_ptr(), _stream())
     _done("attn_tc", code, f"heads {Hq}/{Hkv}, head_dim {D}, page {page_size}")
+
+
+ATTN_TC_WINDOW_FROM = 128  # (token, head) rows per kv head of the longest portion: a whole query tile
+
+
+def window_attention_sizes(dtype: torch.dtype, heads: int, kv_heads: int, dim: int, vdim: int, scale: float) -> bool:
+    """Whether the kernels behind ``window_attention`` take these heads: bfloat16, keys and values alike of 64 or 128 values,
+    up to 16 query heads per kv head, a positive scale."""
+    return (fast_attention_takes(dtype, heads, kv_heads, dim) and dim in (64, 128) and dim == vdim and scale > 0)
+
+
+def window_attention_takes(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor, ctx,
+                           scale: float) -> bool:
+    """Whether ``window_attention`` takes this step: the sizes, the page size, and portions (if there are any) that fill a
+    query tile."""
+    H, D, G, page = q.shape[1], q.shape[2], k_pages.shape[1], k_pages.shape[2]
+    if not (window_attention_sizes(q.dtype, H, G, D, v_pages.shape[3], scale) and out.is_contiguous() and out.data_ptr() % 16 == 0):
+        return False
+    if ctx.num_decode > 0 and not decode_tma_takes(D, page):
+        return False
+    return ctx.num_seqs == ctx.num_decode or (attn_tc_takes(D, page, 0) and ctx.max_q_len * (H // G) >= ATTN_TC_WINDOW_FROM)
+
+
+def window_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor, ctx, table: torch.Tensor,
+                     window: int, scale: float, sink: Optional[torch.Tensor], status: torch.Tensor,
+                     partial: torch.Tensor) -> None:
+    """Softmax attention of a mixed batch over the last ``window`` tokens (``NO_WINDOW``: all), exp(``sink``) (float32 [H] or
+    None) in the denominator: rows that bring one token on the split-KV decode kernel (``partial``: its scratch), portions on
+    the tcgen05 kernel.  ``out`` [T, H * D]."""
+    H, D, G, n = q.shape[1], q.shape[2], k_pages.shape[1], ctx.num_decode
+    if n > 0:
+        splits = decode_splits(n, G, ctx.max_kv_len, min(window, ctx.max_kv_len), D, blocks_per_sm=3, wide_blocks_per_sm=4)
+        splits = max(1, min(splits, partial.numel() // (n * H * (D + 2))))
+        attn_decode(q, k_pages, v_pages, out, partial, ctx.q_start, ctx.kv_len, table, n, scale, window, splits, status,
+                    loader="tma", sink=sink)
+    if ctx.num_seqs > n:
+        attn_tc_window(q, k_pages, v_pages, out, ctx.q_start[n:], ctx.kv_len[n:], table[n:], ctx.num_seqs - n, ctx.max_q_len,
+                       window, scale, sink, status)
+
+
+def attn_tc_window(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor, q_start: torch.Tensor,
+                   kv_len: torch.Tensor, table: torch.Tensor, num_seqs: int, max_q_len: int, window: int, scale: float,
+                   sink: Optional[torch.Tensor], status: torch.Tensor) -> None:
+    """``attn_tc`` over the last ``window`` tokens (``NO_WINDOW``: all), exp(``sink``) (float32 [H] or None) in the softmax's
+    denominator.  ``out`` [T, H * D]."""
+    _check("attn_tc_window.q", q, torch.bfloat16)
+    _check("attn_tc_window.out", out, torch.bfloat16)
+    for name, t in (("k_pages", k_pages), ("v_pages", v_pages)):
+        _check(f"attn_tc_window.{name}", t, torch.bfloat16)
+    for name, t in (("q_start", q_start), ("kv_len", kv_len), ("table", table)):
+        _check(f"attn_tc_window.{name}", t, torch.int32)
+    _dist_args("attn_tc_window", None, sink, q.shape[1])
+    T, H, D = q.shape
+    pages, G, page_size, _ = k_pages.shape
+    if tuple(out.shape) != (T, H * D) or k_pages.shape[3] != D or v_pages.shape != k_pages.shape or H % G:
+        raise KernelError(f"attn_tc_window: q {tuple(q.shape)}, k pages {tuple(k_pages.shape)}, v pages {tuple(v_pages.shape)}, "
+                          f"out {tuple(out.shape)}")
+    code = library().q3_attn_tc_window(q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), q_start.data_ptr(),
+                                       kv_len.data_ptr(), table.data_ptr(), table.shape[1], page_size, pages, int(num_seqs),
+                                       int(max_q_len), H, G, D, float(scale), int(window), _ptr(sink), status.data_ptr(),
+                                       _stream())
+    _done("attn_tc_window", code, f"heads {H}/{G}, dim {D}, page {page_size}, window {window}")
 
 
 def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor,
@@ -2666,16 +2744,16 @@ class ChannelDecay:
         self.logw, self.bonus = logw, bonus
 
 
-def low_rank_decay(low: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor, logw: torch.Tensor) -> None:
-    """logw[t, c] = -exp(sum_r w2[c, r] tanh(low[t, r]) + w0[c]) in float32 (held at -104, whose exponential is zero):
-    the logarithms of decays that a low-rank projection makes.  ``low`` [T, any] (the first ``w2.shape[1]`` columns)."""
-    for name, t in (("low", low), ("w2", w2), ("w0", w0), ("logw", logw)):
+def low_rank_decay(low: torch.Tensor, w2t: torch.Tensor, w0: torch.Tensor, logw: torch.Tensor) -> None:
+    """logw[t, c] = -exp(sum_r w2t[r, c] tanh(low[t, r]) + w0[c]) in float32 (held at -104, whose exponential is zero):
+    the logarithms of decays that a low-rank projection makes.  ``low`` [T, any] (the first ``len(w2t)`` columns)."""
+    for name, t in (("low", low), ("w2t", w2t), ("w0", w0), ("logw", logw)):
         _check(f"low_rank_decay.{name}", t, torch.float32)
     T, ld = low.shape
-    C, R = w2.shape
+    R, C = w2t.shape
     if tuple(logw.shape) != (T, C) or w0.numel() != C or R > ld:
-        raise KernelError(f"low_rank_decay: low {tuple(low.shape)}, w2 {tuple(w2.shape)}, logw {tuple(logw.shape)}")
-    code = library().q3_low_rank_decay(low.data_ptr(), ld, w2.data_ptr(), w0.data_ptr(), logw.data_ptr(), T, C, R, _stream())
+        raise KernelError(f"low_rank_decay: low {tuple(low.shape)}, w2t {tuple(w2t.shape)}, logw {tuple(logw.shape)}")
+    code = library().q3_low_rank_decay(low.data_ptr(), ld, w2t.data_ptr(), w0.data_ptr(), logw.data_ptr(), T, C, R, _stream())
     _done("low_rank_decay", code, f"{C} channels of rank {R}")
 
 

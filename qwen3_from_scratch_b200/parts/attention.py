@@ -509,8 +509,10 @@ class KeptWindowAttention(Mixer):
     has (of the same head counts, sizes and rotation) and does not write it.
 
     One paged cache (planes ``k`` and ``v``), of which the manager keeps the pages of the last ``window`` tokens and those
-    of the first ``keep_first`` (all pages without a window).  The attention kernels are those of the window with pooled blocks, run with blocks of
-    one token whose pages are the token pages themselves and with no more than ``keep_first`` of them.  ``scale`` is used
+    of the first ``keep_first`` (all pages without a window).  The attention kernels are those of the window with pooled
+    blocks, run with blocks of one token whose pages are the token pages themselves and with no more than ``keep_first`` of
+    them; a window alone, with or without a sink, runs on the TMA-fed decode kernel and the tcgen05 portion kernel where those
+    take the sizes.  ``scale`` is used
     as given.  Angles, scores, weights and the gate are float32 in every run.  ``names``: the tensors' names after the
     part's own."""
 
@@ -604,6 +606,11 @@ class KeptWindowAttention(Mixer):
         elif self.sink is not None:  # the kernels take a sink beside a bias: one of zeros
             self.dist_bias = torch.zeros(self.num_heads, 1, dtype=torch.float32, device=rt.device)
         self._q = rt.shared("kwattn.q", rt.max_tokens, self.num_heads, self.dim)
+        self._window_partial = None  # scratch of the kernels for a window alone
+        if (not self.bias and (self.keep_first == 0 or self.window is None)
+                and ops.window_attention_sizes(rt.dtype, self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.scale)):
+            self._window_partial = rt.shared("attn.partial", ops.decode_partial_numel(rt.max_seqs, self.num_heads, self.dim),
+                                             dtype=torch.float32)
         self._partial = None
         if ops.pw_attention_fast(rt.dtype, self.dim, self.vdim):
             self._partial = ops.pw_attn_partial(rt.shared, rt.max_seqs, self.num_heads, self.vdim)
@@ -634,6 +641,12 @@ class KeptWindowAttention(Mixer):
             ops.pw_qkv_post(proj, column, k_col, v_col, H, G, D, Dv, None, None, 0.0, self.dims, self.freq, self.magnitude,
                             ctx.positions, ctx.tok_seq, table, q, k_pages, v_pages, write_cache, status)
         window, first = (ops.NO_WINDOW, 0) if self.window is None else (self.window, self.keep_first)
+        if (self._window_partial is not None and out_scale == 1.0
+                and ops.window_attention_takes(q, k_pages, v_pages, out, ctx, self.scale)):
+            ops.window_attention(q, k_pages, v_pages, out, ctx, table, window, self.scale, self.sink, status, self._window_partial)
+            if self.has_gate:
+                ops.sigmoid_gate(out, proj, v_col + G * Dv)
+            return
         # the kept first tokens are "blocks" of one token read from the token pages, at most keep_first of them
         ops.pooled_window_attention(q, k_pages, v_pages, k_pages, v_pages, ctx, table, table, out, window, 1,
                                     self.scale, None, out_scale, status, self._partial, block_limit=first,

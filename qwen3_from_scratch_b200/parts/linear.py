@@ -115,7 +115,8 @@ class Linear:
 class GroupedLinear:
     """Several projections with inputs of their own (each ``[T, in_features]``) and one output ``[T, sum of rows]``, the
     projections' results side by side.  With up to 16 rows in bfloat16 (and projections of equal sizes in multiples of 16
-    rows) one launch streams all the weights; otherwise a product per projection stores into its columns."""
+    rows) one launch streams all the weights; more rows of equal sizes go to the library's batched product; otherwise a
+    product per projection stores into its columns."""
 
     def __init__(self, weights: Sequence[torch.Tensor], rt: Runtime, tag: str):
         self.rows = [w.shape[0] for w in weights]
@@ -141,6 +142,9 @@ class GroupedLinear:
         out = self._out[:T]
         if self.one_launch and ops.gemm_skinny_takes(T, self.weight) and x.dtype == torch.bfloat16:
             ops.gemm_skinny_groups(x, self.weight, out)
+            return out
+        if len(set(self.rows)) == 1 and not self.full_precision and x.dtype == self.weight.dtype == self.out_dtype:
+            torch.bmm(x, self.weight.view(n, self.rows[0], K).transpose(1, 2), out=out.view(T, n, self.rows[0]).transpose(0, 1))
             return out
         wide, at = self._out32[:T], 0
         for i, rows in enumerate(self.rows):

@@ -673,9 +673,10 @@ class TimeMixing(Mixer, _NamedTensors):
         self.mu = torch.stack([weights[t[f"mu_{s}"]] for s in self.MIXES]).contiguous()
         self.proj = GroupedLinear([weights.pop(t[s]) for s in "rkvg"], rt, tag="tmix.proj")  # columns: r, k, v, g
         w1 = weights.pop(t["w1"])
-        self.w2, self.w0 = weights[t["w2"]], weights[t["w0"]]
-        if w1.shape[0] != self.w2.shape[1]:
-            raise ValueError(f"mixer {self.name}: {t['w1']} leaves {w1.shape[0]} values, {t['w2']} reads {self.w2.shape[1]}")
+        w2, self.w0 = weights[t["w2"]], weights[t["w0"]]
+        if w1.shape[0] != w2.shape[1]:
+            raise ValueError(f"mixer {self.name}: {t['w1']} leaves {w1.shape[0]} values, {t['w2']} reads {w2.shape[1]}")
+        self.w2t = w2.t().contiguous()
         self.low = Linear(_stack_rows([w1]), rt, tag="tmix.low", out_dtype=torch.float32)
         self.bonus, self.norm_weight = weights[t["u"]], weights[t["norm"]]
         self.out_proj = Linear(weights.pop(t["out"]), rt, tag="tmix.out")
@@ -702,7 +703,7 @@ class TimeMixing(Mixer, _NamedTensors):
         n = self.num_heads * self.dim
         proj = self.proj(mix[:4])
         logw, o, gated = self._logw[:T], self._o[:T], self._gated[:T]
-        ops.low_rank_decay(self.low(mix[4]), self.w2, self.w0, logw)
+        ops.low_rank_decay(self.low(mix[4]), self.w2t, self.w0, logw)
         ops.channel_memory_scan(proj, 0, n, 2 * n, ops.ChannelDecay(logw, self.bonus), ctx.state(cache_id, "state"), ctx.q_start,
                                 ctx.slot_ids, ctx.num_seqs, o, self.rt.status, ctx.max_q_len, self._scratch)
         ops.memory_out(o, proj, 3 * n, self.norm_weight, self.norm_eps, "silu", gated, self.num_heads)

@@ -163,14 +163,123 @@ def test_biases_norms_per_head_rotation_and_pages(heads, kv_heads, dim, vdim, di
     assert int((kp.float() == 9.0).all(dim=3).all(dim=1).sum()) == pages * page - T
 
 
-@pytest.mark.parametrize("T,C,R", [(1, 24, 5), (7, 72, 1), (33, 130, 37), (3, 2048, 64), (100, 64, 96)])
+class Batch:
+    """The parts of a step's context that an attention kernel reads: requests with (earlier tokens, tokens of the step), those
+    with a single token first."""
+
+    def __init__(self, portions):
+        self.num_seqs, self.num_decode = len(portions), sum(n == 1 for _, n in portions)
+        self.max_q_len, self.max_kv_len = max(n for _, n in portions), max(past + n for past, n in portions)
+        self.q_start = ints(*([0] + torch.tensor([n for _, n in portions]).cumsum(0).tolist()))
+        self.kv_len = ints(*[past + n for past, n in portions])
+
+
+@pytest.mark.parametrize("H,G,D,page", [(8, 2, 64, 16), (4, 1, 128, 16), (3, 3, 64, 64), (6, 2, 128, 32)])
+@pytest.mark.parametrize("window", [1, 37, 128, 129, 300, 0x7fffffff])
+def test_windowed_attention_of_single_tokens_and_whole_query_tiles(H, G, D, page, window):
+    """The TMA-fed decode kernel and the tcgen05 portion kernel: windows that start inside a tile, at its edge and just beyond
+    it, of the token itself and of everything; portions that start at the request's first token and far behind it, beside single
+    tokens (the first one among them) and alone.  Pages before the windows have been given back (holes in the table),
+    everything that is not a live key is NaN.  Sinks that take nearly all and nothing, or none."""
+    from qwen3_from_scratch_b200.kernels import ops
+    portions = [(1000, 1), (0, 1), (431, 1), (0, 300), (517, 131), (64, 64), (255, 2)]
+    g = torch.Generator().manual_seed(H + D + page)
+    per = -(-1001 // page)
+    total = per * len(portions) + 3
+    k_pages = torch.full((total, G, page, D), float("nan"), dtype=torch.bfloat16)
+    v_pages = k_pages.clone()
+    table = torch.full((len(portions), per), -1, dtype=torch.int32)
+    ids = torch.randperm(total, generator=g).tolist()
+    T = sum(n for _, n in portions)
+    q = torch.randn(T, H, D, generator=g).to(torch.bfloat16)
+    sink = torch.randn(H, generator=g)
+    sink[0], sink[-1] = 9.0, -60.0
+    scale, at = 1.7 / D ** 0.5, 0
+    want = {True: torch.zeros(T, H, D, dtype=F64), False: torch.zeros(T, H, D, dtype=F64)}
+    for b, (past, n) in enumerate(portions):
+        k, v = (torch.randn(past + n, G, D, generator=g).to(torch.bfloat16) for _ in range(2))
+        for j in range(past + n):
+            if (j // page + 1) * page > past - window + 1:  # the page still holds something that the first query reads
+                if table[b, j // page] < 0:
+                    table[b, j // page] = ids.pop()
+                k_pages[table[b, j // page], :, j % page], v_pages[table[b, j // page], :, j % page] = k[j], v[j]
+        back = torch.arange(past, past + n)[:, None] - torch.arange(past + n)[None, :]
+        seen = (back >= 0) & (back < window)
+        for h in range(H):
+            s = (q[at:at + n, h].double() @ k[:, h * G // H].double().t() * scale).masked_fill(~seen, -float("inf"))
+            for taken in (True, False):
+                extra = sink[h].double() if taken else torch.tensor(-float("inf"), dtype=F64)
+                top = torch.maximum(s.max(dim=1).values, extra)[:, None]
+                e = torch.exp(s - top)
+                want[taken][at:at + n, h] = e @ v[:, h * G // H].double() / (e.sum(1, keepdim=True) + torch.exp(extra - top))
+        at += n
+    kd, vd, td = k_pages.cuda(), v_pages.cuda(), table.cuda()
+    partial = torch.full((ops.decode_partial_numel(len(portions), H, D),), float("nan"), device="cuda")
+    singles = sum(n == 1 for _, n in portions)
+    for rows, keep in ((slice(0, len(portions)), slice(0, T)), (slice(0, singles), slice(0, singles)),
+                       (slice(singles, len(portions)), slice(singles, T))):
+        ctx, qd = Batch(portions[rows]), q[keep].contiguous().cuda()
+        for taken in (True, False):
+            out = torch.full((qd.shape[0], H * D), 7.0, dtype=torch.bfloat16, device="cuda")
+            status = ints(0)
+            assert ops.window_attention_takes(qd, kd, vd, out, ctx, scale)
+            ops.window_attention(qd, kd, vd, out, ctx, td[rows].contiguous(), window, scale, sink.cuda() if taken else None, status, partial)
+            assert int(status.item()) == 0
+            expected = want[taken][keep]
+            close(out, expected.reshape(-1, H * D), "bfloat16", f"attention {rows} {taken}", tol=1e-2)
+            close(out.view(-1, H, D)[:, 0], expected[:, 0], "bfloat16", "a head whose sink takes nearly all", tol=1e-2)
+    short = Batch([(9, 1), (5, 128 * G // H - 1)])
+    assert not ops.window_attention_takes(qd, kd, vd, out, short, scale) and not ops.window_attention_takes(qd, kd, vd, out, ctx, -scale)
+    assert not ops.window_attention_takes(qd.float(), kd, vd, out, ctx, scale)
+
+
+@pytest.mark.parametrize("W,E,top,shared", [(2048, 16, 3, True), (40, 7, 2, False), (72, 8, 8, True), (256, 39, 4, True), (136, 1, 1, False),
+                                            (33, 12, 3, True), (64, 60, 5, True)])
+@pytest.mark.parametrize("rows", [1, 16, 70, 600])
+@pytest.mark.parametrize("dtype", list(DT))
+def test_router_with_a_bias_and_the_shared_experts_row(W, E, top, shared, rows, dtype):
+    """Logits with a bias, a softmax over the chosen ones, the shared expert's share from one more row: on the tensor cores in
+    bfloat16 (weights with all the bits of a float32), otherwise lane by lane; a token's result bit for bit the same whatever
+    else is in the step."""
+    from qwen3_from_scratch_b200.kernels import ops
+    g = torch.Generator().manual_seed(W + E + rows)
+    h = torch.randn(rows, W, generator=g).to(DT[dtype])
+    router, bias = torch.randn(E + shared, W, generator=g) * (3.0 / W ** 0.5), torch.randn(E, generator=g)
+    rd, bd = router.cuda(), bias.cuda()
+
+    def route(x):
+        n = x.shape[0]
+        ids, wts = torch.full((n, top), -1, dtype=torch.int32, device="cuda"), torch.zeros(n, top, device="cuda")
+        share = torch.zeros(n, device="cuda") if shared else None
+        ops.moe_route(x.contiguous().cuda(), rd, None, ids, wts, 1.0, "softmax", 1, 1, True, logit_bias=bd, share=share)
+        return ids.cpu(), wts.cpu(), share.cpu() if shared else torch.zeros(n)
+
+    ids, wts, share = route(h)
+    z = h.double() @ router[:E].double().t() + bias.double()
+    clear = 0
+    for t in range(min(rows, 100)):
+        s = z[t].sort(descending=True).values
+        if E > 1 and float((s[:-1] - s[1:]).min()) < 1e-5:
+            continue
+        clear += 1
+        chosen, weights = plain.route(z[t], top)
+        assert ids[t].tolist() == chosen, t
+        close(wts[t], weights, "float32", f"weights of row {t}", tol=2e-5)
+    assert clear > 0.8 * min(rows, 100)
+    if shared:
+        close(share, plain.sigmoid(h.double() @ router[E].double()), "float32", "shares", tol=1e-5)
+    for lo, hi in ((0, 1), (rows // 2, rows // 2 + 2)):
+        assert all(torch.equal(a, b[lo:hi]) for a, b in zip(route(h[lo:hi]), (ids, wts, share)))
+
+
+@pytest.mark.parametrize("T,C,R", [(1, 24, 5), (7, 72, 1), (33, 130, 37), (3, 2048, 64), (100, 64, 96), (700, 200, 64)])
 def test_decays_of_a_low_rank_projection(T, C, R):
     from qwen3_from_scratch_b200.kernels import ops
     g = torch.Generator().manual_seed(C)
     low, w2, w0 = torch.randn(T, R + 3, generator=g), torch.randn(C, R, generator=g), 3 * torch.randn(C, generator=g)
     w0[0], w0[1] = 30.0, -30.0  # gone at once; kept for good
     out = torch.empty(T, C, device="cuda")
-    ops.low_rank_decay(low.cuda(), w2.cuda(), w0.cuda(), out)
+    ops.low_rank_decay(low.cuda(), w2.t().contiguous().cuda(), w0.cuda(), out)
     want = -torch.exp(torch.tanh(low[:, :R].double()) @ w2.double().t() + w0.double())
     assert torch.allclose(out.cpu().double(), want.clamp(min=-104.0), rtol=1e-4, atol=0)
 
@@ -323,7 +432,8 @@ def test_mixer_alone_whole_in_portions_and_beside_another_request(case, dtype):
 
 
 @pytest.mark.parametrize("dtype", list(DT))
-@pytest.mark.parametrize("dim,vdim,heads,kv_heads,window", [(16, 24, 2, 1, 9), (32, 64, 6, 2, 64), (64, 32, 3, 3, 37), (128, 128, 4, 1, 130)])
+@pytest.mark.parametrize("dim,vdim,heads,kv_heads,window", [(16, 24, 2, 1, 9), (32, 64, 6, 2, 64), (64, 32, 3, 3, 37), (128, 128, 4, 1, 130),
+                                                            (64, 64, 12, 3, 101)])
 def test_a_key_just_inside_and_just_outside_the_window_shows(dim, vdim, heads, kv_heads, window, dtype):
     """One token whose key answers every query and whose value stands out: the last position that its window reaches still
     gives its value, the next one nothing of it; a window one longer or shorter would be far off.  Tokens at a page's first and
