@@ -370,22 +370,22 @@ static int memory_scan_sizes(const MemoryIn<T>& in, float* state, const int* q_s
 // ---------------------------------------------------------------- decays from a low-rank projection
 // logw[t, c] = -exp(sum_r w2[c, r] tanh(low[t, r]) + w0[c]), at least LR_LEAST (whose exponential is zero in float32).
 // low: [T, ld]; w2t: [R, C]; w0: [C]; logw: [T, C].  Every sum runs over r in order, so that a token's decays do not depend on how
-// many there are.  For many tokens a block takes TT of them and TC channels, a thread 4 x 4; for a few, a warp per token and
+// many there are.  For many tokens a block takes LR_TT of them and LR_TC channels, a thread 4 x 8; for a few, a warp per token and
 // LF_C channels, with all of their weights in shared memory.
-constexpr int LR_R = 32, LR_TT = 64, LR_TC = 64, LR_THREADS = LR_TT * LR_TC / 16;
+constexpr int LR_R = 32, LR_TT = 64, LR_TC = 128, LR_THREADS = LR_TT * LR_TC / 32;
 constexpr int LF_T = 8, LF_C = 32, LF_MAX_R = 256;
 constexpr float LR_LEAST = -104.f;
 
 __device__ __forceinline__ float log_decay_of(float sum, float w0) { return fmaxf(-expf(sum + w0), LR_LEAST); }
 
-__global__ void __launch_bounds__(LR_THREADS)
+__global__ void __launch_bounds__(LR_THREADS, 4)
 low_rank_decay_kernel(const float* __restrict__ low, int ld, const float* __restrict__ w2t, const float* __restrict__ w0,
                       float* __restrict__ logw, int Ttot, int C, int R) {
   __shared__ __align__(16) float a_s[LR_R][LR_TT + 4], w_s[LR_R][LR_TC + 4];
   const int t0 = blockIdx.y * LR_TT, c0 = blockIdx.x * LR_TC;
-  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;  // channels 4 tx .. 4 tx + 3, tokens 4 ty .. 4 ty + 3
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;  // channels 4 tx .. and 64 + 4 tx .., tokens 4 ty .. 4 ty + 3
   auto weights = [&](int r0) {
-#pragma unroll
+#pragma unroll 4
     for (int i = threadIdx.x; i < LR_TC * LR_R; i += LR_THREADS) {
       const int c = i % LR_TC, r = i / LR_TC;
       w_s[r][c] = c0 + c < C && r0 + r < R ? w2t[(size_t)(r0 + r) * C + c0 + c] : 0.f;
@@ -394,52 +394,57 @@ low_rank_decay_kernel(const float* __restrict__ low, int ld, const float* __rest
   weights(0);  // they do not depend on the kernel before this one
   pdl_wait();
   pdl_launch_dependents();
-  float acc[4][4] = {};
+  float acc[2][4][4] = {};
   for (int r0 = 0; r0 < R; r0 += LR_R) {
     if (r0 > 0) {
       __syncthreads();
       weights(r0);
     }
-#pragma unroll
+#pragma unroll 4
     for (int i = threadIdx.x; i < LR_TT * LR_R; i += LR_THREADS) {
       const int t = i / LR_R, r = i % LR_R;
       a_s[r][t] = t0 + t < Ttot && r0 + r < R ? tanhf(low[(size_t)(t0 + t) * ld + r0 + r]) : 0.f;
     }
     __syncthreads();
-#pragma unroll 8
+#pragma unroll 4
     for (int r = 0; r < LR_R; ++r) {
-      const float4 w = *reinterpret_cast<const float4*>(&w_s[r][4 * tx]);
       const float4 av = *reinterpret_cast<const float4*>(&a_s[r][4 * ty]);
       const float a[4] = {av.x, av.y, av.z, av.w};
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        acc[i][0] = fmaf(a[i], w.x, acc[i][0]);
-        acc[i][1] = fmaf(a[i], w.y, acc[i][1]);
-        acc[i][2] = fmaf(a[i], w.z, acc[i][2]);
-        acc[i][3] = fmaf(a[i], w.w, acc[i][3]);
+      for (int p = 0; p < 2; ++p) {
+        const float4 w = *reinterpret_cast<const float4*>(&w_s[r][64 * p + 4 * tx]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          acc[p][i][0] = fmaf(a[i], w.x, acc[p][i][0]);
+          acc[p][i][1] = fmaf(a[i], w.y, acc[p][i][1]);
+          acc[p][i][2] = fmaf(a[i], w.z, acc[p][i][2]);
+          acc[p][i][3] = fmaf(a[i], w.w, acc[p][i][3]);
+        }
       }
     }
   }
-  const int c = c0 + 4 * tx;
-  if (c >= C) return;
   const bool by4 = (C & 3) == 0;
-  float off[4];
 #pragma unroll
-  for (int j = 0; j < 4; ++j) off[j] = c + j < C ? w0[c + j] : 0.f;
+  for (int p = 0; p < 2; ++p) {
+    const int c = c0 + 64 * p + 4 * tx;
+    if (c >= C) continue;
+    float off[4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int t = t0 + 4 * ty + i;
-    if (t >= Ttot) continue;
-    float* dst = logw + (size_t)t * C + c;
-    const float4 v = make_float4(log_decay_of(acc[i][0], off[0]), log_decay_of(acc[i][1], off[1]), log_decay_of(acc[i][2], off[2]),
-                                 log_decay_of(acc[i][3], off[3]));
-    if (by4) {
-      *reinterpret_cast<float4*>(dst) = v;
-    } else {
-      const float e[4] = {v.x, v.y, v.z, v.w};
+    for (int j = 0; j < 4; ++j) off[j] = c + j < C ? w0[c + j] : 0.f;
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (c + j < C) dst[j] = e[j];
+    for (int i = 0; i < 4; ++i) {
+      const int t = t0 + 4 * ty + i;
+      if (t >= Ttot) continue;
+      float* dst = logw + (size_t)t * C + c;
+      const float v[4] = {log_decay_of(acc[p][i][0], off[0]), log_decay_of(acc[p][i][1], off[1]),
+                          log_decay_of(acc[p][i][2], off[2]), log_decay_of(acc[p][i][3], off[3])};
+      if (by4) {
+        *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (c + j < C) dst[j] = v[j];
+      }
     }
   }
 }

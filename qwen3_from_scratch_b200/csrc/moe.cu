@@ -231,17 +231,18 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
                    wts + (size_t)(t0 + k) * c.top, lane);
 }
 
-// Sixteen tokens to a block; the eight warps share the sum over W, in groups of 32 values of which lane t of a row takes
-// k = 8 t .. 8 t + 7 (see gemm_skinny.cu), and meet in shared memory in order.  W a multiple of 8.
-constexpr int MR_TOK = 16, MR_WARPS = 8, MR_MAX_ROWS = 40;
+// Sixteen tokens to a block; the warps share the sum over W, in groups of 32 values of which lane t of a row takes
+// k = 8 t .. 8 t + 7 (see gemm_skinny.cu), and meet in shared memory in order.  A warp's first MR_BATCH groups of the router are
+// asked for before the wait on the kernel before.  W a multiple of 8.
+constexpr int MR_TOK = 16, MR_WARPS = 16, MR_MAX_ROWS = 40, MR_BATCH = 2;
 
 template <int NT>  // tiles of eight router rows
 __global__ void __launch_bounds__(MR_WARPS * 32)
 moe_route_mma_kernel(const __nv_bfloat16* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ bias,
                      const float* __restrict__ zbias, int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ share,
                      int Ttot, int W, Choice c) {
-  extern __shared__ __align__(16) float score[];  // [16][E] scores, [16][E] keys, [16][groups] flags
-  __shared__ float part[MR_WARPS][MR_TOK][8 * NT + 1];
+  extern __shared__ __align__(16) float score[];  // [16][E] scores, [16][E] keys, [16][groups] flags; before them the partial sums
+  float(*part)[MR_TOK][8 * NT + 1] = reinterpret_cast<float(*)[MR_TOK][8 * NT + 1]>(score + ((MR_TOK * (2 * c.E + c.groups) + 3) & ~3));
   unsigned* key = reinterpret_cast<unsigned*>(score + MR_TOK * c.E);
   unsigned* kept = key + MR_TOK * c.E;
   const int t0 = blockIdx.x * MR_TOK, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, gid = lane >> 2, tid4 = lane & 3;
@@ -251,42 +252,55 @@ moe_route_mma_kernel(const __nv_bfloat16* __restrict__ h, const float* __restric
   float acc[NT][4];
 #pragma unroll
   for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  float4 wv[MR_BATCH][NT][2];
+  auto fetch = [&](int g0) {
+#pragma unroll
+    for (int u = 0; u < MR_BATCH; ++u)
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        const int k = (g0 + u) * 32 + 8 * tid4, e = nt * 8 + gid;
+        const bool in = g0 + u < g_hi && k < W && e < rows;
+        const float4* p = reinterpret_cast<const float4*>(wr + (size_t)e * W + k);
+        wv[u][nt][0] = in ? p[0] : make_float4(0.f, 0.f, 0.f, 0.f);
+        wv[u][nt][1] = in ? p[1] : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+  };
+  fetch(g_lo);
   pdl_wait();
   pdl_launch_dependents();
   const __nv_bfloat16* x_lo = h + (size_t)min(t0 + gid, Ttot - 1) * W;
   const __nv_bfloat16* x_hi = h + (size_t)min(t0 + gid + 8, Ttot - 1) * W;
-#pragma unroll 2
-  for (int g = g_lo; g < g_hi; ++g) {
-    const int k = g * 32 + 8 * tid4;
-    const bool in = k < W;
-    const uint4 lo = in ? *reinterpret_cast<const uint4*>(x_lo + k) : make_uint4(0, 0, 0, 0);
-    const uint4 hi = in ? *reinterpret_cast<const uint4*>(x_hi + k) : make_uint4(0, 0, 0, 0);
-    const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
+  for (int g0 = g_lo; g0 < g_hi; g0 += MR_BATCH) {
+    uint4 lo[MR_BATCH], hi[MR_BATCH];
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) {
-      const int e = nt * 8 + gid;
-      float w[8];
-      if (in && e < rows) {
-        const float4 u = *reinterpret_cast<const float4*>(wr + (size_t)e * W + k);
-        const float4 v = *reinterpret_cast<const float4*>(wr + (size_t)e * W + k + 4);
-        w[0] = u.x, w[1] = u.y, w[2] = u.z, w[3] = u.w, w[4] = v.x, w[5] = v.y, w[6] = v.z, w[7] = v.w;
-      } else {
+    for (int u = 0; u < MR_BATCH; ++u) {
+      const int k = (g0 + u) * 32 + 8 * tid4;
+      const bool in = g0 + u < g_hi && k < W;
+      lo[u] = in ? *reinterpret_cast<const uint4*>(x_lo + k) : make_uint4(0, 0, 0, 0);
+      hi[u] = in ? *reinterpret_cast<const uint4*>(x_hi + k) : make_uint4(0, 0, 0, 0);
+    }
+    if (g0 > g_lo) fetch(g0);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) w[i] = 0.f;
-      }
+    for (int u = 0; u < MR_BATCH; ++u) {
+      const uint32_t a0[4] = {lo[u].x, hi[u].x, lo[u].y, hi[u].y}, a1[4] = {lo[u].z, hi[u].z, lo[u].w, hi[u].w};
 #pragma unroll
-      for (int piece = 0; piece < 3; ++piece) {  // the upper eight bits, the middle, the lower
-        uint32_t b[4];
+      for (int nt = 0; nt < NT; ++nt) {
+        float w[8] = {wv[u][nt][0].x, wv[u][nt][0].y, wv[u][nt][0].z, wv[u][nt][0].w,
+                      wv[u][nt][1].x, wv[u][nt][1].y, wv[u][nt][1].z, wv[u][nt][1].w};
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const __nv_bfloat162 p = __floats2bfloat162_rn(w[2 * i], w[2 * i + 1]);
-          const float2 f = __bfloat1622float2(p);
-          b[i] = *reinterpret_cast<const uint32_t*>(&p);
-          w[2 * i] -= f.x;
-          w[2 * i + 1] -= f.y;
+        for (int piece = 0; piece < 3; ++piece) {  // the upper eight bits, the middle, the lower
+          uint32_t b[4];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const __nv_bfloat162 p = __floats2bfloat162_rn(w[2 * i], w[2 * i + 1]);
+            const float2 f = __bfloat1622float2(p);
+            b[i] = *reinterpret_cast<const uint32_t*>(&p);
+            w[2 * i] -= f.x;
+            w[2 * i + 1] -= f.y;
+          }
+          mma_bf16(acc[nt], a0, b[0], b[1]);
+          mma_bf16(acc[nt], a1, b[2], b[3]);
         }
-        mma_bf16(acc[nt], a0, b[0], b[1]);
-        mma_bf16(acc[nt], a1, b[2], b[3]);
       }
     }
   }
@@ -399,16 +413,17 @@ extern "C" int q3_moe_route(const void* h, const float* wr, const float* bias, c
   const q3::Choice choice{E, top, softmax, groups, keep, renorm, scale};
   const int rows = E + (share ? 1 : 0);
   if (dtype == Q3_BF16 && rows <= q3::MR_MAX_ROWS && W % 8 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)wr % 16 == 0) {
-    auto go = [&](auto kernel) {
+    auto go = [&](auto kernel, int tiles) {
       q3::launch(kernel, dim3((T + q3::MR_TOK - 1) / q3::MR_TOK), dim3(q3::MR_WARPS * 32),
-                 (size_t)q3::MR_TOK * (2 * E + groups) * sizeof(float), stream, (const __nv_bfloat16*)h, wr, bias, zbias, ids, wts,
+                 ((size_t)((q3::MR_TOK * (2 * E + groups) + 3) & ~3) + q3::MR_WARPS * q3::MR_TOK * (8 * tiles + 1)) * sizeof(float),
+                 stream, (const __nv_bfloat16*)h, wr, bias, zbias, ids, wts,
                  share, T, W, choice);
       return q3::launch_status();
     };
-    if (rows <= 8) return go(q3::moe_route_mma_kernel<1>);
-    if (rows <= 16) return go(q3::moe_route_mma_kernel<2>);
-    if (rows <= 24) return go(q3::moe_route_mma_kernel<3>);
-    return go(q3::moe_route_mma_kernel<5>);
+    if (rows <= 8) return go(q3::moe_route_mma_kernel<1>, 1);
+    if (rows <= 16) return go(q3::moe_route_mma_kernel<2>, 2);
+    if (rows <= 24) return go(q3::moe_route_mma_kernel<3>, 3);
+    return go(q3::moe_route_mma_kernel<5>, 5);
   }
   // many tokens: eight to a block, so that the experts' rows are read an eighth as often
   constexpr int MANY = 8;

@@ -123,6 +123,7 @@ head_qkv_post_kernel(const T* __restrict__ proj, int ld, int k_col, int v_col, i
     width = is_v ? Dv : D;
     col = is_q ? u * D : (is_v ? v_col + (u - H - G) * Dv : k_col + (u - H) * D);
   };
+  const T* row = proj + (size_t)t * ld;
   PwPack<T, V> next[PER];
   auto fetch = [&](int u) {  // a head ahead, so that its loads are in flight while the head before is worked on
     int col, width;
@@ -130,7 +131,7 @@ head_qkv_post_kernel(const T* __restrict__ proj, int ld, int k_col, int v_col, i
 #pragma unroll
     for (int k = 0; k < PER; ++k) {
       const int i = (k * 32 + lane) * V;
-      if (i < width) next[k] = *reinterpret_cast<const PwPack<T, V>*>(proj + (size_t)t * ld + col + i);
+      if (i < width) next[k] = *reinterpret_cast<const PwPack<T, V>*>(row + col + i);
     }
   };
   if (warp < H) fetch(warp);

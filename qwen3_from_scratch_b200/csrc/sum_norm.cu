@@ -44,11 +44,11 @@ __device__ __forceinline__ SnPack<float, V> sum_term(const SumTerms<T>& terms, i
   return x;
 }
 
-// What the terms of row t are multiplied by, by the whole block.
-template <typename T, int V>
-__device__ __forceinline__ void sum_factors(const SumTerms<T>& terms, int t, int W, float* red, float (&factor)[SN_TERMS]) {
+// What the terms of row t are multiplied by, by the whole block.  N: how many terms there may be.
+template <typename T, int V, int N>
+__device__ __forceinline__ void sum_factors(const SumTerms<T>& terms, int t, int W, float* red, float (&factor)[N]) {
 #pragma unroll
-  for (int k = 0; k < SN_TERMS; ++k) {
+  for (int k = 0; k < N; ++k) {
     factor[k] = 1.f;
     if (k < terms.count && terms.weight[k]) {
       float ss = 0.f;
@@ -62,13 +62,23 @@ __device__ __forceinline__ void sum_factors(const SumTerms<T>& terms, int t, int
   }
 }
 
-// V values of the new row t from column i on.
-template <typename T, int V>
+// A thread's first V values of row t of the stream, asked for before the terms' statistics are worked out.
+template <int V>
+__device__ __forceinline__ SnPack<float, V> sum_first(const float* __restrict__ stream, int t, int W) {
+  SnPack<float, V> x{};
+  if ((int)threadIdx.x * V < W) x = *reinterpret_cast<const SnPack<float, V>*>(stream + (size_t)t * W + threadIdx.x * V);
+  return x;
+}
+
+// V values of the new row t from column i on; `first`: what sum_first returned.
+template <typename T, int V, int N>
 __device__ __forceinline__ SnPack<float, V> sum_values(const float* __restrict__ stream, const SumTerms<T>& terms,
-                                                       const float (&factor)[SN_TERMS], int t, int W, int i) {
-  SnPack<float, V> x = *reinterpret_cast<const SnPack<float, V>*>(stream + (size_t)t * W + i);
+                                                       const float (&factor)[N], const SnPack<float, V>& first, int t,
+                                                       int W, int i) {
+  SnPack<float, V> x = first;
+  if (i != (int)threadIdx.x * V) x = *reinterpret_cast<const SnPack<float, V>*>(stream + (size_t)t * W + i);
 #pragma unroll
-  for (int k = 0; k < SN_TERMS; ++k) {
+  for (int k = 0; k < N; ++k) {
     if (k >= terms.count) continue;
     const SnPack<float, V> d = sum_term<T, V>(terms, k, (size_t)t * W, i);
     if (terms.weight[k]) {
@@ -84,7 +94,7 @@ __device__ __forceinline__ SnPack<float, V> sum_values(const float* __restrict__
 }
 
 // One block per row; V values per access (4 where width and pointers allow it, else 1).
-template <typename T, int V>
+template <typename T, int V, int N>
 __global__ void sum_norm_kernel(float* __restrict__ stream, SumTerms<T> terms, const float* __restrict__ w1,
                                 T* __restrict__ out1, const float* __restrict__ w2, T* __restrict__ out2,
                                 const int* __restrict__ rows, int W, float eps) {
@@ -93,11 +103,12 @@ __global__ void sum_norm_kernel(float* __restrict__ stream, SumTerms<T> terms, c
   pdl_wait();
   pdl_launch_dependents();
   const int t = rows ? rows[blockIdx.x] : blockIdx.x;
-  float factor[SN_TERMS];
-  sum_factors<T, V>(terms, t, W, red, factor);
+  const SnPack<float, V> row = sum_first<V>(stream, t, W);
+  float factor[N];
+  sum_factors<T, V, N>(terms, t, W, red, factor);
   float ss = 0.f;
   for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
-    const SnPack<float, V> x = sum_values<T, V>(stream, terms, factor, t, W, i);
+    const SnPack<float, V> x = sum_values<T, V, N>(stream, terms, factor, row, t, W, i);
     if (!rows && terms.count) *reinterpret_cast<SnPack<float, V>*>(stream + (size_t)t * W + i) = x;
     if (!w1) {
       if (out1) {
@@ -132,7 +143,7 @@ __global__ void sum_norm_kernel(float* __restrict__ stream, SumTerms<T> terms, c
 }
 
 // One block per token, as above.  mu: [M, W]; out: [M, T, W]; state: [num_slots, W].
-template <typename T, int V>
+template <typename T, int V>  // at most one term
 __global__ void sum_mix_kernel(float* __restrict__ stream, SumTerms<T> terms, const float* __restrict__ mu, int M,
                                float* __restrict__ state, const int* __restrict__ q_start, const int* __restrict__ tok_seq,
                                const int* __restrict__ slot_ids, int num_slots, T* __restrict__ out, int W, int* status) {
@@ -145,10 +156,11 @@ __global__ void sum_mix_kernel(float* __restrict__ stream, SumTerms<T> terms, co
   const bool first = t == q_start[b];
   const int last = q_start[b + 1] - 1;
   float* st = live ? state + (size_t)slot * W : nullptr;
-  float factor[SN_TERMS];
-  sum_factors<T, V>(terms, t, W, red, factor);
+  const SnPack<float, V> row = sum_first<V>(stream, t, W);
+  float factor[1];
+  sum_factors<T, V, 1>(terms, t, W, red, factor);
   for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
-    SnPack<float, V> x = sum_values<T, V>(stream, terms, factor, t, W, i);
+    const SnPack<float, V> x = sum_values<T, V, 1>(stream, terms, factor, row, t, W, i);
     if (terms.count) *reinterpret_cast<SnPack<float, V>*>(stream + (size_t)t * W + i) = x;
     SnPack<float, V> p{};
     if (live) {
@@ -198,12 +210,12 @@ static int sum_norm_launch(float* stream, const void* const* delta, const float*
               (uintptr_t)out1 % 16 == 0 && (uintptr_t)out2 % 16 == 0;
   const size_t smem = w1 ? (size_t)W * sizeof(float) : 0;
   const int threads = sum_norm_threads(W);
-  if (wide)
-    launch(sum_norm_kernel<T, 4>, dim3(n), dim3(threads), smem, cuda_stream, stream, terms, w1, (T*)out1, w2, (T*)out2, rows,
-           W, eps);
-  else
-    launch(sum_norm_kernel<T, 1>, dim3(n), dim3(threads), smem, cuda_stream, stream, terms, w1, (T*)out1, w2, (T*)out2, rows,
-           W, eps);
+  auto go = [&](auto kernel) {
+    launch(kernel, dim3(n), dim3(threads), smem, cuda_stream, stream, terms, w1, (T*)out1, w2, (T*)out2, rows, W, eps);
+  };
+  if (wide && count <= 1) go(sum_norm_kernel<T, 4, 1>);
+  else if (wide) go(sum_norm_kernel<T, 4, SN_TERMS>);
+  else go(sum_norm_kernel<T, 1, SN_TERMS>);
   if (!rows) note_stream_written();
   return launch_status();
 }
